@@ -14,8 +14,10 @@ BASED_BF16 = 1
 IMPL_AUTO = 0
 IMPL_SIMT = 1
 IMPL_TCGEN05 = 2
+ERR_IMPL = -5
 
 _I64P = POINTER(c_int64)
+_POS = [c_void_p, c_int]   # position of a call's first token: device int32 per batch row, or a scalar
 
 # name -> (restype, argtypes); every symbol the header declares
 SIGNATURES = {
@@ -48,6 +50,16 @@ SIGNATURES = {
     "based_tp_outproj_allreduce_emulated": (c_int, [POINTER(c_void_p), POINTER(c_void_p), c_void_p, POINTER(c_void_p)]
                                             + [c_int] * 3 + [c_int64] * 2 + [POINTER(c_void_p), c_int, c_int, c_void_p]),
     "based_rotary_qkv_cache": (c_int, [c_void_p] + [c_int] * 4 + [_I64P, c_void_p, c_void_p, c_void_p, _I64P, c_void_p]),
+    # stateful mixers of hybrid stacks; _POS = (offsets, offset)
+    "based_stream_norm": (c_int, [c_void_p] * 3 + [c_int64, c_void_p, c_int64, c_float] + [c_void_p] * 5
+                          + [c_int64, c_int, c_float, c_int, c_void_p]),
+    "based_rmsnorm": (c_int, [c_void_p] * 3 + [c_int64, c_int, c_int64, c_int64, c_float, c_int, c_void_p]),
+    "based_short_conv": (c_int, [c_void_p] * 5 + [c_int] * 4 + [_I64P] * 2 + _POS + [c_int, c_int, c_void_p]),
+    "based_latent_prepare": (c_int, [c_void_p] * 6 + [c_int] * 8 + [_I64P] * 3 + _POS + [c_float, c_int, c_void_p]),
+    "based_split_key_attention": (c_int, [c_void_p] * 7 + [c_int] * 6 + [_I64P] * 7 + _POS + [c_float, c_int, c_void_p]),
+    "based_delta_prefill": (c_int, [c_void_p] * 11 + [c_int] * 6 + [_I64P] * 6 + _POS + [c_float, c_int, c_void_p]),
+    "based_delta_step": (c_int, [c_void_p] * 10 + [c_int] * 6 + [c_int64] * 3 + _POS + [c_float, c_int, c_void_p]),
+    "based_rglru": (c_int, [c_void_p] * 8 + [c_int] * 4 + [_I64P] * 4 + _POS + [c_int, c_void_p]),
 }
 
 _lib = None

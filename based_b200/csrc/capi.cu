@@ -327,4 +327,124 @@ int based_tp_outproj_allreduce_emulated(const void* const* x, const void* const*
                                      world, 1, static_cast<cudaStream_t>(stream));
 }
 
+// ------------------------------------------------------------------ stateful mixers of the hybrid stacks
+
+int based_stream_norm(const void* tokens, const void* table, const void* table_norm, int64_t V, const void* branch,
+                      int64_t branch_row_stride, float mult, void* residual, const void* w1, const void* w2, void* out1,
+                      void* out2, int64_t M, int D, float eps, int io_dtype, void* stream) {
+  if (!residual || !w1 || !out1 || (w2 == nullptr) != (out2 == nullptr)) return BASED_ERR_NULL;
+  if (tokens && (!table || !table_norm || V <= 0 || branch)) return BASED_ERR_NULL;
+  if (!dtype_ok(io_dtype)) return BASED_ERR_DTYPE;
+  if (M < 0 || D <= 0) return BASED_ERR_SHAPE;
+  if (M == 0) return BASED_OK;
+  return launch_stream_norm(static_cast<const int64_t*>(tokens), table, table_norm, V, branch, branch_row_stride, mult,
+                            static_cast<float*>(residual), w1, w2, out1, out2, M, D, eps, io_dtype,
+                            static_cast<cudaStream_t>(stream));
+}
+
+int based_rmsnorm(const void* x, const void* weight, void* out, int64_t M, int D, int64_t x_row_stride,
+                  int64_t out_row_stride, float eps, int io_dtype, void* stream) {
+  if (!x || !weight || !out) return BASED_ERR_NULL;
+  if (!dtype_ok(io_dtype)) return BASED_ERR_DTYPE;
+  if (M < 0 || D <= 0) return BASED_ERR_SHAPE;
+  if (M == 0) return BASED_OK;
+  if (M > 2147483647LL) return BASED_ERR_TOO_LARGE;
+  return launch_rmsnorm(x, weight, out, M, D, x_row_stride, out_row_stride, eps, io_dtype, static_cast<cudaStream_t>(stream));
+}
+
+int based_short_conv(const void* x, void* y, void* ring, const void* weight, const void* bias, int B, int L, int C,
+                     int taps, const int64_t x_strides[2], const int64_t y_strides[2], const int32_t* offsets, int offset,
+                     int silu, int io_dtype, void* stream) {
+  if (!x || !y || !weight || !x_strides || !y_strides) return BASED_ERR_NULL;
+  if (!dtype_ok(io_dtype)) return BASED_ERR_DTYPE;
+  if (B < 0 || L < 0 || C <= 0 || taps < 1 || offset < 0) return BASED_ERR_SHAPE;
+  if (!ring && (offsets || offset > 0)) return BASED_ERR_NULL;
+  if (B == 0 || L == 0) return BASED_OK;
+  return launch_short_conv(x, y, ring, weight, bias, B, L, C, taps, s2(x_strides), s2(y_strides), offsets, offset, silu,
+                           io_dtype, static_cast<cudaStream_t>(stream));
+}
+
+int based_latent_prepare(const void* z, const void* norm_weight, void* cache, void* q, const void* cos_table,
+                         const void* sin_table, int table_len, int B, int L, int H, int kv_rank, int rot_dim, int dim,
+                         int max_len, const int64_t z_strides[2], const int64_t cache_strides[2],
+                         const int64_t q_strides[2], const int32_t* offsets, int offset, float eps, int io_dtype,
+                         void* stream) {
+  if (!cos_table || !sin_table || (z && (!norm_weight || !cache || !z_strides || !cache_strides)) || (q && !q_strides))
+    return BASED_ERR_NULL;
+  if (!dtype_ok(io_dtype)) return BASED_ERR_DTYPE;
+  if (B < 0 || L < 0 || H <= 0 || kv_rank <= 0 || rot_dim <= 0 || rot_dim % 2 || dim < 0 || offset < 0) return BASED_ERR_SHAPE;
+  if (!offsets && ((int64_t)offset + L > max_len || (int64_t)offset + L > table_len)) return BASED_ERR_SHAPE;
+  if (B == 0 || L == 0) return BASED_OK;
+  const int64_t zero[2] = {0, 0};
+  const int64_t *zs = z ? z_strides : zero, *cs = z ? cache_strides : zero, *qs = q ? q_strides : zero;
+  return launch_latent_prepare(z, norm_weight, cache, q, static_cast<const float*>(cos_table),
+                               static_cast<const float*>(sin_table), table_len, B, L, H, kv_rank, rot_dim, dim, max_len,
+                               zs[0], zs[1], cs[0], cs[1], qs[0], qs[1], offsets, offset, eps, io_dtype,
+                               static_cast<cudaStream_t>(stream));
+}
+
+int based_split_key_attention(const void* q1, const void* q2, const void* k1, const void* k2, const void* v,
+                              const void* gate, void* out, int B, int L, int H, int d1, int d2, int dv,
+                              const int64_t q1_strides[3], const int64_t q2_strides[3], const int64_t k1_strides[3],
+                              const int64_t k2_strides[3], const int64_t v_strides[3], const int64_t out_strides[3],
+                              const int64_t gate_strides[2], const int32_t* offsets, int offset, float scale,
+                              int io_dtype, void* stream) {
+  if (!q1 || !q2 || !k1 || !k2 || !v || !out || (gate && !gate_strides)) return BASED_ERR_NULL;
+  if (!q1_strides || !q2_strides || !k1_strides || !k2_strides || !v_strides || !out_strides) return BASED_ERR_NULL;
+  if (!dtype_ok(io_dtype)) return BASED_ERR_DTYPE;
+  if (B < 0 || L < 0 || H <= 0 || d1 <= 0 || d2 < 0 || dv <= 0 || offset < 0) return BASED_ERR_SHAPE;
+  if (B == 0 || L == 0) return BASED_OK;
+  return launch_split_key_attention(q1, q2, k1, k2, v, gate, out, B, L, H, d1, d2, dv, s3_blh(q1_strides),
+                                    s3_blh(q2_strides), s3_blh(k1_strides), s3_blh(k2_strides), s3_blh(v_strides),
+                                    s3_blh(out_strides), gate ? gate_strides[0] : 0, gate ? gate_strides[1] : 0, offsets,
+                                    offset, scale, io_dtype, static_cast<cudaStream_t>(stream));
+}
+
+int based_delta_prefill(const void* q, const void* k, const void* v, const void* z, const void* a, const void* b,
+                        const void* A_log, const void* dt_bias, const void* norm_weight, void* state, void* out, int B,
+                        int L, int H, int Hk, int d, int dv, const int64_t q_strides[2], const int64_t k_strides[2],
+                        const int64_t v_strides[2], const int64_t z_strides[2], const int64_t gate_strides[2],
+                        const int64_t out_strides[2], const int32_t* offsets, int offset, float eps, int io_dtype,
+                        void* stream) {
+  if (!q || !k || !v || !z || !a || !b || !A_log || !dt_bias || !norm_weight || !state || !out) return BASED_ERR_NULL;
+  if (!q_strides || !k_strides || !v_strides || !z_strides || !gate_strides || !out_strides) return BASED_ERR_NULL;
+  if (!dtype_ok(io_dtype)) return BASED_ERR_DTYPE;
+  if (B < 0 || L < 0 || H <= 0 || Hk <= 0 || H % Hk || d <= 0 || dv <= 0 || offset < 0) return BASED_ERR_SHAPE;
+  if (B == 0 || L == 0) return BASED_OK;
+  return launch_delta_recurrent(q, k, v, z, static_cast<const float*>(a), static_cast<const float*>(b),
+                                static_cast<const float*>(A_log), static_cast<const float*>(dt_bias), norm_weight,
+                                static_cast<float*>(state), out, B, L, H, Hk, d, dv, s2(q_strides), s2(k_strides),
+                                s2(v_strides), s2(z_strides), s2(gate_strides), s2(out_strides), offsets, offset, eps,
+                                io_dtype, static_cast<cudaStream_t>(stream));
+}
+
+int based_delta_step(const void* x, const void* conv_weight, void* ring, const void* a, const void* b, const void* A_log,
+                     const void* dt_bias, const void* norm_weight, void* state, void* out, int B, int H, int Hk, int d,
+                     int dv, int taps, int64_t x_stride, int64_t gate_stride, int64_t out_stride, const int32_t* offsets,
+                     int offset, float eps, int io_dtype, void* stream) {
+  if (!x || !conv_weight || !ring || !a || !b || !A_log || !dt_bias || !norm_weight || !state || !out) return BASED_ERR_NULL;
+  if (!dtype_ok(io_dtype)) return BASED_ERR_DTYPE;
+  if (B < 0 || H <= 0 || Hk <= 0 || H % Hk || d <= 0 || dv <= 0 || taps < 1 || offset < 0) return BASED_ERR_SHAPE;
+  if (B == 0) return BASED_OK;
+  return launch_delta_step(x, conv_weight, ring, static_cast<const float*>(a), static_cast<const float*>(b),
+                           static_cast<const float*>(A_log), static_cast<const float*>(dt_bias), norm_weight,
+                           static_cast<float*>(state), out, B, H, Hk, d, dv, taps, x_stride, gate_stride, out_stride,
+                           offsets, offset, eps, io_dtype, static_cast<cudaStream_t>(stream));
+}
+
+int based_rglru(const void* u, const void* y, const void* gates, const void* r_bias, const void* i_bias, const void* lam,
+                void* state, void* out, int B, int L, int W, int block_width, const int64_t u_strides[2],
+                const int64_t y_strides[2], const int64_t out_strides[2], const int64_t gate_strides[2],
+                const int32_t* offsets, int offset, int io_dtype, void* stream) {
+  if (!u || !y || !gates || !r_bias || !i_bias || !lam || !state || !out) return BASED_ERR_NULL;
+  if (!u_strides || !y_strides || !out_strides || !gate_strides) return BASED_ERR_NULL;
+  if (!dtype_ok(io_dtype)) return BASED_ERR_DTYPE;
+  if (B < 0 || L < 0 || W <= 0 || block_width <= 0 || W % block_width || offset < 0) return BASED_ERR_SHAPE;
+  if (B == 0 || L == 0) return BASED_OK;
+  return launch_rglru(u, y, static_cast<const float*>(gates), r_bias, i_bias, static_cast<const float*>(lam),
+                      static_cast<float*>(state), out, B, L, W, block_width, s2(u_strides), s2(y_strides),
+                      s2(out_strides), gate_strides[0], gate_strides[1], offsets, offset, io_dtype,
+                      static_cast<cudaStream_t>(stream));
+}
+
 }  // extern "C"

@@ -117,4 +117,34 @@ int launch_swa_decode(const void* q, const void* k_new, const void* v_new, void*
                       Strides2 sq, Strides2 sk, Strides2 sv, Strides2 so, int window_left, float scale,
                       int io_dtype, cudaStream_t stream);
 
+// Stateful mixers of the hybrid stacks.  offsets (device, one per batch row) or offset: position of a call's first token.
+int launch_stream_norm(const int64_t* tokens, const void* table, const void* table_norm, int64_t V, const void* branch,
+                       int64_t branch_stride, float mult, float* residual, const void* w1, const void* w2, void* out1,
+                       void* out2, int64_t M, int D, float eps, int io_dtype, cudaStream_t stream);
+int launch_rmsnorm(const void* x, const void* w, void* out, int64_t M, int D, int64_t sx, int64_t so, float eps,
+                   int io_dtype, cudaStream_t stream);
+int launch_short_conv(const void* x, void* y, void* ring, const void* w, const void* bias, int B, int L, int C, int taps,
+                      Strides2 sx, Strides2 sy, const int32_t* offsets, int offset, int silu, int io_dtype,
+                      cudaStream_t stream);
+int launch_latent_prepare(const void* z, const void* norm_w, void* cache, void* q, const float* cosv, const float* sinv,
+                          int table_len, int B, int L, int H, int r, int rd, int d, int max_len, int64_t zb, int64_t zl,
+                          int64_t cb, int64_t cl, int64_t qb, int64_t ql, const int32_t* offsets, int offset, float eps,
+                          int io_dtype, cudaStream_t stream);
+int launch_split_key_attention(const void* q1, const void* q2, const void* k1, const void* k2, const void* v,
+                               const void* gate, void* out, int B, int L, int H, int d1, int d2, int dv, Strides3 sq1,
+                               Strides3 sq2, Strides3 sk1, Strides3 sk2, Strides3 sv, Strides3 so, int64_t gb, int64_t gl,
+                               const int32_t* offsets, int offset, float scale, int io_dtype, cudaStream_t stream);
+int launch_delta_recurrent(const void* q, const void* k, const void* v, const void* z, const float* a, const float* b,
+                           const float* A_log, const float* dt_bias, const void* norm_w, float* state, void* out, int B,
+                           int L, int H, int Hk, int d, int dv, Strides2 sq, Strides2 sk, Strides2 sv, Strides2 sz,
+                           Strides2 sg, Strides2 so, const int32_t* offsets, int offset, float eps, int io_dtype,
+                           cudaStream_t stream);
+int launch_delta_step(const void* x, const void* conv_w, void* ring, const float* a, const float* b, const float* A_log,
+                      const float* dt_bias, const void* norm_w, float* state, void* out, int B, int H, int Hk, int d,
+                      int dv, int taps, int64_t sx, int64_t sg, int64_t so, const int32_t* offsets, int offset, float eps,
+                      int io_dtype, cudaStream_t stream);
+int launch_rglru(const void* u, const void* y, const float* gates, const void* rb, const void* ib, const float* lam,
+                 float* state, void* out, int B, int L, int W, int bw, Strides2 su, Strides2 sy, Strides2 so,
+                 int64_t g_block, int64_t g_row, const int32_t* offsets, int offset, int io_dtype, cudaStream_t stream);
+
 }  // namespace based

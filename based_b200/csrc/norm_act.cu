@@ -9,8 +9,13 @@
 //    Replaces `y, gate = y.chunk(2, dim=-1); y = swiglu(gate, y)` / F.glu in GatedMlp.forward
 //    (based/models/mlp.py:141-154), where the reference uses flash-attn's jiterator swiglu.
 //
-// Both are HBM-bound; 16-byte vector accesses, fp32 arithmetic, one read of every input.
-#include "common.cuh"
+//  * the norm step of a PARALLEL block (x <- x + m * (mixer(norm1(x)) + mlp(norm2(x)))): the previous block's scaled
+//    branch sum is added to the fp32 residual stream and the new stream is normed once and scaled by TWO weights
+//    (the two norms of one x share their root mean square).  With token ids instead of a branch the row is
+//    norm(embedding[token]), so a model's first step is the same launch.
+//
+// All are HBM-bound; 16-byte vector accesses, fp32 arithmetic, one read of every input.
+#include "seq_common.cuh"
 
 namespace based {
 namespace {
@@ -149,6 +154,118 @@ __global__ void __launch_bounds__(NORM_THREADS) add_rmsnorm_kernel(const NormPar
   }
 }
 
+__device__ __forceinline__ float block_sum(float v) {
+  __shared__ float part[NORM_THREADS / 32];
+  __syncthreads();  // part may still be read by a previous call
+  v = warp_sum(v);
+  if ((threadIdx.x & 31) == 0) part[threadIdx.x >> 5] = v;
+  __syncthreads();
+  float tot = 0.f;
+#pragma unroll
+  for (int w = 0; w < NORM_THREADS / 32; ++w) tot += part[w];
+  return tot;
+}
+// Plain RMSNorm of rows of any width and alignment, one value per access.
+template <typename T>
+__global__ void __launch_bounds__(NORM_THREADS) rmsnorm_scalar_kernel(const T* x, const T* w, T* out, int D, int64_t sx,
+                                                                      int64_t so, float eps) {
+  x += blockIdx.x * sx;
+  out += blockIdx.x * so;
+  float ss = 0.f;
+  for (int c = threadIdx.x; c < D; c += NORM_THREADS) { const float z = to_float<T>(x[c]); ss = fmaf(z, z, ss); }
+  const float rstd = rsqrtf(block_sum(ss) / (float)D + eps);
+  for (int c = threadIdx.x; c < D; c += NORM_THREADS) out[c] = from_float<T>(to_float<T>(x[c]) * rstd * to_float<T>(w[c]));
+}
+
+// ---- parallel block: residual stream update and one or two norms of the result
+struct StreamParams {
+  const int64_t* tokens;                  // [M] with table [V, D] and table_norm [D]: the row is norm(table[token])
+  const void *table, *table_norm, *branch;
+  float* residual;                        // [M, D] fp32, read (unless tokens) and written in place
+  const void *w1, *w2;                    // [D] each; w2 / out2 may be null
+  void *out1, *out2;
+  int64_t M, V, sb;                       // sb: row stride of branch; residual and outputs are contiguous
+  int D;
+  float mult, eps;
+};
+
+// One row per block; N values per access (8, or 1 for any D), VPT accesses per thread kept in registers.
+template <typename T, int N, int VPT>
+__global__ void __launch_bounds__(NORM_THREADS) stream_norm_kernel(const StreamParams p) {
+  using seq::Pack;
+  const int64_t row = blockIdx.x;
+  const int groups = p.D / N;
+  float* res = p.residual + row * p.D;
+  float z[VPT][N];
+  auto load_res = [&](int g, float (&v)[N]) {
+    if constexpr (N == 8) load8(res, 0, 8 * g, v);
+    else v[0] = res[g];
+  };
+  auto store_res = [&](int g, const float (&v)[N]) {
+    if constexpr (N == 8) store8(res, 0, 8 * g, v);
+    else res[g] = v[0];
+  };
+  const int64_t tok = p.tokens ? p.tokens[row] : 0;
+  const bool known = tok >= 0 && tok < p.V;   // an id outside the table reads as a zero row
+  const T* src = p.tokens ? static_cast<const T*>(p.table) + (known ? tok : 0) * p.D
+                          : static_cast<const T*>(p.branch) + row * p.sb;
+  float ss = 0.f;
+#pragma unroll
+  for (int v = 0; v < VPT; ++v) {
+    const int g = threadIdx.x + v * NORM_THREADS;
+    if (g < groups) {
+      float b[N];
+      if (p.tokens || p.branch) Pack<T, N>::load(src + (int64_t)g * N, b);
+      if (!p.tokens) load_res(g, z[v]);
+#pragma unroll
+      for (int i = 0; i < N; ++i) {
+        if (p.tokens) z[v][i] = known ? b[i] : 0.f;
+        else if (p.branch) z[v][i] = fmaf(p.mult, b[i], z[v][i]);
+        ss = fmaf(z[v][i], z[v][i], ss);
+      }
+      if (!p.tokens && p.branch) store_res(g, z[v]);
+    }
+  }
+  float tot = block_sum(ss);
+  if (p.tokens) {
+    const float rstd = rsqrtf(tot / (float)p.D + p.eps);
+    ss = 0.f;
+#pragma unroll
+    for (int v = 0; v < VPT; ++v) {
+      const int g = threadIdx.x + v * NORM_THREADS;
+      if (g < groups) {
+        float w[N];
+        Pack<T, N>::load(static_cast<const T*>(p.table_norm) + (int64_t)g * N, w);
+#pragma unroll
+        for (int i = 0; i < N; ++i) {
+          z[v][i] *= rstd * w[i];
+          ss = fmaf(z[v][i], z[v][i], ss);
+        }
+        store_res(g, z[v]);
+      }
+    }
+    tot = block_sum(ss);
+  }
+  const float rstd = rsqrtf(tot / (float)p.D + p.eps);
+#pragma unroll
+  for (int v = 0; v < VPT; ++v) {
+    const int g = threadIdx.x + v * NORM_THREADS;
+    if (g < groups) {
+      float w[N], o[N];
+      Pack<T, N>::load(static_cast<const T*>(p.w1) + (int64_t)g * N, w);
+#pragma unroll
+      for (int i = 0; i < N; ++i) o[i] = z[v][i] * rstd * w[i];
+      Pack<T, N>::store(static_cast<T*>(p.out1) + row * p.D + (int64_t)g * N, o);
+      if (p.out2) {
+        Pack<T, N>::load(static_cast<const T*>(p.w2) + (int64_t)g * N, w);
+#pragma unroll
+        for (int i = 0; i < N; ++i) o[i] = z[v][i] * rstd * w[i];
+        Pack<T, N>::store(static_cast<T*>(p.out2) + row * p.D + (int64_t)g * N, o);
+      }
+    }
+  }
+}
+
 struct ActParams {
   const void *y, *gate;
   void* out;
@@ -194,7 +311,46 @@ __global__ void __launch_bounds__(NORM_THREADS) gated_act_kernel(const ActParams
   }
 }
 
+template <typename T>
+__global__ void __launch_bounds__(NORM_THREADS) gated_act_scalar_kernel(const ActParams p) {
+  const int64_t row = blockIdx.x;
+  for (int c = threadIdx.x; c < p.F; c += NORM_THREADS) {
+    const float g = to_float<T>(static_cast<const T*>(p.gate)[row * p.sg + c]);
+    static_cast<T*>(p.out)[row * p.so + c] =
+        from_float<T>(to_float<T>(static_cast<const T*>(p.y)[row * p.sy + c]) * act_fn(g, p.act));
+  }
+}
+
+template <typename T>
+int launch_stream_norm_t(const StreamParams& p, cudaStream_t stream) {
+  const unsigned grid = (unsigned)p.M;
+  const bool vec = p.D % 8 == 0 && aligned16(p.table) && aligned16(p.table_norm) && aligned16(p.branch) &&
+                   aligned16(p.residual) && aligned16(p.w1) && aligned16(p.w2) && aligned16(p.out1) &&
+                   aligned16(p.out2) && p.sb % 8 == 0;
+  const int vpt = (p.D / (vec ? 8 : 1) + NORM_THREADS - 1) / NORM_THREADS;
+  if (vec) {
+    if (vpt <= 1) stream_norm_kernel<T, 8, 1><<<grid, NORM_THREADS, 0, stream>>>(p);
+    else if (vpt <= 2) stream_norm_kernel<T, 8, 2><<<grid, NORM_THREADS, 0, stream>>>(p);
+    else if (vpt <= 4) stream_norm_kernel<T, 8, 4><<<grid, NORM_THREADS, 0, stream>>>(p);
+    else if (vpt <= 8) stream_norm_kernel<T, 8, 8><<<grid, NORM_THREADS, 0, stream>>>(p);
+    else return BASED_ERR_SHAPE;   // rows up to 8192 wide
+  } else {
+    if (vpt <= 4) stream_norm_kernel<T, 1, 4><<<grid, NORM_THREADS, 0, stream>>>(p);
+    else if (vpt <= 32) stream_norm_kernel<T, 1, 32><<<grid, NORM_THREADS, 0, stream>>>(p);
+    else return BASED_ERR_SHAPE;   // rows up to 4096 wide
+  }
+  return (int)cudaGetLastError();
+}
+
 }  // namespace
+
+int launch_stream_norm(const int64_t* tokens, const void* table, const void* table_norm, int64_t V, const void* branch,
+                       int64_t branch_stride, float mult, float* residual, const void* w1, const void* w2, void* out1,
+                       void* out2, int64_t M, int D, float eps, int io_dtype, cudaStream_t stream) {
+  if (M > 2147483647LL) return BASED_ERR_TOO_LARGE;
+  const StreamParams p{tokens, table, table_norm, branch, residual, w1, w2, out1, out2, M, V, branch_stride, D, mult, eps};
+  return io_dtype == BASED_BF16 ? launch_stream_norm_t<__nv_bfloat16>(p, stream) : launch_stream_norm_t<float>(p, stream);
+}
 
 int launch_add_rmsnorm(const void* x, const void* residual, const void* weight, const void* bias, void* out,
                        void* residual_out, int64_t M, int D, int64_t sx, int64_t sr, int64_t so, int64_t sro, float eps,
@@ -216,16 +372,33 @@ int launch_add_rmsnorm(const void* x, const void* residual, const void* weight, 
   return (int)cudaGetLastError();
 }
 
+int launch_rmsnorm(const void* x, const void* w, void* out, int64_t M, int D, int64_t sx, int64_t so, float eps,
+                   int io_dtype, cudaStream_t stream) {
+  const int rc = launch_add_rmsnorm(x, nullptr, w, nullptr, out, nullptr, M, D, sx, 0, so, 0, eps, io_dtype, io_dtype,
+                                    io_dtype, 0, stream);
+  if (rc != BASED_ERR_SHAPE && rc != BASED_ERR_ALIGN) return rc;
+  if (io_dtype == BASED_BF16)
+    rmsnorm_scalar_kernel<__nv_bfloat16><<<(unsigned)M, NORM_THREADS, 0, stream>>>(
+        static_cast<const __nv_bfloat16*>(x), static_cast<const __nv_bfloat16*>(w), static_cast<__nv_bfloat16*>(out), D, sx,
+        so, eps);
+  else
+    rmsnorm_scalar_kernel<float><<<(unsigned)M, NORM_THREADS, 0, stream>>>(
+        static_cast<const float*>(x), static_cast<const float*>(w), static_cast<float*>(out), D, sx, so, eps);
+  return (int)cudaGetLastError();
+}
+
 int launch_gated_act(const void* y, const void* gate, void* out, int64_t M, int F, int64_t sy, int64_t sg, int64_t so,
                      int act, int io_dtype, cudaStream_t stream) {
   const int N = io_dtype == BASED_BF16 ? 8 : 4;
-  if (F % N != 0) return BASED_ERR_SHAPE;
-  if (!aligned16(y) || !aligned16(gate) || !aligned16(out) || sy % N || sg % N || so % N) return BASED_ERR_ALIGN;
   if (M > 2147483647LL) return BASED_ERR_TOO_LARGE;
   const int nvec = F / N, vpt = (nvec + NORM_THREADS - 1) / NORM_THREADS;
-  if (vpt > 16) return BASED_ERR_SHAPE;  // F up to 16384 (bf16) / 8192 (fp32)
   ActParams p{y, gate, out, M, sy, sg, so, F, act};
   const unsigned grid = (unsigned)M;
+  if (F % N != 0 || vpt > 16 || !aligned16(y) || !aligned16(gate) || !aligned16(out) || sy % N || sg % N || so % N) {
+    if (io_dtype == BASED_BF16) gated_act_scalar_kernel<__nv_bfloat16><<<grid, NORM_THREADS, 0, stream>>>(p);
+    else gated_act_scalar_kernel<float><<<grid, NORM_THREADS, 0, stream>>>(p);
+    return (int)cudaGetLastError();
+  }
 #define BASED_LAUNCH_ACT(T)                                                                      \
   do {                                                                                           \
     if (vpt <= 1) gated_act_kernel<T, 1><<<grid, NORM_THREADS, 0, stream>>>(p);                  \

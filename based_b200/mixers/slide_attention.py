@@ -16,7 +16,8 @@ from ..sharding import all_reduce_sum_, head_slice, row_parallel_decode_linear
 
 class RotaryEmbedding(nn.Module):
     """cos/sin tables as the reference's rotary module builds them (fp32 ``outer(t, inv_freq)``,
-    ``inv_freq = base**(-arange(0, dim, 2)/dim)``, cast to the model dtype)."""
+    ``inv_freq = base**(-arange(0, dim, 2)/dim)``, cast to the model dtype).  :meth:`tables_f32` gives tables in
+    float32 from float64 angles, for mixers that rotate in 32-bit."""
 
     def __init__(self, dim: int, base=10000.0, interleaved=False, scale_base=None, device=None):
         super().__init__()
@@ -36,6 +37,15 @@ class RotaryEmbedding(nn.Module):
             freqs = torch.outer(t, inv_freq)
             self._cos_cached = torch.cos(freqs).to(dtype).contiguous()
             self._sin_cached = torch.sin(freqs).to(dtype).contiguous()
+
+    def tables_f32(self, seqlen, device):
+        if self._cos_cached is None or self._cos_cached.shape[0] < seqlen or self._cos_cached.device != torch.device(device):
+            inv_freq = self.base ** (-torch.arange(0, self.dim, 2, dtype=torch.float64) / self.dim)
+            ang = torch.outer(torch.arange(seqlen, dtype=torch.float64), inv_freq)
+            self._seq_len_cached = seqlen
+            self._cos_cached = torch.cos(ang).float().to(device).contiguous()
+            self._sin_cached = torch.sin(ang).float().to(device).contiguous()
+        return self._cos_cached, self._sin_cached
 
     def forward(self, qkv: torch.Tensor, seqlen_offset=0, max_seqlen=None):
         """In-place RoPE on q and k of packed ``qkv [B, L, 3, H, hd]`` (slide_attention.py:553-556)."""

@@ -10,7 +10,7 @@ block of block.py:134-163 with an fp32 residual stream, layer selection by index
 steps split of based/generation.py:93-204, and optional CUDA-graph replay of the decode step
 (:689-739).  Training, dropout, tensor-parallel embeddings and sampling strategies are not.
 """
-from dataclasses import dataclass, field
+from dataclasses import dataclass, field, fields
 from typing import List, Optional
 
 import torch
@@ -18,33 +18,9 @@ import torch.nn as nn
 import torch.nn.functional as F
 
 from . import ops
-from .generation import InferenceParams
+from .generation import GenerationMixin, sample_token  # noqa: F401
 from .mixers import BaseConv, LinearAttention, SlidingAttention, TaylorExp
 from .modules import GatedMlp, RMSNorm
-
-
-def sample_token(logits: torch.Tensor, top_k: int = 1, top_p: float = 0.0, temperature: float = 1.0) -> torch.Tensor:
-    """Next token per row of ``logits [B, V]``: greedy for ``top_k == 1``; otherwise restrict to the ``top_k`` largest
-    logits (all of them for ``top_k <= 0``), divide by ``temperature``, drop the low-probability tail whose
-    cumulative probability is at most ``1 - top_p`` (nucleus sampling; no-op for ``top_p`` outside (0, 1)), and draw
-    from the softmax of what is left.  Same policy as ``sample`` in based/generation.py:38-92."""
-    if top_k == 1:
-        return logits.argmax(dim=-1)
-    if not 0.0 <= top_p <= 1.0:
-        raise ValueError("top_p must be in [0, 1]")
-    if top_k > 0:
-        vals, idx = torch.topk(logits, min(top_k, logits.size(-1)), dim=-1)       # descending
-    else:
-        vals, idx = torch.sort(logits, dim=-1, descending=True)
-    vals = vals.float()
-    if temperature != 1.0:
-        vals = vals / temperature
-    if 0.0 < top_p < 1.0:
-        probs = vals.softmax(dim=-1)
-        tail = probs.flip(-1).cumsum(dim=-1).flip(-1)     # mass of this candidate and everything less likely
-        vals = vals.masked_fill(tail <= 1.0 - top_p, float("-inf"))
-    choice = torch.multinomial(vals.softmax(dim=-1), num_samples=1)
-    return idx.gather(-1, choice).squeeze(-1)
 
 
 @dataclass
@@ -72,6 +48,11 @@ class BasedConfig:
     def padded_vocab_size(self):
         m = self.pad_vocab_size_multiple
         return (self.vocab_size + m - 1) // m * m
+
+    @classmethod
+    def from_dict(cls, d):
+        """From the keys of a config file; keys that are not fields of this class are ignored."""
+        return cls(**{f.name: d[f.name] for f in fields(cls) if f.name in d})
 
     @classmethod
     def based_360m(cls):
@@ -152,12 +133,27 @@ class BasedModel(nn.Module):
                          round_input=True)
 
 
-class BasedLMHeadModel(nn.Module):
+class BasedLMHeadModel(GenerationMixin, nn.Module):
     def __init__(self, config: BasedConfig, device=None, dtype=None):
         super().__init__()
         self.config = config
         self.transformer = BasedModel(config, device=device, dtype=dtype)
         self.lm_head = nn.Linear(config.n_embd, config.padded_vocab_size, bias=False, device=device, dtype=dtype)
+        self.tie_weights()
+
+    @classmethod
+    def from_config(cls, d, device=None, dtype=None):
+        return cls(BasedConfig.from_dict(d), device=device, dtype=dtype)
+
+    def load_tensors(self, tensors):
+        """Weights by the reference's parameter names (``tensors`` as :class:`based_b200.weights.SafeTensors`)."""
+        own = {k: v for k, v in self.state_dict().items() if k != "lm_head.weight"}
+        missing = [k for k in own if k not in tensors]
+        if missing:
+            raise KeyError(f"missing tensors: {missing[:5]}")
+        with torch.no_grad():
+            for k, v in own.items():
+                v.copy_(tensors.get(k, tuple(v.shape)))
         self.tie_weights()
 
     def tie_weights(self):
@@ -172,81 +168,3 @@ class BasedLMHeadModel(nn.Module):
         if num_last_tokens > 0:
             hidden_states = hidden_states[:, -num_last_tokens:]
         return ops.linear(hidden_states, self.lm_head.weight, self.lm_head.bias)
-
-    @torch.inference_mode()
-    def generate(self, input_ids, max_new_tokens: int, cg: bool = False, timings: Optional[dict] = None,
-                 top_k: int = 1, top_p: float = 0.0, temperature: float = 1.0):
-        """Decoding: one prompt pass, then one token per step (generation.py:93-204); greedy by default, top-k /
-        nucleus / temperature sampling as :func:`sample_token` otherwise.  With ``cg`` the decode step is
-        captured once in a CUDA graph and replayed (:689-739).  Returns ``[B, L + max_new_tokens]``.
-        ``timings``, when given, receives device times in ms: ``prefill_ms``, ``decode_ms`` (all steps)."""
-        B, L = input_ids.shape
-        dtype = self.lm_head.weight.dtype
-        ip = InferenceParams(max_seqlen=L + max_new_tokens, max_batch_size=B)
-        ip.key_value_memory_dict = self.allocate_inference_cache(B, ip.max_seqlen, dtype=dtype)
-        ip.lengths_per_sample = torch.full((B,), L, dtype=torch.int32, device=input_ids.device)
-        ev = [torch.cuda.Event(enable_timing=True) for _ in range(3)]
-        out = torch.empty(B, L + max_new_tokens, dtype=input_ids.dtype, device=input_ids.device)
-        out[:, :L] = input_ids
-        ev[0].record()
-        logits = self.forward(input_ids, inference_params=ip, num_last_tokens=1)
-        token = sample_token(logits[:, -1, : self.config.vocab_size], top_k, top_p, temperature).unsqueeze(-1)
-        ev[1].record()
-        ip.seqlen_offset = L
-        if max_new_tokens > 0:
-            out[:, L] = token[:, 0]
-        cur = token.clone()
-
-        def step():
-            lg = self.forward(cur, inference_params=ip, num_last_tokens=1)
-            cur.copy_(sample_token(lg[:, -1, : self.config.vocab_size], top_k, top_p, temperature).unsqueeze(-1))
-            ip.lengths_per_sample.add_(1)
-
-        graph = None
-        steps_left = max_new_tokens - 1
-        if cg and steps_left > 2:
-            # warm-up on a side stream (the first calls may build rotary tables), then capture one step
-            s = torch.cuda.Stream()
-            s.wait_stream(torch.cuda.current_stream())
-            saved = self._snapshot_state(ip, cur)
-            with torch.cuda.stream(s):
-                for _ in range(2):
-                    step()
-            torch.cuda.current_stream().wait_stream(s)
-            self._restore_state(ip, cur, saved)
-            graph = torch.cuda.CUDAGraph()
-            with torch.cuda.graph(graph):
-                step()
-            self._restore_state(ip, cur, saved)
-        for i in range(steps_left):
-            if graph is not None:
-                graph.replay()
-            else:
-                step()
-            ip.seqlen_offset += 1
-            out[:, L + 1 + i] = cur[:, 0]
-        ev[2].record()
-        if timings is not None:
-            torch.cuda.synchronize()
-            ops.check_status()   # the device is idle here: a tensor-core kernel that gave up on a wait shows now
-            timings["prefill_ms"] = ev[0].elapsed_time(ev[1])
-            timings["decode_ms"] = ev[1].elapsed_time(ev[2])
-        return out
-
-    @staticmethod
-    def _flat_state(ip):
-        for v in ip.key_value_memory_dict.values():
-            if isinstance(v, dict):
-                yield from v.values()
-            elif isinstance(v, (tuple, list)):
-                yield from v
-            else:
-                yield v
-
-    def _snapshot_state(self, ip, cur):
-        return [t.clone() for t in self._flat_state(ip)] + [ip.lengths_per_sample.clone(), cur.clone()]
-
-    def _restore_state(self, ip, cur, saved):
-        tensors = list(self._flat_state(ip)) + [ip.lengths_per_sample, cur]
-        for t, s in zip(tensors, saved):
-            t.copy_(s)

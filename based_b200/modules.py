@@ -49,7 +49,8 @@ class GatedMlp(nn.Module):
         self.activation = activation
         self.fc2 = nn.Linear(hidden_features, out_features, bias=bias2, **fk)
 
-    def forward(self, x):
+    def hidden(self, x, out=None):
+        """fc1 and the gated activation; ``out``: a ``[..., hidden]`` tensor or column slice to write."""
         if self.activation in (F.sigmoid, torch.sigmoid):
             act = "sigmoid"
         elif self.activation is F.silu:
@@ -57,9 +58,10 @@ class GatedMlp(nn.Module):
         else:
             raise NotImplementedError("GatedMlp: activation must be F.silu (SwiGLU) or F.sigmoid (GLU)")
         if ops.DECODE_LINEAR_USE["gated"] and ops._decode_rows(x, self.fc1.weight) and self.fc1.weight.shape[0] % 16 == 0:
-            # decode step: fc1 and the gated activation in one launch, fc2 in another
-            y = ops.decode_linear(x, self.fc1.weight, self.fc1.bias, epilogue="gated", activation=act)
-        else:
-            y = ops.gated_act(self.fc1(x), act)
-        y = ops.linear(y, self.fc2.weight, self.fc2.bias)
+            # decode step: fc1 and the gated activation in one launch
+            return ops.decode_linear(x, self.fc1.weight, self.fc1.bias, epilogue="gated", activation=act, out=out)
+        return ops.gated_act(self.fc1(x), act, out=out)
+
+    def forward(self, x):
+        y = ops.linear(self.hidden(x), self.fc2.weight, self.fc2.bias)
         return y if not self.return_residual else (y, x)

@@ -54,6 +54,40 @@ def _inner_contig(t, name):
         raise ValueError(f"{name}: innermost stride must be 1")
 
 
+def _rows(t, width):
+    """``t [..., width]`` as a ``[M, width]`` view of the same memory (rows one constant stride apart)."""
+    if t.shape[-1] != width or t.stride(-1) != 1:
+        raise ValueError(f"out must be a [..., {width}] tensor with contiguous rows")
+    return flat_rows(t)
+
+
+def flat_rows(t):
+    """``t [..., W]`` as ``[M, W]`` without a copy; raises when its rows are not one constant stride apart."""
+    dims = [(n, st) for n, st in zip(t.shape[:-1], t.stride()[:-1]) if n != 1]
+    for (_, outer), (n, inner) in zip(dims, dims[1:]):
+        if outer != inner * n:
+            raise ValueError("rows are not one constant stride apart")
+    m = 1
+    for n, _ in dims:
+        m *= n
+    return t.as_strided((m, t.shape[-1]), (dims[-1][1] if dims else t.shape[-1], t.stride(-1)))
+
+
+def _position(pos, like):
+    """(device pointer or None, scalar) of a call's first position: an int, or an int32 CUDA tensor with one per row."""
+    if torch.is_tensor(pos):
+        if pos.dtype != torch.int32 or pos.device != like.device or not pos.is_contiguous():
+            raise TypeError("positions must be a contiguous int32 tensor on the inputs' device")
+        if pos.numel() < like.shape[0]:
+            raise ValueError("positions: one per batch row is needed")
+        return pos.data_ptr(), 0
+    return None, int(pos)
+
+
+def _ptr(t):
+    return None if t is None else t.data_ptr()
+
+
 def _stream():
     return torch.cuda.current_stream().cuda_stream
 
@@ -389,15 +423,16 @@ def add_rmsnorm(x: torch.Tensor, weight: torch.Tensor, bias: Optional[torch.Tens
 _ACTS = {"silu": 0, "swiglu": 0, "sigmoid": 1, "glu": 1}
 
 
-def gated_act(y: torch.Tensor, activation: str = "silu") -> torch.Tensor:
-    """``first_half * act(second_half)`` over the last dim of ``y [..., 2F]`` (mlp.py:141-154)."""
-    _need_cuda(y)
+def gated_act(y: torch.Tensor, activation: str = "silu", out: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """``first_half * act(second_half)`` over the last dim of ``y [..., 2F]`` (mlp.py:141-154).  ``out``: a ``[..., F]``
+    tensor or column slice to write (rows one constant stride apart)."""
+    _need_cuda(y, out)
     F2 = y.shape[-1]
     F = F2 // 2
     y2 = y.reshape(-1, F2)
     _inner_contig(y2, "y")
     M = y2.shape[0]
-    out = torch.empty(M, F, dtype=y.dtype, device=y.device)
+    out = torch.empty(M, F, dtype=y.dtype, device=y.device) if out is None else _rows(out, F)
     if M > 0:
         a, g = y2[:, :F], y2[:, F:]
         with torch.cuda.device(y.device):
@@ -416,7 +451,8 @@ DECODE_LINEAR_USE = {"plain": False, "gated": True, "conv": False}
 
 def decode_linear(x: torch.Tensor, weight: torch.Tensor, bias: Optional[torch.Tensor] = None, *,
                   epilogue: str = "plain", activation: str = "silu", conv_state: Optional[torch.Tensor] = None,
-                  conv_weight: Optional[torch.Tensor] = None, conv_bias: Optional[torch.Tensor] = None) -> torch.Tensor:
+                  conv_weight: Optional[torch.Tensor] = None, conv_bias: Optional[torch.Tensor] = None,
+                  out: Optional[torch.Tensor] = None) -> torch.Tensor:
     """``x W^T (+ bias)`` for the few rows of a decode step (bf16), with a fused epilogue:
     ``"plain"``; ``"gated"`` -> ``first_half * act(second_half)`` (mlp.py:146-154); ``"conv"`` -> the BaseConv
     decode step on the first half (``conv_state [M, N/2, k]`` updated in place), silu, gate by the second half
@@ -432,7 +468,7 @@ def decode_linear(x: torch.Tensor, weight: torch.Tensor, bias: Optional[torch.Te
         raise ValueError("weight must be a contiguous [N, K] tensor")
     epi = {"plain": 0, "gated": 1, "conv": 2}[epilogue]
     n_out = N if epi == 0 else N // 2
-    out = torch.empty(M, n_out, dtype=torch.bfloat16, device=x.device)
+    out = torch.empty(M, n_out, dtype=torch.bfloat16, device=x.device) if out is None else _rows(out, n_out)
     if bias is not None:
         bias = bias.to(torch.bfloat16).contiguous()
     ck, cw_dt = 0, BASED_BF16
@@ -564,3 +600,244 @@ def tp_outproj_allreduce_emulated(xs, weights, bias, workspaces, max_rows: int):
             _stream())
     _capi.check(code, "based_tp_outproj_allreduce_emulated")
     return outs
+
+
+# --------------------------------------------------------------------------- stateful mixers of hybrid stacks
+# ``pos``: position of a call's first token, an int or an int32 CUDA tensor with one entry per batch row.  A sequence
+# that starts (position 0) reads no state, so state tensors need no clearing between sequences.
+
+def linear_f32(x: torch.Tensor, weight: torch.Tensor) -> torch.Tensor:
+    """``x W^T`` with an fp32 result (fp32 accumulation of the operands' products, not rounded to their dtype)."""
+    _need_cuda(x, weight)
+    if x.dtype == torch.float32:
+        return torch.nn.functional.linear(x, weight)
+    y = torch.mm(x.reshape(-1, x.shape[-1]), weight.t(), out_dtype=torch.float32)
+    return y.view(*x.shape[:-1], weight.shape[0])
+
+
+def stream_norm(residual: torch.Tensor, w1: torch.Tensor, w2: Optional[torch.Tensor] = None, *,
+                branch: Optional[torch.Tensor] = None, mult: float = 1.0, tokens: Optional[torch.Tensor] = None,
+                table: Optional[torch.Tensor] = None, table_norm: Optional[torch.Tensor] = None, eps: float = 1e-6):
+    """The norm step of a parallel block: the fp32 stream ``residual [..., D]`` becomes ``residual + mult * branch`` (or,
+    with ``tokens``, ``rmsnorm(table[token]) * table_norm``) IN PLACE; returns its RMSNorm scaled by ``w1`` and by ``w2``
+    (None without ``w2``), in the weights' dtype."""
+    _need_cuda(residual, w1, w2, branch, tokens, table, table_norm)
+    D = residual.shape[-1]
+    if residual.dtype != torch.float32 or not residual.is_contiguous():
+        raise TypeError("residual must be a contiguous float32 tensor")
+    M = residual.numel() // D if D else 0
+    out1 = torch.empty(residual.shape, dtype=w1.dtype, device=residual.device)
+    out2 = torch.empty_like(out1) if w2 is not None else None
+    sb = 0
+    if branch is not None:
+        branch = branch.reshape(-1, D)
+        _inner_contig(branch, "branch")
+        sb = branch.stride(0)
+    V = 0
+    if tokens is not None:
+        if tokens.dtype != torch.int64 or tokens.numel() != M:
+            raise TypeError("tokens must be int64, one per row")
+        tokens, V = tokens.contiguous(), table.shape[0]
+    for t in (w1, w2, branch, table, table_norm):
+        if t is not None and (t.dtype != w1.dtype or (t is not branch and not t.is_contiguous())):
+            raise TypeError("weights, table and branch must share a dtype and be contiguous")
+    if M > 0:
+        with torch.cuda.device(residual.device):
+            code = _capi.lib().based_stream_norm(
+                _ptr(tokens), _ptr(table), _ptr(table_norm), V, _ptr(branch), sb, float(mult), residual.data_ptr(),
+                w1.data_ptr(), _ptr(w2), out1.data_ptr(), _ptr(out2), M, D, float(eps), _dt(w1.dtype), _stream())
+        _capi.check(code, "based_stream_norm")
+    return out1, out2
+
+
+def rmsnorm(x: torch.Tensor, weight: torch.Tensor, eps: float) -> torch.Tensor:
+    """``x / sqrt(mean(x^2) + eps) * weight`` over the last dim of ``x [..., D]`` (a column slice is fine), contiguous."""
+    _need_cuda(x, weight)
+    D = x.shape[-1]
+    x2 = flat_rows(x) if x.dim() > 1 else x.view(1, D)
+    _inner_contig(x2, "x")
+    out = torch.empty(x.shape, dtype=x.dtype, device=x.device)
+    if weight.dtype != x.dtype:
+        raise TypeError("weight must be in x's dtype")
+    if out.numel() > 0:
+        with torch.cuda.device(x.device):
+            code = _capi.lib().based_rmsnorm(x2.data_ptr(), weight.data_ptr(), out.data_ptr(), x2.shape[0], D, x2.stride(0), D,
+                                             float(eps), _dt(x.dtype), _stream())
+        _capi.check(code, "based_rmsnorm")
+    return out
+
+
+def short_conv(x: torch.Tensor, weight: torch.Tensor, bias: Optional[torch.Tensor] = None, *,
+               ring: Optional[torch.Tensor] = None, pos=0, silu: bool = False) -> torch.Tensor:
+    """Depthwise causal convolution ``x [B, L, C]`` by ``weight [C, taps]`` for tokens that start at ``pos``; ``ring
+    [B, taps, C]`` carries earlier inputs (position p in slot p mod taps) and is updated.  Contiguous ``[B, L, C]``."""
+    _need_cuda(x, weight, bias, ring)
+    B, L, C = x.shape
+    taps = weight.shape[1]
+    _inner_contig(x, "x")
+    if weight.shape[0] != C or weight.dtype != x.dtype or not weight.is_contiguous() or (bias is not None and bias.dtype != x.dtype):
+        raise ValueError("weight must be a contiguous [C, taps] tensor in x's dtype (bias [C] too)")
+    if ring is not None and (ring.shape[0] < B or ring.shape[1:] != (taps, C) or ring.dtype != x.dtype or not ring.is_contiguous()):
+        raise ValueError("ring must be a contiguous [>= B, taps, C] tensor in x's dtype")
+    y = torch.empty(B, L, C, dtype=x.dtype, device=x.device)
+    if y.numel() == 0:
+        return y
+    off, scalar = _position(pos, x)
+    with torch.cuda.device(x.device):
+        code = _capi.lib().based_short_conv(x.data_ptr(), y.data_ptr(), _ptr(ring), weight.data_ptr(), _ptr(bias), B, L, C, taps,
+                                            _capi.strides(*x.stride()[:2]), _capi.strides(*y.stride()[:2]), off, scalar,
+                                            int(silu), _dt(x.dtype), _stream())
+    _capi.check(code, "based_short_conv")
+    return y
+
+
+def latent_prepare_(q: torch.Tensor, cos: torch.Tensor, sin: torch.Tensor, dim: int, *, z: Optional[torch.Tensor] = None,
+                    norm_weight: Optional[torch.Tensor] = None, cache: Optional[torch.Tensor] = None, kv_rank: int = 1,
+                    pos=0, eps: float = 1e-6) -> torch.Tensor:
+    """Rotate the last dims of every head of ``q [B, L, H, dim + rot]`` IN PLACE and, with ``z [B, L, kv_rank + rot]``,
+    append the normed latent and the rotated shared key to ``cache [B, max_len, kv_rank + rot]``.  fp32 tables."""
+    _need_cuda(q, cos, sin, z, norm_weight, cache)
+    B, L, H, dq = q.shape
+    rd = dq - dim
+    if not q.is_contiguous() or cos.dtype != torch.float32 or cos.shape[1] * 2 != rd or not (cos.is_contiguous() and sin.is_contiguous()):
+        raise ValueError("q must be contiguous and the tables float32 [positions, rot / 2]")
+    zs = cs = None
+    max_len = 2147483647
+    if z is not None:
+        _inner_contig(z, "z")
+        if z.dtype != q.dtype or cache.dtype != q.dtype or cache.shape[0] < B or cache.shape[2] != kv_rank + rd or cache.stride(2) != 1:
+            raise ValueError("cache must be [>= B, max_len, kv_rank + rot] in the inputs' dtype")
+        zs, cs, max_len = _capi.strides(*z.stride()[:2]), _capi.strides(*cache.stride()[:2]), cache.shape[1]
+    if q.numel() == 0:
+        return q
+    off, scalar = _position(pos, q)
+    with torch.cuda.device(q.device):
+        code = _capi.lib().based_latent_prepare(_ptr(z), _ptr(norm_weight), _ptr(cache), q.data_ptr(), cos.data_ptr(), sin.data_ptr(),
+                                                cos.shape[0], B, L, H, int(kv_rank), rd, int(dim), max_len, zs, cs,
+                                                _capi.strides(*q.stride()[:2]), off, scalar, float(eps), _dt(q.dtype), _stream())
+    _capi.check(code, "based_latent_prepare")
+    return q
+
+
+def split_key_attention(q1, q2, k1, k2, v, scale: float, *, gate: Optional[torch.Tensor] = None, pos=0,
+                        out: torch.Tensor) -> torch.Tensor:
+    """Causal attention with score ``(q1 . k1 + q2 . k2) * scale`` on CUDA cores (fp32 arithmetic): q1, q2 ``[B, L, H, .]``,
+    k1, k2, v ``[B, T, H, .]`` (expand the head dim to share keys), ``gate [B, L, H]`` pre-sigmoid, ``out [B, L, H, dv]``."""
+    _need_cuda(q1, q2, k1, k2, v, gate, out)
+    B, L, H, d1 = q1.shape
+    for t, n in ((q1, "q1"), (q2, "q2"), (k1, "k1"), (k2, "k2"), (v, "v"), (out, "out")):
+        _inner_contig(t, n)
+        if t.dtype != q1.dtype:
+            raise TypeError("all tensors must share a dtype")
+    off, scalar = _position(pos, q1)
+    if off is None and k1.shape[1] < scalar + L:
+        raise ValueError("fewer keys than the last query sees")
+    gs = _capi.strides(*gate.stride()[:2]) if gate is not None else None
+    if gate is not None:
+        _inner_contig(gate, "gate")
+    if out.numel() == 0:
+        return out
+    with torch.cuda.device(q1.device):
+        code = _capi.lib().based_split_key_attention(
+            q1.data_ptr(), q2.data_ptr(), k1.data_ptr(), k2.data_ptr(), v.data_ptr(), _ptr(gate), out.data_ptr(), B, L, H, d1,
+            q2.shape[-1], v.shape[-1], _capi.strides(*q1.stride()[:3]), _capi.strides(*q2.stride()[:3]),
+            _capi.strides(*k1.stride()[:3]), _capi.strides(*k2.stride()[:3]), _capi.strides(*v.stride()[:3]),
+            _capi.strides(*out.stride()[:3]), gs, off, scalar, float(scale), _dt(q1.dtype), _stream())
+    _capi.check(code, "based_split_key_attention")
+    return out
+
+
+def _check_delta(state, B, H, d, dv, *params):
+    if state.shape[0] < B or state.shape[1:] != (H, d, dv) or state.dtype != torch.float32 or not state.is_contiguous():
+        raise ValueError("state must be a contiguous float32 [>= B, H, d, dv] tensor")
+    for t in params:
+        if t.dtype != torch.float32 or t.stride(-1) != 1:
+            raise TypeError("decay and step-size inputs must be float32")
+
+
+def delta_prefill(q, k, v, z, a, b, A_log, dt_bias, norm_weight, state, *, pos=0, eps: float = 1e-6,
+                  out: torch.Tensor) -> torch.Tensor:
+    """Gated delta rule over ``L`` tokens: q, k ``[B, L, Hk, d]``, v, z ``[B, L, H, dv]`` (token-strided views, heads
+    contiguous), a, b ``[B, L, H]`` fp32 pre-activations, ``state [B, H, d, dv]`` fp32 updated IN PLACE; ``out [B, L, H * dv]``."""
+    _need_cuda(q, k, v, z, a, b, A_log, dt_bias, norm_weight, state, out)
+    B, L, Hk, d = q.shape
+    H, dv = v.shape[2:]
+    _check_delta(state, B, H, d, dv, a, b, A_log, dt_bias)
+    for t, w in ((q, d), (k, d), (v, dv), (z, dv)):
+        if t.stride(3) != 1 or (t.shape[2] > 1 and t.stride(2) != w) or t.dtype != q.dtype:
+            raise ValueError("q, k, v, z: heads must be contiguous inside a token and share a dtype")
+    if a.stride()[:2] != b.stride()[:2]:
+        raise ValueError("a and b must have the same strides")
+    _inner_contig(out, "out")
+    off, scalar = _position(pos, q)
+    if out.numel() == 0:
+        return out
+    with torch.cuda.device(q.device):
+        code = _capi.lib().based_delta_prefill(
+            q.data_ptr(), k.data_ptr(), v.data_ptr(), z.data_ptr(), a.data_ptr(), b.data_ptr(), A_log.data_ptr(), dt_bias.data_ptr(),
+            norm_weight.data_ptr(), state.data_ptr(), out.data_ptr(), B, L, H, Hk, d, dv, _capi.strides(*q.stride()[:2]),
+            _capi.strides(*k.stride()[:2]), _capi.strides(*v.stride()[:2]), _capi.strides(*z.stride()[:2]),
+            _capi.strides(*a.stride()[:2]), _capi.strides(*out.stride()[:2]), off, scalar, float(eps), _dt(q.dtype), _stream())
+    _capi.check(code, "based_delta_prefill")
+    return out
+
+
+def delta_step(x, conv_weight, ring, a, b, A_log, dt_bias, norm_weight, state, kv_heads: int, *, pos, eps: float = 1e-6,
+               out: torch.Tensor) -> bool:
+    """One token per row in one launch: packed projection ``x [B, q | k | v | z]``, ``ring [B, taps, C]`` and ``state
+    [B, H, d, dv]`` updated IN PLACE, ``out [B, H * dv]``.  Returns False, nothing launched, for sizes it does not take."""
+    _need_cuda(x, conv_weight, ring, a, b, A_log, dt_bias, norm_weight, state, out)
+    B, (_, H, d, dv) = x.shape[0], state.shape
+    _check_delta(state, B, H, d, dv, a, b, A_log, dt_bias)
+    C, taps = conv_weight.shape
+    if C != 2 * kv_heads * d + H * dv or x.shape[1] < C + H * dv or x.stride(1) != 1 or out.stride(1) != 1 or a.stride(0) != b.stride(0):
+        raise ValueError("x must be [B, >= 2 kv_heads d + 2 H dv] and conv_weight [2 kv_heads d + H dv, taps]")
+    if ring.shape[0] < B or ring.shape[1:] != (taps, C) or ring.dtype != x.dtype or not ring.is_contiguous() or not conv_weight.is_contiguous():
+        raise ValueError("ring must be a contiguous [>= B, taps, C] tensor in x's dtype")
+    off, scalar = _position(pos, x)
+    if B == 0:
+        return True
+    with torch.cuda.device(x.device):
+        code = _capi.lib().based_delta_step(
+            x.data_ptr(), conv_weight.data_ptr(), ring.data_ptr(), a.data_ptr(), b.data_ptr(), A_log.data_ptr(), dt_bias.data_ptr(),
+            norm_weight.data_ptr(), state.data_ptr(), out.data_ptr(), B, H, int(kv_heads), d, dv, taps, x.stride(0), a.stride(0),
+            out.stride(0), off, scalar, float(eps), _dt(x.dtype), _stream())
+    if code == _capi.ERR_IMPL:
+        return False
+    _capi.check(code, "based_delta_step")
+    return True
+
+
+def block_gates(u: torch.Tensor, weight: torch.Tensor) -> torch.Tensor:
+    """Block-diagonal product with an fp32 result: ``u [B, L, blocks * n]`` by ``weight [blocks, n, out]`` ->
+    ``[blocks, B * L, out]``."""
+    _need_cuda(u, weight)
+    nb, n, _ = weight.shape
+    x = u.reshape(-1, nb, n).transpose(0, 1)
+    if u.dtype == torch.float32:
+        return torch.bmm(x, weight)
+    return torch.bmm(x, weight, out_dtype=torch.float32)
+
+
+def rglru(u, y, gates, r_bias, i_bias, lam, state, *, pos=0, out: torch.Tensor) -> torch.Tensor:
+    """Real-gated linear recurrent unit: u, y ``[B, L, W]``, ``gates [blocks, B * L, 2 n]`` fp32 (r half, i half),
+    ``lam [W]`` fp32, ``state [B, W]`` fp32 updated IN PLACE; ``out [B, L, W] = S * gelu_tanh(y)``."""
+    _need_cuda(u, y, gates, r_bias, i_bias, lam, state, out)
+    B, L, W = u.shape
+    nb, rows, n2 = gates.shape
+    if rows != B * L or nb * n2 != 2 * W or gates.dtype != torch.float32 or gates.stride(2) != 1:
+        raise ValueError("gates must be float32 [blocks, B * L, 2 * W / blocks]")
+    if state.shape[0] < B or state.shape[1] != W or state.dtype != torch.float32 or lam.dtype != torch.float32 or not state.is_contiguous():
+        raise ValueError("state must be a contiguous float32 [>= B, W] tensor and lam float32")
+    for t, n in ((u, "u"), (y, "y"), (out, "out")):
+        _inner_contig(t, n)
+    off, scalar = _position(pos, u)
+    if out.numel() == 0:
+        return out
+    with torch.cuda.device(u.device):
+        code = _capi.lib().based_rglru(
+            u.data_ptr(), y.data_ptr(), gates.data_ptr(), r_bias.data_ptr(), i_bias.data_ptr(), lam.data_ptr(), state.data_ptr(),
+            out.data_ptr(), B, L, W, n2 // 2, _capi.strides(*u.stride()[:2]), _capi.strides(*y.stride()[:2]),
+            _capi.strides(*out.stride()[:2]), _capi.strides(gates.stride(0), gates.stride(1)), off, scalar, _dt(u.dtype), _stream())
+    _capi.check(code, "based_rglru")
+    return out

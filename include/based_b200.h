@@ -399,6 +399,95 @@ int based_tp_outproj_allreduce_emulated(const void* const* x, const void* const*
                                         int M, int N, int K, int64_t x_row_stride, int64_t out_row_stride,
                                         void* const* workspaces, int max_rows, int world, void* stream);
 
+/*
+ * ---------------------------------------------------------------------------------------------------------------
+ * Stateful mixers of hybrid stacks (gated delta rule, real-gated linear recurrent unit, latent attention) and the
+ * norm step of a parallel block.  No counterpart in the reference.
+ *
+ * A call's tokens continue their sequence at any position: the first one's position is offsets[b] (device array, one
+ * int32 per batch row) or, when offsets is NULL, the scalar `offset`.  A sequence that starts (position 0) reads
+ * neither state nor ring, so buffers need no clearing between sequences.  Norms, rotations, softmax, gates of the
+ * recurrences and the recurrent state are fp32 whatever io_dtype is; weights named here without a dtype are in
+ * io_dtype, `a`, `b`, `A_log`, `dt_bias`, `lam`, `gates`, tables, `residual` and `state` are fp32.
+ */
+
+/*
+ * z = residual + mult * branch (branch may be NULL), or, with tokens [M] (int64), z = norm(table[token]) * table_norm;
+ * z -> residual (fp32, contiguous [M, D]); out1 = norm(z) * w1, out2 = norm(z) * w2 (w2 / out2 may be NULL), contiguous.
+ */
+int based_stream_norm(const void* tokens, const void* table, const void* table_norm, int64_t V, const void* branch,
+                      int64_t branch_row_stride, float mult, void* residual, const void* w1, const void* w2, void* out1,
+                      void* out2, int64_t M, int D, float eps, int io_dtype, void* stream);
+
+/* out = x / sqrt(mean(x^2) + eps) * weight for rows of any width and alignment. */
+int based_rmsnorm(const void* x, const void* weight, void* out, int64_t M, int D, int64_t x_row_stride,
+                  int64_t out_row_stride, float eps, int io_dtype, void* stream);
+
+/*
+ * Depthwise causal convolution (weight [C, taps], last column = current token, bias [C] or NULL), optionally silu.
+ * ring [B, taps, C] holds the input of position p in slot p mod taps and is updated (NULL: no state, offset 0 only).
+ * Strides are (batch, token).
+ */
+int based_short_conv(const void* x, void* y, void* ring, const void* weight, const void* bias, int B, int L, int C,
+                     int taps, const int64_t x_strides[2], const int64_t y_strides[2], const int32_t* offsets, int offset,
+                     int silu, int io_dtype, void* stream);
+
+/*
+ * Between the projections and the attention of a latent-attention layer: z [B, L, kv_rank + rot_dim] -> RMSNorm of the
+ * latent, rotation of the shared key part, append to cache rows [.., kv_rank + rot_dim] of their positions (z NULL: the
+ * layer reads another layer's cache); rotation of the last rot_dim of every head of q [B, L, H, dim + rot_dim] in place.
+ * Tables [table_len, rot_dim / 2].  Positions past max_len or table_len are skipped (device offsets) or rejected (scalar).
+ */
+int based_latent_prepare(const void* z, const void* norm_weight, void* cache, void* q, const void* cos_table,
+                         const void* sin_table, int table_len, int B, int L, int H, int kv_rank, int rot_dim, int dim,
+                         int max_len, const int64_t z_strides[2], const int64_t cache_strides[2],
+                         const int64_t q_strides[2], const int32_t* offsets, int offset, float eps, int io_dtype,
+                         void* stream);
+
+/*
+ * Causal softmax attention with score (q1 . k1 + q2 . k2) * scale on CUDA cores, fp32 arithmetic, any sizes up to
+ * dv 1024; strides are (batch, token, head), a head stride of 0 shares keys or values between heads; the output of a
+ * head is multiplied by sigmoid(gate[b, l, h]) when gate is given.  Query l sees keys 0 .. offset + l.
+ */
+int based_split_key_attention(const void* q1, const void* q2, const void* k1, const void* k2, const void* v,
+                              const void* gate, void* out, int B, int L, int H, int d1, int d2, int dv,
+                              const int64_t q1_strides[3], const int64_t q2_strides[3], const int64_t k1_strides[3],
+                              const int64_t k2_strides[3], const int64_t v_strides[3], const int64_t out_strides[3],
+                              const int64_t gate_strides[2], const int32_t* offsets, int offset, float scale,
+                              int io_dtype, void* stream);
+
+/*
+ * Gated delta rule over the tokens of a call.  q, k [B, L, Hk, d], v, z [B, L, H, dv] (after convolution and silu;
+ * unit norms are taken here), a, b [B, L, H] pre-activations of decay and step size, state [B, H, d, dv] updated,
+ * out [B, L, H, dv] = normed read-out * norm_weight * silu(z).  Strides are (batch, token), heads contiguous.
+ */
+int based_delta_prefill(const void* q, const void* k, const void* v, const void* z, const void* a, const void* b,
+                        const void* A_log, const void* dt_bias, const void* norm_weight, void* state, void* out, int B,
+                        int L, int H, int Hk, int d, int dv, const int64_t q_strides[2], const int64_t k_strides[2],
+                        const int64_t v_strides[2], const int64_t z_strides[2], const int64_t gate_strides[2],
+                        const int64_t out_strides[2], const int32_t* offsets, int offset, float eps, int io_dtype,
+                        void* stream);
+
+/*
+ * One token per row, from the packed projection x [B, q | k | v | z] to the gated output in one launch (convolution
+ * over ring [B, taps, 2 Hk d + H dv], silu, unit norms, gates, state update, read-out, norm, gate).
+ * BASED_ERR_IMPL for sizes it does not take (dv % 4, d * dv above 32 K): use based_short_conv + based_delta_prefill.
+ */
+int based_delta_step(const void* x, const void* conv_weight, void* ring, const void* a, const void* b, const void* A_log,
+                     const void* dt_bias, const void* norm_weight, void* state, void* out, int B, int H, int Hk, int d,
+                     int dv, int taps, int64_t x_stride, int64_t gate_stride, int64_t out_stride, const int32_t* offsets,
+                     int offset, float eps, int io_dtype, void* stream);
+
+/*
+ * Real-gated linear recurrent unit over the tokens of a call: u, y [B, L, W], gates = block-diagonal products in fp32,
+ * element (block, row b L + l, j) at block * gate_strides[0] + row * gate_strides[1] + j, the r half first, the i half
+ * block_width further; state [B, W] updated; out = S * gelu_tanh(y).
+ */
+int based_rglru(const void* u, const void* y, const void* gates, const void* r_bias, const void* i_bias, const void* lam,
+                void* state, void* out, int B, int L, int W, int block_width, const int64_t u_strides[2],
+                const int64_t y_strides[2], const int64_t out_strides[2], const int64_t gate_strides[2],
+                const int32_t* offsets, int offset, int io_dtype, void* stream);
+
 #ifdef __cplusplus
 }
 #endif
