@@ -57,7 +57,13 @@ SIGNATURES = {
     "based_short_conv": (c_int, [c_void_p] * 5 + [c_int] * 4 + [_I64P] * 2 + _POS + [c_int, c_int, c_void_p]),
     "based_latent_prepare": (c_int, [c_void_p] * 6 + [c_int] * 8 + [_I64P] * 3 + _POS + [c_float, c_int, c_void_p]),
     "based_split_key_attention": (c_int, [c_void_p] * 7 + [c_int] * 6 + [_I64P] * 7 + _POS + [c_float, c_int, c_void_p]),
-    "based_delta_prefill": (c_int, [c_void_p] * 11 + [c_int] * 6 + [_I64P] * 6 + _POS + [c_float, c_int, c_void_p]),
+    "based_latent_prefill": (c_int, [c_void_p] * 7 + [c_int] * 7 + [_I64P] * 7 + [c_int, c_float, c_int, c_int, c_void_p]),
+    "based_latent_decode_scratch_bytes": (ctypes.c_size_t, [c_int] * 5),
+    "based_latent_decode": (c_int, [c_void_p] * 6 + [ctypes.c_size_t] + [c_int] * 6 + [_I64P] * 5 + _POS
+                            + [c_float, c_int, c_void_p]),
+    "based_delta_prefill_scratch_bytes": (ctypes.c_size_t, [c_int] * 5),
+    "based_delta_prefill": (c_int, [c_void_p] * 11 + [c_int] * 6 + [_I64P] * 6 + _POS
+                            + [c_float, c_int, c_int, c_void_p, ctypes.c_size_t, c_void_p]),
     "based_delta_step": (c_int, [c_void_p] * 10 + [c_int] * 6 + [c_int64] * 3 + _POS + [c_float, c_int, c_void_p]),
     "based_rglru": (c_int, [c_void_p] * 8 + [c_int] * 4 + [_I64P] * 4 + _POS + [c_int, c_void_p]),
 }

@@ -36,11 +36,13 @@ const char* based_error_string(int code) {
 }
 
 int based_read_status(unsigned int* out, int reset) {
-  unsigned int a = 0, b = 0, c = 0;
+  unsigned int a = 0, b = 0, c = 0, d = 0, e = 0;
   int rc = read_tc_status(&a, reset);
   if (rc == 0) rc = read_tc_status_swa(&b, reset);
   if (rc == 0) rc = read_tp_status(&c, reset);
-  if (out) *out = a | b | c;
+  if (rc == 0) rc = read_tc_status_latent(&d, reset);
+  if (rc == 0) rc = read_tc_status_delta(&e, reset);
+  if (out) *out = a | b | c | d | e;
   return rc;
 }
 
@@ -400,22 +402,94 @@ int based_split_key_attention(const void* q1, const void* q2, const void* k1, co
                                     offset, scale, io_dtype, static_cast<cudaStream_t>(stream));
 }
 
+int based_latent_prefill(const void* q1, const void* q2, const void* k1, const void* k2, const void* v, const void* gate,
+                         void* out, int B, int L, int T, int H, int d1, int d2, int dv, const int64_t q1_strides[3],
+                         const int64_t q2_strides[3], const int64_t k1_strides[3], const int64_t k2_strides[2],
+                         const int64_t v_strides[3], const int64_t out_strides[3], const int64_t gate_strides[2],
+                         int offset, float scale, int io_dtype, int impl, void* stream) {
+  if (!q1 || !q2 || !k1 || !k2 || !v || !out || (gate && !gate_strides)) return BASED_ERR_NULL;
+  if (!q1_strides || !q2_strides || !k1_strides || !k2_strides || !v_strides || !out_strides) return BASED_ERR_NULL;
+  if (!dtype_ok(io_dtype)) return BASED_ERR_DTYPE;
+  if (B < 0 || L < 0 || H <= 0 || d1 <= 0 || d2 <= 0 || dv <= 0 || offset < 0 || (int64_t)offset + L > T) return BASED_ERR_SHAPE;
+  if (B == 0 || L == 0) return BASED_OK;
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  const Strides3 sk2{k2_strides[0], 0, k2_strides[1]};
+  const int64_t gb = gate ? gate_strides[0] : 0, gl = gate ? gate_strides[1] : 0;
+  if (impl == BASED_IMPL_TCGEN05 || (impl == BASED_IMPL_AUTO && io_dtype == BASED_BF16)) {
+    if (io_dtype != BASED_BF16) return BASED_ERR_IMPL;
+    const int rc = launch_latent_prefill_tc(q1, q2, k1, k2, v, gate, out, B, L, T, H, d1, d2, dv, s3_blh(q1_strides),
+                                            s3_blh(q2_strides), s3_blh(k1_strides), sk2, s3_blh(v_strides),
+                                            s3_blh(out_strides), gb, gl, nullptr, offset, scale, st);
+    if (!(impl == BASED_IMPL_AUTO && rc == BASED_ERR_IMPL)) return rc;
+  }
+  return launch_split_key_attention(q1, q2, k1, k2, v, gate, out, B, L, H, d1, d2, dv, s3_blh(q1_strides),
+                                    s3_blh(q2_strides), s3_blh(k1_strides), sk2, s3_blh(v_strides), s3_blh(out_strides),
+                                    gb, gl, nullptr, offset, scale, io_dtype, st);
+}
+
+size_t based_latent_decode_scratch_bytes(int B, int L, int H, int kv_rank, int max_len) {
+  if (B <= 0 || L <= 0 || H <= 0 || kv_rank <= 0 || max_len <= 0) return 0;
+  return latent_decode_scratch_bytes(B, L * H, kv_rank, max_len);
+}
+
+int based_latent_decode(const void* qa, const void* qr, const void* cache, const void* gate, void* out, void* scratch,
+                        size_t scratch_bytes, int B, int L, int H, int kv_rank, int rot_dim, int max_len,
+                        const int64_t qa_strides[3], const int64_t qr_strides[3], const int64_t cache_strides[2],
+                        const int64_t out_strides[3], const int64_t gate_strides[2], const int32_t* offsets, int offset,
+                        float scale, int io_dtype, void* stream) {
+  if (!qa || !qr || !cache || !out || (gate && !gate_strides)) return BASED_ERR_NULL;
+  if (!qa_strides || !qr_strides || !cache_strides || !out_strides) return BASED_ERR_NULL;
+  if (!dtype_ok(io_dtype)) return BASED_ERR_DTYPE;
+  if (B < 0 || L < 0 || H <= 0 || kv_rank <= 0 || rot_dim <= 0 || max_len <= 0 || offset < 0) return BASED_ERR_SHAPE;
+  if (!offsets && (int64_t)offset + L > max_len) return BASED_ERR_SHAPE;
+  if (B == 0 || L == 0) return BASED_OK;
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  const int64_t gb = gate ? gate_strides[0] : 0, gl = gate ? gate_strides[1] : 0;
+  if (io_dtype == BASED_BF16) {
+    const int rc = launch_latent_decode(qa, qr, cache, gate, out, scratch, scratch_bytes, B, L, H, kv_rank, rot_dim, max_len,
+                                        s3_blh(qa_strides), s3_blh(qr_strides), cache_strides[0], cache_strides[1],
+                                        s3_blh(out_strides), gb, gl, offsets, offset, scale, st);
+    if (rc != BASED_ERR_IMPL) return rc;
+  }
+  // fp32 models and other sizes: the cached rows as keys and values of every head
+  const Strides3 sc{cache_strides[0], 0, cache_strides[1]};
+  const char* rot = static_cast<const char*>(cache) + kv_rank * dtype_size(io_dtype);
+  return launch_split_key_attention(qa, qr, cache, rot, cache, gate, out, B, L, H, kv_rank, rot_dim, kv_rank,
+                                    s3_blh(qa_strides), s3_blh(qr_strides), sc, sc, sc, s3_blh(out_strides), gb, gl, offsets,
+                                    offset, scale, io_dtype, st);
+}
+
 int based_delta_prefill(const void* q, const void* k, const void* v, const void* z, const void* a, const void* b,
                         const void* A_log, const void* dt_bias, const void* norm_weight, void* state, void* out, int B,
                         int L, int H, int Hk, int d, int dv, const int64_t q_strides[2], const int64_t k_strides[2],
                         const int64_t v_strides[2], const int64_t z_strides[2], const int64_t gate_strides[2],
                         const int64_t out_strides[2], const int32_t* offsets, int offset, float eps, int io_dtype,
-                        void* stream) {
+                        int impl, void* scratch, size_t scratch_bytes, void* stream) {
   if (!q || !k || !v || !z || !a || !b || !A_log || !dt_bias || !norm_weight || !state || !out) return BASED_ERR_NULL;
   if (!q_strides || !k_strides || !v_strides || !z_strides || !gate_strides || !out_strides) return BASED_ERR_NULL;
   if (!dtype_ok(io_dtype)) return BASED_ERR_DTYPE;
   if (B < 0 || L < 0 || H <= 0 || Hk <= 0 || H % Hk || d <= 0 || dv <= 0 || offset < 0) return BASED_ERR_SHAPE;
   if (B == 0 || L == 0) return BASED_OK;
+  // AUTO: chunks for bf16 from a handful of tokens on, else token by token
+  if (impl == BASED_IMPL_TCGEN05 || (impl == BASED_IMPL_AUTO && io_dtype == BASED_BF16 && L >= 8)) {
+    if (io_dtype != BASED_BF16) return BASED_ERR_IMPL;
+    const int rc = launch_delta_chunk(q, k, v, z, static_cast<const float*>(a), static_cast<const float*>(b),
+                                      static_cast<const float*>(A_log), static_cast<const float*>(dt_bias), norm_weight,
+                                      static_cast<float*>(state), out, scratch, scratch_bytes, B, L, H, Hk, d, dv,
+                                      s2(q_strides), s2(k_strides), s2(v_strides), s2(z_strides), s2(gate_strides),
+                                      s2(out_strides), offsets, offset, eps, static_cast<cudaStream_t>(stream));
+    if (!(impl == BASED_IMPL_AUTO && rc == BASED_ERR_IMPL)) return rc;
+  }
   return launch_delta_recurrent(q, k, v, z, static_cast<const float*>(a), static_cast<const float*>(b),
                                 static_cast<const float*>(A_log), static_cast<const float*>(dt_bias), norm_weight,
                                 static_cast<float*>(state), out, B, L, H, Hk, d, dv, s2(q_strides), s2(k_strides),
                                 s2(v_strides), s2(z_strides), s2(gate_strides), s2(out_strides), offsets, offset, eps,
                                 io_dtype, static_cast<cudaStream_t>(stream));
+}
+
+size_t based_delta_prefill_scratch_bytes(int B, int L, int H, int d, int dv) {
+  if (B <= 0 || L <= 0 || H <= 0 || d <= 0 || dv <= 0) return 0;
+  return delta_chunk_scratch_bytes(B, L, H, d, dv);
 }
 
 int based_delta_step(const void* x, const void* conv_weight, void* ring, const void* a, const void* b, const void* A_log,

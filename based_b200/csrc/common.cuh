@@ -147,4 +147,24 @@ int launch_rglru(const void* u, const void* y, const float* gates, const void* r
                  float* state, void* out, int B, int L, int W, int bw, Strides2 su, Strides2 sy, Strides2 so,
                  int64_t g_block, int64_t g_row, const int32_t* offsets, int offset, int io_dtype, cudaStream_t stream);
 
+int launch_latent_prefill_tc(const void* q1, const void* q2, const void* k1, const void* k2, const void* v,
+                             const void* gate, void* out, int B, int L, int T, int H, int d1, int d2, int dv, Strides3 sq1,
+                             Strides3 sq2, Strides3 sk1, Strides3 sk2, Strides3 sv, Strides3 so, int64_t gb, int64_t gl,
+                             const int32_t* offsets, int offset, float scale, cudaStream_t stream);
+int read_tc_status_latent(unsigned int* out, int reset);
+int latent_decode_splits(int B, int R, int max_len);
+size_t latent_decode_scratch_bytes(int B, int R, int r, int max_len);
+int launch_latent_decode(const void* q1, const void* q2, const void* cache, const void* gate, void* out, void* scratch,
+                         size_t scratch_bytes, int B, int L, int H, int r, int rd, int max_len, Strides3 sq1, Strides3 sq2,
+                         int64_t cb, int64_t cl, Strides3 so, int64_t gb, int64_t gl, const int32_t* offsets, int offset,
+                         float scale, cudaStream_t stream);
+
+int launch_delta_chunk(const void* q, const void* k, const void* v, const void* z, const float* a, const float* b,
+                       const float* A_log, const float* dt_bias, const void* norm_w, float* state, void* out, void* scratch,
+                       size_t scratch_bytes, int B, int L, int H, int Hk, int d, int dv, Strides2 sq, Strides2 sk,
+                       Strides2 sv, Strides2 sz, Strides2 sg, Strides2 so, const int32_t* offsets, int offset, float eps,
+                       cudaStream_t stream);
+size_t delta_chunk_scratch_bytes(int B, int L, int H, int d, int dv);
+int read_tc_status_delta(unsigned int* out, int reset);
+
 }  // namespace based

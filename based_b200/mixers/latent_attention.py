@@ -85,9 +85,7 @@ class LatentAttention(StatefulMixer):
         qa = torch.bmm(rows[..., :d].transpose(0, 1), uk)                        # [H, B L, r]
         ctx = torch.empty_like(qa)
         qa4, ctx4 = qa.view(H, B, L, r).permute(1, 2, 0, 3), ctx.view(H, B, L, r).permute(1, 2, 0, 3)
-        shared = cache.unsqueeze(2).expand(-1, -1, H, -1)
-        ops.split_key_attention(qa4, q[..., d:], shared[..., :r], shared[..., r:], shared[..., :r], self.scale, gate=gate,
-                                pos=pos, out=ctx4)
+        ops.latent_decode(qa4, q[..., d:], cache, self.scale, gate=gate, pos=pos, out=ctx4)
         # the gate scales a head's context, which commutes with W_uv
         torch.bmm(ctx, uv.transpose(1, 2), out=out.transpose(0, 1))
 
@@ -97,5 +95,4 @@ class LatentAttention(StatefulMixer):
         T = pos + L
         kv = ops.linear(cache[:, :T, :r], self.kv_up)                             # [B, T, H d + H dv]
         k, v = kv[..., :H * d].unflatten(-1, (H, d)), kv[..., H * d:].unflatten(-1, (H, dv))
-        kr = cache[:, :T, r:].unsqueeze(2).expand(-1, -1, H, -1)
-        ops.split_key_attention(q[..., :d], q[..., d:], k, kr, v, self.scale, gate=gate, pos=pos, out=out)
+        ops.latent_prefill(q[..., :d], q[..., d:], k, cache[:, :T, r:], v, self.scale, gate=gate, pos=pos, out=out)

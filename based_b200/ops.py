@@ -747,6 +747,62 @@ def split_key_attention(q1, q2, k1, k2, v, scale: float, *, gate: Optional[torch
     return out
 
 
+def latent_prefill(q1, q2, k1, k2, v, scale: float, *, gate: Optional[torch.Tensor] = None, pos: int = 0,
+                   out: torch.Tensor, impl: str = "auto") -> torch.Tensor:
+    """Expanded latent attention over a prompt or portion: q1, q2 ``[B, L, H, .]`` at positions ``pos ..``, per-head keys
+    k1 and values v ``[B, T, H, .]``, shared key part k2 ``[B, T, d2]``, ``gate [B, L, H]`` pre-sigmoid -> ``out [B, L, H, dv]``."""
+    _need_cuda(q1, q2, k1, k2, v, gate, out)
+    B, L, H, d1 = q1.shape
+    for t, n in ((q1, "q1"), (q2, "q2"), (k1, "k1"), (k2, "k2"), (v, "v"), (out, "out")):
+        _inner_contig(t, n)
+        if t.dtype != q1.dtype:
+            raise TypeError("all tensors must share a dtype")
+    if gate is not None:
+        _inner_contig(gate, "gate")
+    if out.numel() == 0:
+        return out
+    with torch.cuda.device(q1.device):
+        code = _capi.lib().based_latent_prefill(
+            q1.data_ptr(), q2.data_ptr(), k1.data_ptr(), k2.data_ptr(), v.data_ptr(), _ptr(gate), out.data_ptr(), B, L, k1.shape[1],
+            H, d1, q2.shape[-1], v.shape[-1], _capi.strides(*q1.stride()[:3]), _capi.strides(*q2.stride()[:3]),
+            _capi.strides(*k1.stride()[:3]), _capi.strides(*k2.stride()[:2]), _capi.strides(*v.stride()[:3]),
+            _capi.strides(*out.stride()[:3]), _capi.strides(*gate.stride()[:2]) if gate is not None else None, int(pos),
+            float(scale), _dt(q1.dtype), _IMPLS[impl], _stream())
+    _capi.check(code, "based_latent_prefill")
+    return out
+
+
+def latent_decode(qa, qr, cache, scale: float, *, gate: Optional[torch.Tensor] = None, pos=0,
+                  out: torch.Tensor) -> torch.Tensor:
+    """Absorbed latent attention for a few query rows: qa ``[B, L, H, kv_rank]``, qr ``[B, L, H, rot]``, ``cache [B, max_len,
+    kv_rank + rot]`` -> gated context ``out [B, L, H, kv_rank]``."""
+    _need_cuda(qa, qr, cache, gate, out)
+    B, L, H, r = qa.shape
+    rd = qr.shape[-1]
+    for t, n in ((qa, "qa"), (qr, "qr"), (cache, "cache"), (out, "out")):
+        _inner_contig(t, n)
+        if t.dtype != qa.dtype:
+            raise TypeError("all tensors must share a dtype")
+    if cache.shape[0] < B or cache.shape[2] != r + rd:
+        raise ValueError("cache must be [>= B, max_len, kv_rank + rot]")
+    if gate is not None:
+        _inner_contig(gate, "gate")
+    if out.numel() == 0:
+        return out
+    off, scalar = _position(pos, qa)
+    with torch.cuda.device(qa.device):
+        lib = _capi.lib()
+        need = lib.based_latent_decode_scratch_bytes(B, L, H, r, cache.shape[1])
+        scratch = torch.empty(need, dtype=torch.uint8, device=qa.device) if need else None
+        code = lib.based_latent_decode(
+            qa.data_ptr(), qr.data_ptr(), cache.data_ptr(), _ptr(gate), out.data_ptr(), _ptr(scratch), need, B, L, H, r, rd,
+            cache.shape[1], _capi.strides(*qa.stride()[:3]), _capi.strides(*qr.stride()[:3]), _capi.strides(*cache.stride()[:2]),
+            _capi.strides(*out.stride()[:3]), _capi.strides(*gate.stride()[:2]) if gate is not None else None, off, scalar,
+            float(scale), _dt(qa.dtype), _stream())
+    _capi.check(code, "based_latent_decode")
+    return out
+
+
 def _check_delta(state, B, H, d, dv, *params):
     if state.shape[0] < B or state.shape[1:] != (H, d, dv) or state.dtype != torch.float32 or not state.is_contiguous():
         raise ValueError("state must be a contiguous float32 [>= B, H, d, dv] tensor")
@@ -756,7 +812,7 @@ def _check_delta(state, B, H, d, dv, *params):
 
 
 def delta_prefill(q, k, v, z, a, b, A_log, dt_bias, norm_weight, state, *, pos=0, eps: float = 1e-6,
-                  out: torch.Tensor) -> torch.Tensor:
+                  out: torch.Tensor, impl: str = "auto") -> torch.Tensor:
     """Gated delta rule over ``L`` tokens: q, k ``[B, L, Hk, d]``, v, z ``[B, L, H, dv]`` (token-strided views, heads
     contiguous), a, b ``[B, L, H]`` fp32 pre-activations, ``state [B, H, d, dv]`` fp32 updated IN PLACE; ``out [B, L, H * dv]``."""
     _need_cuda(q, k, v, z, a, b, A_log, dt_bias, norm_weight, state, out)
@@ -773,11 +829,14 @@ def delta_prefill(q, k, v, z, a, b, A_log, dt_bias, norm_weight, state, *, pos=0
     if out.numel() == 0:
         return out
     with torch.cuda.device(q.device):
+        need = _capi.lib().based_delta_prefill_scratch_bytes(B, L, H, d, dv) if q.dtype == torch.bfloat16 and impl != "simt" else 0
+        scratch = torch.empty(need, dtype=torch.uint8, device=q.device) if need else None
         code = _capi.lib().based_delta_prefill(
             q.data_ptr(), k.data_ptr(), v.data_ptr(), z.data_ptr(), a.data_ptr(), b.data_ptr(), A_log.data_ptr(), dt_bias.data_ptr(),
             norm_weight.data_ptr(), state.data_ptr(), out.data_ptr(), B, L, H, Hk, d, dv, _capi.strides(*q.stride()[:2]),
             _capi.strides(*k.stride()[:2]), _capi.strides(*v.stride()[:2]), _capi.strides(*z.stride()[:2]),
-            _capi.strides(*a.stride()[:2]), _capi.strides(*out.stride()[:2]), off, scalar, float(eps), _dt(q.dtype), _stream())
+            _capi.strides(*a.stride()[:2]), _capi.strides(*out.stride()[:2]), off, scalar, float(eps), _dt(q.dtype), _IMPLS[impl],
+            _ptr(scratch), need, _stream())
     _capi.check(code, "based_delta_prefill")
     return out
 

@@ -457,16 +457,44 @@ int based_split_key_attention(const void* q1, const void* q2, const void* k1, co
                               int io_dtype, void* stream);
 
 /*
+ * The expanded form over a prompt or a portion of one: queries q1, q2 [B, L, H, .] at positions offset .. offset + L - 1,
+ * per-head keys k1 and values v [B, T, H, .], T >= offset + L, the shared key part k2 [B, T, d2] (strides batch, token).
+ * AUTO: the tensor-core kernel for bf16 when it takes the sizes (d1, d2, dv multiples of 16, dv <= 128, queries and at
+ * least one K and V tile in shared memory, strides multiples of 8, 16-byte alignment), else the CUDA-core kernel.
+ */
+int based_latent_prefill(const void* q1, const void* q2, const void* k1, const void* k2, const void* v, const void* gate,
+                         void* out, int B, int L, int T, int H, int d1, int d2, int dv, const int64_t q1_strides[3],
+                         const int64_t q2_strides[3], const int64_t k1_strides[3], const int64_t k2_strides[2],
+                         const int64_t v_strides[3], const int64_t out_strides[3], const int64_t gate_strides[2],
+                         int offset, float scale, int io_dtype, int impl, void* stream);
+
+/*
+ * The absorbed form for a few query rows: qa [B, L, H, kv_rank] = W_uk^T q, qr [B, L, H, rot_dim], cache rows
+ * [B, max_len, kv_rank + rot_dim] (strides batch, token) -> gated context out [B, L, H, kv_rank], to be multiplied by
+ * W_uv.  scratch: based_latent_decode_scratch_bytes bytes, 16-byte aligned (NULL when that is 0).
+ */
+size_t based_latent_decode_scratch_bytes(int B, int L, int H, int kv_rank, int max_len);
+int based_latent_decode(const void* qa, const void* qr, const void* cache, const void* gate, void* out, void* scratch,
+                        size_t scratch_bytes, int B, int L, int H, int kv_rank, int rot_dim, int max_len,
+                        const int64_t qa_strides[3], const int64_t qr_strides[3], const int64_t cache_strides[2],
+                        const int64_t out_strides[3], const int64_t gate_strides[2], const int32_t* offsets, int offset,
+                        float scale, int io_dtype, void* stream);
+
+/*
  * Gated delta rule over the tokens of a call.  q, k [B, L, Hk, d], v, z [B, L, H, dv] (after convolution and silu;
  * unit norms are taken here), a, b [B, L, H] pre-activations of decay and step size, state [B, H, d, dv] updated,
  * out [B, L, H, dv] = normed read-out * norm_weight * silu(z).  Strides are (batch, token), heads contiguous.
+ * AUTO: the chunked tensor-core kernel (BASED_IMPL_TCGEN05) for bf16 calls of 8 tokens or more with d in {32, 64, 96, 128},
+ * dv a multiple of 16, strides multiples of 8 and 16-byte alignment, else token by token (BASED_IMPL_SIMT).  scratch:
+ * based_delta_prefill_scratch_bytes bytes, 16-byte aligned (NULL when that is 0).
  */
+size_t based_delta_prefill_scratch_bytes(int B, int L, int H, int d, int dv);
 int based_delta_prefill(const void* q, const void* k, const void* v, const void* z, const void* a, const void* b,
                         const void* A_log, const void* dt_bias, const void* norm_weight, void* state, void* out, int B,
                         int L, int H, int Hk, int d, int dv, const int64_t q_strides[2], const int64_t k_strides[2],
                         const int64_t v_strides[2], const int64_t z_strides[2], const int64_t gate_strides[2],
                         const int64_t out_strides[2], const int32_t* offsets, int offset, float eps, int io_dtype,
-                        void* stream);
+                        int impl, void* scratch, size_t scratch_bytes, void* stream);
 
 /*
  * One token per row, from the packed projection x [B, q | k | v | z] to the gated output in one launch (convolution
