@@ -137,7 +137,7 @@ struct StepP {
 
 // NR float4 rows of the state per thread; thread t owns columns 4 (t mod dv/4) .. +3 of rows t / (dv/4), + R, ...
 template <typename T, int NR>
-__global__ void __launch_bounds__(kThreads) delta_step_kernel(const StepP p) {
+__global__ void __launch_bounds__(kThreads, NR <= 8 ? 3 : NR <= 16 ? 2 : 1) delta_step_kernel(const StepP p) {
   extern __shared__ float sm[];
   const int h = blockIdx.x, b = blockIdx.y, tid = threadIdx.x;
   const int hk = h / (p.H / p.Hk);

@@ -8,8 +8,9 @@
 // S^T -> (K S0)^T -> u^T -> S^T never leaves registers and warps meet only in the output norm.
 //
 // 32-bit without 32-bit operands: q and k enter as the bf16 values the convolution stored, their norms and all decays
-// are fp32 factors applied to fp32 sums; every fp32 matrix (S, u, A, P, the residual) is used as a bf16 pair hi + lo
-// (16 mantissa bits), products of two pairs as hi hi + hi lo + lo hi.
+// are fp32 factors applied to fp32 sums; in everything that enters the recurrence an fp32 matrix (S, u, A, T, the
+// residual) is used as a bf16 pair hi + lo (16 mantissa bits), products of two pairs as hi hi + hi lo + lo hi.  The
+// read-out S0^T q + P u, which nothing feeds back, multiplies bf16 operands once, like P V of an attention.
 //
 // The triangular system is solved by 16-token blocks: u_b = T_b (y_b - sum_{c<b} A_bc u_c) with T_b = (I + A_bb)^-1.
 //
@@ -20,6 +21,7 @@
 // Two buffers; `ready` hands a prepared chunk to the consumers, `done` hands the read-out and the buffer back.
 #include <initializer_list>
 #include <mutex>
+#include <type_traits>
 
 #include "seq_common.cuh"
 #include "tcgen05.cuh"
@@ -35,6 +37,7 @@ using bf16 = __nv_bfloat16;
 
 constexpr int C = 64;               // tokens per chunk
 constexpr int LT = C + 8;           // row stride of the [64, 64] operand tiles
+constexpr int LI = 20;              // row stride of the diagonal blocks, stored transposed
 constexpr int kConsumers = 8, kHelpers = 8;
 constexpr int NT = 32 * (kConsumers + kHelpers), HT = 32 * kHelpers;
 constexpr float kUnitEps = 1e-6f;
@@ -52,21 +55,23 @@ struct Params {
 };
 
 struct Layout {                     // byte offsets in shared memory
-  int ldk, ldv, K, Q, V, R, inv, gates, bars, total, tile_k, tile_v, region, ldo;
+  int ldk, ldv, K, Q, V, R, inv, gates, z, w, bars, total, tile_k, tile_v, region, ldo;
   __host__ __device__ Layout(int d, int vs) {
     ldk = d + 8; ldv = vs + 8; ldo = vs + 20;
     tile_k = C * ldk * 2; tile_v = C * ldv * 2;
-    const int mats = 4 * C * LT * 2, stage = C * ldo * 4;
+    const int mats = 3 * C * LT * 2, stage = C * ldo * 4;
     region = mats > stage ? mats : stage;
     K = 0; Q = K + 2 * tile_k; V = Q + 2 * tile_k; R = V + 2 * tile_v;
     inv = R + 2 * region;
-    gates = inv + 4 * 16 * 17 * 4;
-    bars = gates + 2 * 8 * C * 4;
+    gates = inv + 4 * 16 * LI * 4;
+    z = gates + 3 * 9 * C * 4;
+    w = z + HT * vs / 16 * 8;
+    bars = w + ((vs * 4 + 15) & ~15);
     total = bars + 64;
   }
 };
-// gates of one buffer, C floats each
-enum { G_CUM = 0, G_BETA, G_RK, G_RQ, G_EGK, G_EGQ, G_W, G_TOT };
+// gates of one chunk, C floats each; chunk c's sit in slot c mod 3
+enum { G_CUM = 0, G_BETA, G_RK, G_RQ, G_EGK, G_EGQ, G_W, G_COL, G_TOT, G_N };
 
 __device__ __forceinline__ void ldsm4(uint32_t (&r)[4], uint32_t a) {
   asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];\n" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(a));
@@ -122,51 +127,74 @@ __global__ void __launch_bounds__(NT, 1) delta_chunk_kernel(const Params p) {
     const float A = expf(p.A_log[h]), dt = p.dt_bias[h];
     const int g = lane >> 2, t4 = lane & 3;
 
-    auto prepare = [&](int c) {
-      const int buf = c & 1, base = c * C, n = min(C, p.L - base);
-      float* gt = reinterpret_cast<float*>(sm + lay.gates) + buf * 8 * C;
-      const uint32_t kt = sb + lay.K + buf * lay.tile_k, qt = sb + lay.Q + buf * lay.tile_k, vt = sb + lay.V + buf * lay.tile_v;
-      const bf16 *kp = p.k + b * p.sk.b + (int64_t)hk * d, *qp = p.q + b * p.sq.b + (int64_t)hk * d,
-                 *vp = p.v + b * p.sv.b + (int64_t)h * p.dv + v0;
-      for (int e = ht; e < C * (d / 8); e += HT) {
-        const int i = e / (d / 8), cc = e % (d / 8);
-        const bool ok = i < n;
-        const int64_t l = base + (ok ? i : 0);
-        cp_async16(kt + i * lay.ldk * 2 + cc * 16, kp + l * p.sk.h + cc * 8, ok);
-        cp_async16(qt + i * lay.ldk * 2 + cc * 16, qp + l * p.sq.h + cc * 8, ok);
+    const bf16 *kp = p.k + b * p.sk.b + (int64_t)hk * d, *qp = p.q + b * p.sq.b + (int64_t)hk * d,
+               *vp = p.v + b * p.sv.b + (int64_t)h * p.dv + v0;
+    auto gates_of = [&](int c) { return reinterpret_cast<float*>(sm + lay.gates) + (c % 3) * G_N * C; };
+    // decays and step sizes of chunk c, two tokens per lane of one warp; tokens past the end neither decay nor write
+    auto gates = [&](int c) {
+      float* gt = gates_of(c);
+      float lg[2] = {0.f, 0.f}, be[2] = {0.f, 0.f};
+#pragma unroll
+      for (int e = 0; e < 2; ++e) {
+        const int l = c * C + 2 * lane + e;
+        if (l < p.L) {
+          const int64_t gi = b * p.sg.b + (int64_t)l * p.sg.h + h;
+          lg[e] = -A * seq::softplus_acc(p.a[gi] + dt);
+          be[e] = seq::sigmoid_acc(p.b[gi]);
+        }
       }
-      const int vc = p.vs / 8;
-      for (int e = ht; e < C * vc; e += HT) {
-        const int i = e / vc, cc = e - i * vc;
+      float s = lg[0] + lg[1];
+#pragma unroll
+      for (int o = 1; o < 32; o <<= 1) {
+        const float t = __shfl_up_sync(0xffffffffu, s, o);
+        if (lane >= o) s += t;
+      }
+      gt[G_CUM * C + 2 * lane] = s - lg[1];
+      gt[G_CUM * C + 2 * lane + 1] = s;
+      gt[G_BETA * C + 2 * lane] = be[0];
+      gt[G_BETA * C + 2 * lane + 1] = be[1];
+      if (lane == 31) gt[G_TOT * C] = s;
+    };
+    // q, k, v of chunk c into its buffer, and those of the chunk after it towards L2
+    auto load = [&](int c) {
+      const int buf = c & 1, base = c * C, n = min(C, p.L - base);
+      const uint32_t kt = sb + lay.K + buf * lay.tile_k, qt = sb + lay.Q + buf * lay.tile_k, vt = sb + lay.V + buf * lay.tile_v;
+      constexpr int RS = HT / (d / 8);   // rows per pass (HT is a multiple of d / 8 for d = 32, 64, 128; d = 96 leaves threads idle)
+      const int r0 = ht / (d / 8), cc = ht % (d / 8);
+      if (r0 < RS) {
+        const bf16 *ks = kp + (int64_t)(base + r0) * p.sk.h + cc * 8, *qs = qp + (int64_t)(base + r0) * p.sq.h + cc * 8;
+        uint32_t dst = r0 * lay.ldk * 2 + cc * 16;
+#pragma unroll
+        for (int i = r0; i < C; i += RS) {
+          const bool ok = i < n;
+          cp_async16(kt + dst, ok ? ks : kp, ok);
+          cp_async16(qt + dst, ok ? qs : qp, ok);
+          ks += RS * p.sk.h;
+          qs += RS * p.sq.h;
+          dst += RS * lay.ldk * 2;
+        }
+      }
+      {
+        const int i = ht >> 2;   // four threads per row
         const bool ok = i < n;
-        cp_async16(vt + i * lay.ldv * 2 + cc * 16, vp + (int64_t)(base + (ok ? i : 0)) * p.sv.h + cc * 8, ok);
+        const bf16* src = vp + (int64_t)(base + (ok ? i : 0)) * p.sv.h;
+        for (int cc = ht & 3; cc < p.vs / 8; cc += 4) cp_async16(vt + i * lay.ldv * 2 + cc * 16, src + cc * 8, ok);
+        const int64_t next = base + C + i;
+        if (next < p.L) {
+          for (int x = 32 * (ht & 3); x < d; x += 128) {   // 64-byte pieces
+            asm volatile("prefetch.global.L2 [%0];" ::"l"(kp + next * p.sk.h + x));
+            asm volatile("prefetch.global.L2 [%0];" ::"l"(qp + next * p.sq.h + x));
+          }
+          for (int x = 32 * (ht & 3); x < p.vs; x += 128) asm volatile("prefetch.global.L2 [%0];" ::"l"(vp + next * p.sv.h + x));
+        }
       }
       cp_async_commit();
-      if (hw == 0) {  // gates: two tokens per lane; tokens past the end neither decay nor write
-        float lg[2], be[2];
-#pragma unroll
-        for (int e = 0; e < 2; ++e) {
-          const int i = 2 * lane + e;
-          lg[e] = 0.f; be[e] = 0.f;
-          if (i < n) {
-            const int64_t gi = b * p.sg.b + (int64_t)(base + i) * p.sg.h + h;
-            lg[e] = -A * seq::softplus_acc(p.a[gi] + dt);
-            be[e] = seq::sigmoid_acc(p.b[gi]);
-          }
-        }
-        float s = lg[0] + lg[1];
-#pragma unroll
-        for (int o = 1; o < 32; o <<= 1) {
-          const float t = __shfl_up_sync(0xffffffffu, s, o);
-          if (lane >= o) s += t;
-        }
-        gt[G_CUM * C + 2 * lane] = s - lg[1];
-        gt[G_CUM * C + 2 * lane + 1] = s;
-        gt[G_BETA * C + 2 * lane] = be[0];
-        gt[G_BETA * C + 2 * lane + 1] = be[1];
-        if (lane == 31) gt[G_TOT * C] = s;
-      }
-      cp_async_wait_all();
+    };
+    auto prepare = [&](int c) {
+      const int buf = c & 1;
+      float* gt = gates_of(c);
+      const uint32_t kt = sb + lay.K + buf * lay.tile_k, qt = sb + lay.Q + buf * lay.tile_k;
+      cp_async_wait_1();   // only the gate values of the next read-out may still be on their way
       bar_sync(1, HT);
       {  // squared norms of the 64 k rows and the 64 q rows, two threads per row
         const int row = ht >> 1, i = row & (C - 1);
@@ -191,114 +219,179 @@ __global__ void __launch_bounds__(NT, 1) delta_chunk_kernel(const Params p) {
             gt[G_RK * C + i] = r;
             gt[G_EGK * C + i] = expf(G) * r;
             gt[G_W * C + i] = expf(gt[G_TOT * C] - G) * r;
+            gt[G_COL * C + i] = expf(gt[G_CUM * C + (i | 15)] - G) * r;   // decay from here to the end of the 16-block
           }
         }
       }
       bar_sync(1, HT);
-      // 16 x 16 blocks of K K^T (below and on the diagonal) and Q K^T
+      // 16 x 16 blocks of K K^T and Q K^T on and below the diagonal, both products of a block by one warp; the diagonal
+      // ones first.  Off the diagonal e^{G_i - G_j} splits at the end of j's block into two factors of at most 1.
       bf16* Th = reinterpret_cast<bf16*>(sm + lay.R + buf * lay.region);
-      bf16 *Tl = Th + C * LT, *Ph = Tl + C * LT, *Pl = Ph + C * LT;
-      for (int t = hw; t < 20; t += kHelpers) {
-        const bool is_q = t >= 10;
-        int x = is_q ? t - 10 : t, bi = 0;
-        while (x > bi) { x -= bi + 1; ++bi; }
-        const int bj = x;
-        float acc[2][4] = {};
-        const uint32_t aa = (is_q ? qt : kt) + ((bi * 16 + (lane & 15)) * lay.ldk + (lane >> 4) * 8) * 2;
+      bf16 *Tl = Th + C * LT, *Ph = Tl + C * LT;
+      for (int t = hw; t < 10; t += kHelpers) {
+        const int bi = t < 4 ? t : t == 4 ? 1 : t < 7 ? 2 : 3, bj = t < 4 ? t : t == 4 ? 0 : t < 7 ? t - 5 : t - 7;
+        float kk2[2][4] = {}, qk2[2][4] = {};
+        const uint32_t ra = ((bi * 16 + (lane & 15)) * lay.ldk + (lane >> 4) * 8) * 2;
         const uint32_t ba = kt + ((bj * 16 + (lane & 7) + (lane >> 4) * 8) * lay.ldk + ((lane >> 3) & 1) * 8) * 2;
 #pragma unroll
         for (int kk = 0; kk < DK; ++kk) {
-          uint32_t fa[4], fb[4];
-          ldsm4(fa, aa + kk * 32);
+          uint32_t fk[4], fq[4], fb[4];
           ldsm4(fb, ba + kk * 32);
-          mma(acc[0], fa, fb[0], fb[1]);
-          mma(acc[1], fa, fb[2], fb[3]);
+          ldsm4(fk, kt + ra + kk * 32);
+          ldsm4(fq, qt + ra + kk * 32);
+          mma(kk2[0], fk, fb[0], fb[1]);
+          mma(kk2[1], fk, fb[2], fb[3]);
+          mma(qk2[0], fq, fb[0], fb[1]);
+          mma(qk2[1], fq, fb[2], fb[3]);
         }
+        const bool diag = bi == bj;
+        const float end = gt[G_CUM * C + bj * 16 + 15];
 #pragma unroll
         for (int half = 0; half < 2; ++half) {
-          const int i = bi * 16 + g + 8 * half;
-          const float Gi = gt[G_CUM * C + i], fi = is_q ? gt[G_RQ * C + i] : gt[G_BETA * C + i] * gt[G_RK * C + i];
+          const int ii = g + 8 * half, i = bi * 16 + ii;
+          const float Gi = gt[G_CUM * C + i];
+          float fk = gt[G_BETA * C + i] * gt[G_RK * C + i], fq = gt[G_RQ * C + i];
+          if (!diag) {
+            const float ei = expf(Gi - end);
+            fk *= -ei;
+            fq *= ei;
+          }
 #pragma unroll
           for (int nt = 0; nt < 2; ++nt) {
-            const int j = bj * 16 + nt * 8 + 2 * t4;
-            float val[2];
-#pragma unroll
-            for (int e = 0; e < 2; ++e) {
-              const bool seen = is_q ? j + e <= i : j + e < i;
-              val[e] = seen ? acc[nt][2 * half + e] * fi * gt[G_RK * C + j + e] * expf(Gi - gt[G_CUM * C + j + e]) : 0.f;
-            }
-            if (!is_q && bi == bj) {
-              inv[(bi * 16 + g + 8 * half) * 17 + nt * 8 + 2 * t4] = val[0];
-              inv[(bi * 16 + g + 8 * half) * 17 + nt * 8 + 2 * t4 + 1] = val[1];
+            const int jj = nt * 8 + 2 * t4, j = bj * 16 + jj;
+            float a0 = kk2[nt][2 * half] * fk, a1 = kk2[nt][2 * half + 1] * fk, p0 = qk2[nt][2 * half] * fq, p1 = qk2[nt][2 * half + 1] * fq;
+            if (diag) {
+              const float2 gj = *reinterpret_cast<const float2*>(gt + G_CUM * C + j), rk = *reinterpret_cast<const float2*>(gt + G_RK * C + j);
+              const float e0 = jj <= ii ? expf(Gi - gj.x) * rk.x : 0.f, e1 = jj + 1 <= ii ? expf(Gi - gj.y) * rk.y : 0.f;
+              inv[(bi * 16 + jj) * LI + ii] = jj < ii ? a0 * e0 : 0.f;
+              inv[(bi * 16 + jj + 1) * LI + ii] = jj + 1 < ii ? a1 * e1 : 0.f;
+              p0 *= e0;
+              p1 *= e1;
             } else {
+              const float2 cj = *reinterpret_cast<const float2*>(gt + G_COL * C + j);
               uint32_t hi, lo;
-              if (is_q) split(val[0], val[1], hi, lo);
-              else split(-val[0], -val[1], hi, lo);
-              *reinterpret_cast<uint32_t*>((is_q ? Ph : Th) + i * LT + j) = hi;
-              *reinterpret_cast<uint32_t*>((is_q ? Pl : Tl) + i * LT + j) = lo;
+              split(a0 * cj.x, a1 * cj.y, hi, lo);
+              *reinterpret_cast<uint32_t*>(Th + i * LT + j) = hi;
+              *reinterpret_cast<uint32_t*>(Tl + i * LT + j) = lo;
+              p0 *= cj.x;
+              p1 *= cj.y;
             }
+            *reinterpret_cast<uint32_t*>(Ph + i * LT + j) = pack_bf16(p0, p1);
           }
         }
       }
+      if (hw == kHelpers - 1 && c + 1 < nc) gates(c + 1);
       bar_sync(1, HT);
-      if (ht < C) {  // one column of one diagonal block's inverse per thread, by forward substitution
-        const int blk = ht >> 4, col = ht & 15;
+      if (hw < 4 && lane < 16) {  // one column of one diagonal block's inverse per thread
         float t[16];
 #pragma unroll
-        for (int i = 0; i < 16; ++i) {
-          float s = i == col ? 1.f : 0.f;
+        for (int i = 0; i < 16; ++i) t[i] = i == lane ? 1.f : 0.f;
 #pragma unroll
-          for (int k = 0; k < i; ++k) s = fmaf(-inv[(blk * 16 + i) * 17 + k], t[k], s);
-          t[i] = s;
-          const bf16 hi = __float2bfloat16_rn(s);
-          Th[(blk * 16 + i) * LT + blk * 16 + col] = hi;
-          Tl[(blk * 16 + i) * LT + blk * 16 + col] = __float2bfloat16_rn(s - __bfloat162float(hi));
+        for (int k = 0; k < 15; ++k) {
+          float col[16];   // column k of the block, from its diagonal's 4-group on
+#pragma unroll
+          for (int i4 = k / 4 * 4; i4 < 16; i4 += 4) {
+            const float4 x = *reinterpret_cast<const float4*>(inv + (hw * 16 + k) * LI + i4);
+            col[i4] = x.x; col[i4 + 1] = x.y; col[i4 + 2] = x.z; col[i4 + 3] = x.w;
+          }
+#pragma unroll
+          for (int i = k + 1; i < 16; ++i) t[i] = fmaf(-col[i], t[k], t[i]);
+        }
+#pragma unroll
+        for (int i = 0; i < 16; ++i) {
+          const bf16 hi = __float2bfloat16_rn(t[i]);
+          Th[(hw * 16 + i) * LT + hw * 16 + lane] = hi;
+          Tl[(hw * 16 + i) * LT + hw * 16 + lane] = __float2bfloat16_rn(t[i] - __bfloat162float(hi));
         }
       }
       mbar_arrive(READY + 8 * buf);
     };
 
+    // 4 threads per token of a chunk, every 4th group of 4 values
+    const int fi = ht >> 2, fpart = ht & 3, groups = p.vs / 4;
+    constexpr int FG = 8;      // groups per thread at 128 columns
+    // z values of the next read-out, 8 bytes per group, read back by the thread that copied them
+    const uint32_t zs = sb + lay.z + ht * 8;
+    const uint2* zr = reinterpret_cast<const uint2*>(sm + lay.z) + ht;
+    auto fetch_z = [&](int c) {
+      const int l = c * C + fi;
+      if (!p.raw && l < p.L) {
+        const bf16* zp = p.z + b * p.sz.b + (int64_t)l * p.sz.h + (int64_t)h * p.dv;
+#pragma unroll
+        for (int r = 0; r < FG; ++r)
+          if (fpart + 4 * r < groups)
+            asm volatile("cp.async.ca.shared.global [%0], [%1], 8;\n" ::"r"(zs + r * HT * 8), "l"(zp + 4 * (fpart + 4 * r)) : "memory");
+      }
+      cp_async_commit();
+    };
     auto finish = [&](int c) {  // read-out of chunk c -> output
-      const int buf = c & 1, base = c * C, n = min(C, p.L - base);
-      const float* st = reinterpret_cast<const float*>(sm + lay.R + buf * lay.region);
-      const int i = ht >> 2, part = ht & 3, groups = p.vs / 4;   // 4 threads per token, every 4th group of 4 values
+      const int buf = c & 1, l = c * C + fi;
+      const float* st = reinterpret_cast<const float*>(sm + lay.R + buf * lay.region) + fi * lay.ldo;
       if (p.raw) {
-        if (i < n) {
-          float* dst = p.raw + (((int64_t)b * p.L + base + i) * p.H + h) * p.dv + v0;
-          for (int e = part; e < groups; e += 4)
-            *reinterpret_cast<float4*>(dst + 4 * e) = *reinterpret_cast<const float4*>(st + i * lay.ldo + 4 * e);
+        if (l < p.L) {
+          float* dst = p.raw + (((int64_t)b * p.L + l) * p.H + h) * p.dv + v0;
+          for (int e = fpart; e < groups; e += 4)
+            *reinterpret_cast<float4*>(dst + 4 * e) = *reinterpret_cast<const float4*>(st + 4 * e);
         }
         return;
       }
+      const float* wn = reinterpret_cast<const float*>(sm + lay.w);
       float ss = 0.f;
-      for (int e = part; e < groups; e += 4) {
-        const float4 x = *reinterpret_cast<const float4*>(st + i * lay.ldo + 4 * e);
+      for (int e = fpart; e < groups; e += 4) {
+        const float4 x = *reinterpret_cast<const float4*>(st + 4 * e);
         ss += x.x * x.x + x.y * x.y + x.z * x.z + x.w * x.w;
       }
       ss += __shfl_xor_sync(0xffffffffu, ss, 1);
       ss += __shfl_xor_sync(0xffffffffu, ss, 2);
-      if (i >= n) return;
+      if (l >= p.L) return;
       const float rstd = rsqrtf(ss / (float)p.dv + p.eps);
-      const bf16* zp = p.z + b * p.sz.b + (int64_t)(base + i) * p.sz.h + (int64_t)h * p.dv;
-      bf16* op = p.out + b * p.so.b + (int64_t)(base + i) * p.so.h + (int64_t)h * p.dv;
-      for (int e = part; e < groups; e += 4) {
-        const float4 x = *reinterpret_cast<const float4*>(st + i * lay.ldo + 4 * e);
-        float zv[4], w[4];
-        seq::Pack<bf16, 4>::load(zp + 4 * e, zv);
-        seq::Pack<bf16, 4>::load(p.norm_w + 4 * e, w);
-        const float xv[4] = {x.x, x.y, x.z, x.w};
-        float o[4];
+      bf16* op = p.out + b * p.so.b + (int64_t)l * p.so.h + (int64_t)h * p.dv;
+      auto some = [&](int r0, auto count) {   // groups r0 .. r0 + count - 1 of this thread, without branches in between
+        constexpr int N = decltype(count)::value;
+        float4 x[N], w[N];
+        uint2 z[N];
 #pragma unroll
-        for (int r = 0; r < 4; ++r) o[r] = xv[r] * rstd * w[r] * seq::silu_t<bf16>(zv[r]);
-        seq::Pack<bf16, 4>::store(op + 4 * e, o);
-      }
+        for (int r = 0; r < N; ++r) {
+          const int e = fpart + 4 * (r0 + r);
+          x[r] = *reinterpret_cast<const float4*>(st + 4 * e);
+          w[r] = *reinterpret_cast<const float4*>(wn + 4 * e);
+          z[r] = zr[(r0 + r) * HT];
+        }
+#pragma unroll
+        for (int r = 0; r < N; ++r) {
+          const float o[4] = {x[r].x * rstd * w[r].x * seq::silu_t<bf16>(seq::bf16_lo(z[r].x)),
+                              x[r].y * rstd * w[r].y * seq::silu_t<bf16>(seq::bf16_hi(z[r].x)),
+                              x[r].z * rstd * w[r].z * seq::silu_t<bf16>(seq::bf16_lo(z[r].y)),
+                              x[r].w * rstd * w[r].w * seq::silu_t<bf16>(seq::bf16_hi(z[r].y))};
+          seq::Pack<bf16, 4>::store(op + 4 * (fpart + 4 * (r0 + r)), o);
+        }
+      };
+      const int mine = p.vs / 16;
+      int r0 = 0;
+      for (; r0 + 4 <= mine; r0 += 4) some(r0, std::integral_constant<int, 4>{});
+      for (; r0 < mine; ++r0) some(r0, std::integral_constant<int, 1>{});
     };
 
+    // Copy groups in order: tiles(0), z(0), [tiles(1),] then per chunk tiles(c + 2), z(c + 1): whoever waits for a group
+    // leaves one younger group in flight.
+    if (!p.raw)
+      for (int e = ht; e < p.vs; e += HT) reinterpret_cast<float*>(sm + lay.w)[e] = __bfloat162float(p.norm_w[e]);
+    if (hw == kHelpers - 1) gates(0);
+    load(0);
+    fetch_z(0);
     prepare(0);
-    if (nc > 1) prepare(1);
+    if (nc > 1) {
+      load(1);
+      cp_async_commit();   // an empty group, so that the wait below is for the tiles
+      prepare(1);
+    }
     for (int c = 0; c < nc; ++c) {
       mbar_wait_bounded(DONE + 8 * (c & 1), (c >> 1) & 1, abort_flag, p.status, 1u << 16);
+      if (c + 2 < nc) load(c + 2);   // lands while the read-out is finished
+      else cp_async_commit();
+      cp_async_wait_1();             // z(c)
       finish(c);
+      if (c + 1 < nc) fetch_z(c + 1);
       if (c + 2 < nc) {
         bar_sync(1, HT);   // every helper has read the stage before the next chunk's matrices overwrite it
         prepare(c + 2);
@@ -324,9 +417,9 @@ __global__ void __launch_bounds__(NT, 1) delta_chunk_kernel(const Params p) {
       const uint32_t v_lane = ((lane & 15) * lay.ldv + (lane >> 4) * 8 + 16 * warp) * 2;                // transposed: [tokens 16][cols 16]
       for (int c = 0; c < nc; ++c) {
         const int buf = c & 1;
-        const float* gt = reinterpret_cast<const float*>(sm + lay.gates) + buf * 8 * C;
+        const float* gt = reinterpret_cast<const float*>(sm + lay.gates) + (c % 3) * G_N * C;
         const uint32_t kt = sb + lay.K + buf * lay.tile_k, qt = sb + lay.Q + buf * lay.tile_k, vt = sb + lay.V + buf * lay.tile_v;
-        const uint32_t th = sb + lay.R + buf * lay.region + t_lane, tl = th + C * LT * 2, ph = tl + C * LT * 2, pl = ph + C * LT * 2;
+        const uint32_t th = sb + lay.R + buf * lay.region + t_lane, tl = th + C * LT * 2, ph = tl + C * LT * 2;
         mbar_wait_bounded(READY + 8 * buf, (c >> 1) & 1, abort_flag, p.status, 1u << 17);
         float x[8][4], o[8][4];   // [16 value columns, 64 tokens]: S0^T k, then the residual, then u; S0^T q, then the read-out
 #pragma unroll
@@ -348,8 +441,6 @@ __global__ void __launch_bounds__(NT, 1) delta_chunk_kernel(const Params p) {
             ldsm4(fb, qt + b_lane + (np * 16 * lay.ldk + kk * 16) * 2);
             mma(o[2 * np], ah, fb[0], fb[1]);
             mma(o[2 * np + 1], ah, fb[2], fb[3]);
-            mma(o[2 * np], al, fb[0], fb[1]);
-            mma(o[2 * np + 1], al, fb[2], fb[3]);
           }
         }
         // y = beta (v - e^G S0^T khat); decayed read-out of S0
@@ -401,11 +492,6 @@ __global__ void __launch_bounds__(NT, 1) delta_chunk_kernel(const Params p) {
               mma(x[2 * np + 1], fh, mh[2], mh[3]);
             }
             ldsm4(mh, ph + (np * 16 * LT + bb * 16) * 2);
-            ldsm4(ml, pl + (np * 16 * LT + bb * 16) * 2);
-            mma(o[2 * np], fl, mh[0], mh[1]);
-            mma(o[2 * np + 1], fl, mh[2], mh[3]);
-            mma(o[2 * np], fh, ml[0], ml[1]);
-            mma(o[2 * np + 1], fh, ml[2], ml[3]);
             mma(o[2 * np], fh, mh[0], mh[1]);
             mma(o[2 * np + 1], fh, mh[2], mh[3]);
           }

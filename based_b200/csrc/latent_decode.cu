@@ -1,7 +1,7 @@
 // Latent attention in its absorbed form for a few query rows: every head of every query attends over the SAME cached
 // rows [latent | rotated key], so 16 (query, head) rows share one read of the cache.
 //   s[row, t] = (qa[row] . c_t + qr[row] . kr_t) * scale,   ctx[row] = sigmoid(gate[row]) * sum_t softmax(s)[row, t] c_t
-// HBM-bound on the cache.  A CTA of 4 warps walks its share of the keys in tiles of 32, two tiles in flight
+// HBM-bound on the cache.  A CTA of 8 warps walks its share of the keys in tiles of 32, two tiles in flight
 // (cp.async), two CTAs per SM so that one's products run under the other's waits; scores and context use mma.sync m16n8k16 (16 rows are exactly the tile height, the operands are a few
 // hundred flops per cached byte at most), softmax in fp32.  Several CTAs split the keys of a sequence; a second launch
 // merges their partial results.  The split follows the sequence's current length, read on the device.
@@ -13,7 +13,7 @@
 namespace based {
 namespace {
 
-constexpr int kWarps = 4, kThreads = kWarps * 32, kTile = 32, kPad = 8;
+constexpr int kWarps = 8, kThreads = kWarps * 32, kTile = 32, kPad = 8;
 constexpr int kRows = 16 / kWarps;   // softmax rows per warp
 
 struct P {
@@ -47,8 +47,8 @@ __global__ void __launch_bounds__(kThreads, 2) latent_decode_kernel(const P p) {
   const int D = p.r + p.rd, ld = D + kPad;      // row stride: an odd number of 16-byte units, so ldmatrix has no conflicts
   __nv_bfloat16* Q = reinterpret_cast<__nv_bfloat16*>(smem);                 // [16][ld]
   __nv_bfloat16* K = Q + 16 * ld;                                            // [2][32][ld]
-  float* S = reinterpret_cast<float*>(K + 2 * kTile * ld);                   // [16][32 + 4]
-  __nv_bfloat16* Pm = reinterpret_cast<__nv_bfloat16*>(S + 16 * (kTile + 4)); // [16][32 + 8]
+  float* S = reinterpret_cast<float*>(K + 2 * kTile * ld);                   // [2][16][32 + 4]: two halves of the dims
+  __nv_bfloat16* Pm = reinterpret_cast<__nv_bfloat16*>(S + 32 * (kTile + 4)); // [16][32 + 8]
   float* corr = reinterpret_cast<float*>(Pm + 16 * (kTile + 8));             // [16]
   float* msum = corr + 16;                                                   // [16][2]
   const int pos0 = seq::position0(p.offsets, p.offset, b);
@@ -99,32 +99,29 @@ __global__ void __launch_bounds__(kThreads, 2) latent_decode_kernel(const P p) {
     }
     __syncthreads();
     const __nv_bfloat16* Kt = K + buf * kTile * ld;
-    {  // scores of keys 8 warp .. 8 warp + 7
+    {  // scores of keys 8 (warp mod 4) .. + 7 over one half of the dims, in pairs of 16
+      const int kq = warp & 3, pairs = (D / 16 + 1) / 2, kb = (warp >> 2) ? (pairs + 1) / 2 : 0, ke = (warp >> 2) ? pairs : (pairs + 1) / 2;
       float s[2][4] = {};
       const uint32_t qa = tc::smem_u32(Q + (lane & 15) * ld + (lane >> 4) * 8);
-      const uint32_t ka = tc::smem_u32(Kt + (8 * warp + (lane & 7)) * ld + (lane >> 3) * 8);   // four k-halves: 32 columns
-      int k = 0;
-#pragma unroll 4
-      for (; k + 2 <= D / 16; k += 2) {
+      const uint32_t krow = tc::smem_u32(Kt + (8 * kq + (lane & 7)) * ld), ka = krow + (lane >> 3) * 16;   // four k-halves
+#pragma unroll 3
+      for (int k = kb; k < ke; ++k) {
         uint32_t a0[4], a1[4], bb[4];
-        ldsm4(a0, qa + k * 32);
-        ldsm4(a1, qa + k * 32 + 32);
-        ldsm4(bb, ka + k * 32);
-        mma16816(s[0], a0, bb[0], bb[1]);
-        mma16816(s[1], a1, bb[2], bb[3]);
+        ldsm4(a0, qa + k * 64);
+        if (2 * k + 1 < D / 16) {
+          ldsm4(a1, qa + k * 64 + 32);
+          ldsm4(bb, ka + k * 64);
+          mma16816(s[0], a0, bb[0], bb[1]);
+          mma16816(s[1], a1, bb[2], bb[3]);
+        } else {   // the last 16 of an odd number: the upper lanes repeat their addresses
+          ldsm4(bb, krow + ((lane >> 3) & 1) * 16 + k * 64);
+          mma16816(s[0], a0, bb[0], bb[1]);
+        }
       }
-      if (k < D / 16) {
-        uint32_t a0[4], bb[4];
-        ldsm4(a0, qa + k * 32);
-        // only the first two k-halves exist; the upper lanes repeat their addresses
-        ldsm4(bb, tc::smem_u32(Kt + (8 * warp + (lane & 7)) * ld + ((lane >> 3) & 1) * 8) + k * 32);
-        mma16816(s[0], a0, bb[0], bb[1]);
-      }
-      const int c = 8 * warp + 2 * t4;
-      S[g * (kTile + 4) + c] = s[0][0] + s[1][0];
-      S[g * (kTile + 4) + c + 1] = s[0][1] + s[1][1];
-      S[(g + 8) * (kTile + 4) + c] = s[0][2] + s[1][2];
-      S[(g + 8) * (kTile + 4) + c + 1] = s[0][3] + s[1][3];
+      float* Sh = S + (warp >> 2) * 16 * (kTile + 4);
+      const int c = 8 * kq + 2 * t4;
+      *reinterpret_cast<float2*>(Sh + g * (kTile + 4) + c) = make_float2(s[0][0] + s[1][0], s[0][1] + s[1][1]);
+      *reinterpret_cast<float2*>(Sh + (g + 8) * (kTile + 4) + c) = make_float2(s[0][2] + s[1][2], s[0][3] + s[1][3]);
     }
     __syncthreads();
 #pragma unroll
@@ -132,7 +129,7 @@ __global__ void __launch_bounds__(kThreads, 2) latent_decode_kernel(const P p) {
       const int rr = kRows * warp + i, row = row0 + rr;
       const int last = row < p.R ? pos0 + row / p.H : -1;   // last key this row sees
       const int key = t * kTile + lane;
-      const float a = key <= last ? S[rr * (kTile + 4) + lane] * p.scale_log2e : -INFINITY;
+      const float a = key <= last ? (S[rr * (kTile + 4) + lane] + S[(16 + rr) * (kTile + 4) + lane]) * p.scale_log2e : -INFINITY;
       const float mn = fmaxf(m[i], warp_max(a));
       const float base = mn == -INFINITY ? 0.f : mn;
       const float ea = exp2f(a - base), f = exp2f(m[i] - base);
@@ -194,22 +191,28 @@ __global__ void __launch_bounds__(kThreads, 2) latent_decode_kernel(const P p) {
   }
 }
 
-// grid (R, B, ceil(r / 64)): 32 column pairs x 4 groups of splits per block
+// G groups of splits times 128 / G column pairs per block; grid (R, B, ceil(r / (256 / G)))
+template <int G>
 __global__ void __launch_bounds__(128) latent_decode_merge_kernel(const P p) {
-  const int row = blockIdx.x, b = blockIdx.y, tid = threadIdx.x, grp = tid >> 5;
-  const int c = blockIdx.z * 64 + 2 * (tid & 31);
+  constexpr int W = 128 / G;
+  const int row = blockIdx.x, b = blockIdx.y, tid = threadIdx.x, grp = tid / W, lane = tid % W;
+  const int c = blockIdx.z * 2 * W + 2 * lane;
   const int64_t stride = (int64_t)p.B * p.R * (p.r + 2);
   const float* src = p.part + ((int64_t)b * p.R + row) * (p.r + 2);
-  __shared__ float red[4], wsum[4], acc[4][64];
   float m = -INFINITY;
-  for (int s = tid; s < p.splits; s += 128) m = fmaxf(m, src[s * stride + p.r]);
-  m = warp_max(m);
-  if ((tid & 31) == 0) red[grp] = m;
-  __syncthreads();
-  m = fmaxf(fmaxf(red[0], red[1]), fmaxf(red[2], red[3]));
+  if (G > 1) {
+    __shared__ float red[4];
+    for (int s = tid; s < p.splits; s += 128) m = fmaxf(m, src[s * stride + p.r]);
+    m = warp_max(m);
+    if ((tid & 31) == 0) red[tid >> 5] = m;
+    __syncthreads();
+    m = fmaxf(fmaxf(red[0], red[1]), fmaxf(red[2], red[3]));
+  } else {
+    for (int s = 0; s < p.splits; ++s) m = fmaxf(m, src[s * stride + p.r]);
+  }
   float sum = 0.f, x = 0.f, y = 0.f;
 #pragma unroll 4
-  for (int s = grp; s < p.splits; s += 4) {
+  for (int s = grp; s < p.splits; s += G) {
     const float ms = src[s * stride + p.r];
     const float w = ms == -INFINITY ? 0.f : exp2f(ms - m);   // a split without keys wrote zeros
     sum = fmaf(w, src[s * stride + p.r + 1], sum);
@@ -219,21 +222,26 @@ __global__ void __launch_bounds__(128) latent_decode_merge_kernel(const P p) {
       y = fmaf(w, v.y, y);
     }
   }
-  if ((tid & 31) == 0) wsum[grp] = sum;
-  acc[grp][2 * (tid & 31)] = x;
-  acc[grp][2 * (tid & 31) + 1] = y;
-  __syncthreads();
-  if (grp != 0 || c >= p.r) return;
-  const int l = row / p.H, h = row - l * p.H, e = 2 * tid;
-  float f = 1.0f / (wsum[0] + wsum[1] + wsum[2] + wsum[3]);
+  if (G > 1) {
+    __shared__ float wsum[G], acc[G][2 * W];
+    if (lane == 0) wsum[grp] = sum;
+    acc[grp][2 * lane] = x;
+    acc[grp][2 * lane + 1] = y;
+    __syncthreads();
+    if (grp != 0) return;
+    sum = x = y = 0.f;
+#pragma unroll
+    for (int i = 0; i < G; ++i) { sum += wsum[i]; x += acc[i][2 * lane]; y += acc[i][2 * lane + 1]; }
+  }
+  if (c >= p.r) return;
+  const int l = row / p.H, h = row - l * p.H;
+  float f = 1.0f / sum;
   if (p.gate) f *= seq::sigmoid_acc(__bfloat162float(p.gate[b * p.gb + l * p.gl + h]));
-  x = acc[0][e] + acc[1][e] + acc[2][e] + acc[3][e];
-  y = acc[0][e + 1] + acc[1][e + 1] + acc[2][e + 1] + acc[3][e + 1];
   *reinterpret_cast<uint32_t*>(p.out + b * p.so.b + l * p.so.l + h * p.so.h + c) = seq::bf16x2_bits(x * f, y * f);
 }
 
 size_t smem_bytes(int D) {
-  return (size_t)(16 + 2 * kTile) * (D + kPad) * 2 + 16 * (kTile + 4) * 4 + 16 * (kTile + 8) * 2 + 16 * 3 * 4;
+  return (size_t)(16 + 2 * kTile) * (D + kPad) * 2 + 32 * (kTile + 4) * 4 + 16 * (kTile + 8) * 2 + 16 * 3 * 4;
 }
 constexpr int kMaxSmem = 227 * 1024;
 
@@ -242,7 +250,8 @@ int launch_nw(const P& p, cudaStream_t st) {
   const cudaError_t e = cudaFuncSetAttribute(latent_decode_kernel<NW>, cudaFuncAttributeMaxDynamicSharedMemorySize, kMaxSmem);
   if (e != cudaSuccess) return (int)e;
   latent_decode_kernel<NW><<<dim3(p.splits, (p.R + 15) / 16, p.B), kThreads, smem_bytes(p.r + p.rd), st>>>(p);
-  if (p.splits > 1) latent_decode_merge_kernel<<<dim3(p.R, p.B, (p.r + 63) / 64), 128, 0, st>>>(p);
+  if (p.splits > 16) latent_decode_merge_kernel<8><<<dim3(p.R, p.B, (p.r + 31) / 32), 128, 0, st>>>(p);
+  else if (p.splits > 1) latent_decode_merge_kernel<1><<<dim3(p.R, p.B, (p.r + 255) / 256), 128, 0, st>>>(p);
   return (int)cudaGetLastError();
 }
 
@@ -284,8 +293,7 @@ int launch_latent_decode(const void* q1, const void* q2, const void* cache, cons
   if (nw <= 1) return launch_nw<1>(p, stream);
   if (nw <= 2) return launch_nw<2>(p, stream);
   if (nw <= 4) return launch_nw<4>(p, stream);
-  if (nw <= 8) return launch_nw<8>(p, stream);
-  return launch_nw<16>(p, stream);
+  return launch_nw<8>(p, stream);
 }
 
 }  // namespace based
