@@ -65,6 +65,7 @@ SIGNATURES = {
     "based_delta_prefill": (c_int, [c_void_p] * 11 + [c_int] * 6 + [_I64P] * 6 + _POS
                             + [c_float, c_int, c_int, c_void_p, ctypes.c_size_t, c_void_p]),
     "based_delta_step": (c_int, [c_void_p] * 10 + [c_int] * 6 + [c_int64] * 3 + _POS + [c_float, c_int, c_void_p]),
+    "based_rglru_gated": (c_int, [c_void_p] * 8 + [c_int] * 4 + [_I64P] * 3 + _POS + [c_int, c_void_p]),
     "based_rglru": (c_int, [c_void_p] * 8 + [c_int] * 4 + [_I64P] * 4 + _POS + [c_int, c_void_p]),
 }
 

@@ -36,13 +36,14 @@ const char* based_error_string(int code) {
 }
 
 int based_read_status(unsigned int* out, int reset) {
-  unsigned int a = 0, b = 0, c = 0, d = 0, e = 0;
+  unsigned int a = 0, b = 0, c = 0, d = 0, e = 0, f = 0;
   int rc = read_tc_status(&a, reset);
   if (rc == 0) rc = read_tc_status_swa(&b, reset);
   if (rc == 0) rc = read_tp_status(&c, reset);
   if (rc == 0) rc = read_tc_status_latent(&d, reset);
   if (rc == 0) rc = read_tc_status_delta(&e, reset);
-  if (out) *out = a | b | c | d | e;
+  if (rc == 0) rc = read_tc_status_rglru(&f, reset);
+  if (out) *out = a | b | c | d | e | f;
   return rc;
 }
 
@@ -519,6 +520,21 @@ int based_rglru(const void* u, const void* y, const void* gates, const void* r_b
                       static_cast<float*>(state), out, B, L, W, block_width, s2(u_strides), s2(y_strides),
                       s2(out_strides), gate_strides[0], gate_strides[1], offsets, offset, io_dtype,
                       static_cast<cudaStream_t>(stream));
+}
+
+int based_rglru_gated(const void* u, const void* y, const void* gate_weight, const void* r_bias, const void* i_bias,
+                      const void* lam, void* state, void* out, int B, int L, int W, int block_width,
+                      const int64_t u_strides[2], const int64_t y_strides[2], const int64_t out_strides[2],
+                      const int32_t* offsets, int offset, int io_dtype, void* stream) {
+  if (!u || !y || !gate_weight || !r_bias || !i_bias || !lam || !state || !out) return BASED_ERR_NULL;
+  if (!u_strides || !y_strides || !out_strides) return BASED_ERR_NULL;
+  if (!dtype_ok(io_dtype)) return BASED_ERR_DTYPE;
+  if (B < 0 || L < 0 || W <= 0 || block_width <= 0 || W % block_width || offset < 0) return BASED_ERR_SHAPE;
+  if (B == 0 || L == 0) return BASED_OK;
+  if (io_dtype != BASED_BF16) return BASED_ERR_IMPL;
+  return launch_rglru_tc(u, y, gate_weight, r_bias, i_bias, static_cast<const float*>(lam), static_cast<float*>(state), out,
+                         B, L, W, block_width, s2(u_strides), s2(y_strides), s2(out_strides), offsets, offset,
+                         static_cast<cudaStream_t>(stream));
 }
 
 }  // extern "C"

@@ -167,4 +167,9 @@ int launch_delta_chunk(const void* q, const void* k, const void* v, const void* 
 size_t delta_chunk_scratch_bytes(int B, int L, int H, int d, int dv);
 int read_tc_status_delta(unsigned int* out, int reset);
 
+int launch_rglru_tc(const void* u, const void* y, const void* w, const void* rb, const void* ib, const float* lam,
+                    float* state, void* out, int B, int L, int W, int n, Strides2 su, Strides2 sy, Strides2 so,
+                    const int32_t* offsets, int offset, cudaStream_t stream);
+int read_tc_status_rglru(unsigned int* out, int reset);
+
 }  // namespace based

@@ -114,11 +114,12 @@ class GenerationMixin:
         """Decoding: one prompt pass, then one token per step (generation.py:93-204); greedy by default, top-k /
         nucleus / temperature sampling as :func:`sample_token` otherwise.  With ``cg`` the decode step is
         captured once in a CUDA graph and replayed (:689-739).  Returns ``[B, L + max_new_tokens]``.
-        ``timings``, when given, receives device times in ms: ``prefill_ms``, ``decode_ms`` (all steps).
+        ``timings``, when given, receives device times in ms: ``prefill_ms``, ``decode_ms`` (all steps, with the graph's
+        capture), ``steps_ms`` (the steps alone).
         ``portion`` > 0 feeds the prompt that many tokens at a time (models that support portions)."""
         B, L = input_ids.shape
         ip = self.new_inference_params(B, L + max_new_tokens)
-        ev = [torch.cuda.Event(enable_timing=True) for _ in range(3)]
+        ev = [torch.cuda.Event(enable_timing=True) for _ in range(4)]
         out = torch.empty(B, L + max_new_tokens, dtype=input_ids.dtype, device=input_ids.device)
         out[:, :L] = input_ids
         ev[0].record()
@@ -151,6 +152,7 @@ class GenerationMixin:
             with torch.cuda.graph(graph):
                 step()
             self._restore_state(ip, cur, saved)
+        ev[3].record()
         for i in range(steps_left):
             if graph is not None:
                 graph.replay()
@@ -164,6 +166,7 @@ class GenerationMixin:
             ops.check_status()   # the device is idle here: a tensor-core kernel that gave up on a wait shows now
             timings["prefill_ms"] = ev[0].elapsed_time(ev[1])
             timings["decode_ms"] = ev[1].elapsed_time(ev[2])
+            timings["steps_ms"] = ev[3].elapsed_time(ev[2])
         return out
 
     @staticmethod

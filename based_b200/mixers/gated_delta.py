@@ -9,7 +9,7 @@ import torch
 import torch.nn as nn
 
 from .. import ops
-from .stateful import PackedLinear, StatefulMixer
+from .stateful import PackedLinear, StatefulMixer, pad_up
 
 
 class GatedDelta(StatefulMixer):
@@ -23,7 +23,7 @@ class GatedDelta(StatefulMixer):
         self.conv_channels = 2 * kv_heads * dim + heads * vdim
         self.in_proj = PackedLinear(width, [("qkv", self.conv_channels), ("g", heads * vdim)], **fk)
         self.z_offset = self.in_proj.offsets["g"][0]
-        self.gate_proj = nn.Linear(width, 2 * heads, bias=False, **fk)          # a, then b
+        self.gate_proj = nn.Parameter(torch.zeros(pad_up(2 * heads), width, **fk))   # a, then b
         self.conv_weight = nn.Parameter(torch.zeros(self.conv_channels, conv, **fk))
         self.norm_weight = nn.Parameter(torch.ones(vdim, **fk))
         self.A_log = nn.Parameter(torch.zeros(heads, device=device, dtype=torch.float32))
@@ -43,8 +43,8 @@ class GatedDelta(StatefulMixer):
                 self.conv_weight[at:at + n].copy_(t.get(prefix + name + ".conv", (n, self.taps)))
                 at += n
             self.in_proj.set("g", t.get(prefix + "g", (H * dv, W)))
-            self.gate_proj.weight[:H].copy_(t.get(prefix + "a", (H, W)))
-            self.gate_proj.weight[H:].copy_(t.get(prefix + "b", (H, W)))
+            self.gate_proj[:H].copy_(t.get(prefix + "a", (H, W)))
+            self.gate_proj[H:2 * H].copy_(t.get(prefix + "b", (H, W)))
             self.A_log.copy_(t.get(prefix + "A_log", (H,)))
             self.dt_bias.copy_(t.get(prefix + "dt_bias", (H,)))
             self.norm_weight.copy_(t.get(prefix + "norm", (dv,)))
@@ -61,8 +61,8 @@ class GatedDelta(StatefulMixer):
         st = self.state(inference_params, h.dtype)
         pos = self.position(inference_params, L)
         x = self.in_proj(h)
-        ab = ops.linear_f32(h, self.gate_proj.weight)
-        a, b = ab[..., :H], ab[..., H:]
+        ab = ops.linear_f32(h, self.gate_proj)
+        a, b = ab[..., :H], ab[..., H:2 * H]
         if L == 1 and self.z_offset == C:
             if ops.delta_step(x[:, 0], self.conv_weight, st["ring"], a[:, 0], b[:, 0], self.A_log, self.dt_bias,
                               self.norm_weight, st["state"], Hk, pos=pos, eps=self.eps, out=out[:, 0]):

@@ -20,7 +20,7 @@ class RGLRU(StatefulMixer):
         self.in_proj = PackedLinear(width, [("x", inner), ("y", inner)], bias=True, **fk)
         self.conv_weight = nn.Parameter(torch.zeros(inner, conv, **fk))
         self.conv_bias = nn.Parameter(torch.zeros(inner, **fk))
-        self.gate_weight = nn.Parameter(torch.zeros(blocks, n, 2 * n, **fk))    # [in, (r | i) out] per block
+        self.gate_weight = nn.Parameter(torch.zeros(blocks, 2, n, n, **fk))    # r and i matrices, [out, in]
         self.r_bias = nn.Parameter(torch.zeros(inner, **fk))
         self.i_bias = nn.Parameter(torch.zeros(inner, **fk))
         self.lam = nn.Parameter(torch.zeros(inner, device=device, dtype=torch.float32))
@@ -37,8 +37,8 @@ class RGLRU(StatefulMixer):
                 self.in_proj.set(name, t.get(prefix + name, (R, W)), t.get(prefix + name + ".b", (R,)))
             self.conv_weight.copy_(t.get(prefix + "conv", (R, self.taps)))
             self.conv_bias.copy_(t.get(prefix + "conv.b", (R,)))
-            self.gate_weight[..., :n].copy_(t.get(prefix + "ra", (nb, n, n)).transpose(1, 2))
-            self.gate_weight[..., n:].copy_(t.get(prefix + "ri", (nb, n, n)).transpose(1, 2))
+            self.gate_weight[:, 0].copy_(t.get(prefix + "ra", (nb, n, n)))
+            self.gate_weight[:, 1].copy_(t.get(prefix + "ri", (nb, n, n)))
             self.r_bias.copy_(t.get(prefix + "ra.b", (nb, n)).reshape(R))
             self.i_bias.copy_(t.get(prefix + "ri.b", (nb, n)).reshape(R))
             self.lam.copy_(t.get(prefix + "lam", (R,)))
@@ -55,5 +55,5 @@ class RGLRU(StatefulMixer):
         pos = self.position(inference_params, L)
         x = self.in_proj(h)
         u = ops.short_conv(self.in_proj.slice(x, "x"), self.conv_weight, self.conv_bias, ring=st["ring"], pos=pos)
-        gates = ops.block_gates(u, self.gate_weight)
-        ops.rglru(u, self.in_proj.slice(x, "y"), gates, self.r_bias, self.i_bias, self.lam, st["state"], pos=pos, out=out)
+        ops.rglru_gated(u, self.in_proj.slice(x, "y"), self.gate_weight, self.r_bias, self.i_bias, self.lam, st["state"], pos=pos,
+                        out=out)

@@ -868,14 +868,14 @@ def delta_step(x, conv_weight, ring, a, b, A_log, dt_bias, norm_weight, state, k
 
 
 def block_gates(u: torch.Tensor, weight: torch.Tensor) -> torch.Tensor:
-    """Block-diagonal product with an fp32 result: ``u [B, L, blocks * n]`` by ``weight [blocks, n, out]`` ->
-    ``[blocks, B * L, out]``."""
+    """Block-diagonal gate products with an fp32 result: ``u [B, L, blocks * n]`` by ``weight [blocks, 2, n, n]`` (r and i
+    matrices, stored [out, in]) -> ``[blocks, B * L, 2 n]``."""
     _need_cuda(u, weight)
-    nb, n, _ = weight.shape
-    x = u.reshape(-1, nb, n).transpose(0, 1)
+    nb, _, n, _ = weight.shape
+    x, w = u.reshape(-1, nb, n).transpose(0, 1), weight.view(nb, 2 * n, n).transpose(1, 2)
     if u.dtype == torch.float32:
-        return torch.bmm(x, weight)
-    return torch.bmm(x, weight, out_dtype=torch.float32)
+        return torch.bmm(x, w)
+    return torch.bmm(x, w, out_dtype=torch.float32)
 
 
 def rglru(u, y, gates, r_bias, i_bias, lam, state, *, pos=0, out: torch.Tensor) -> torch.Tensor:
@@ -900,3 +900,31 @@ def rglru(u, y, gates, r_bias, i_bias, lam, state, *, pos=0, out: torch.Tensor) 
             _capi.strides(*out.stride()[:2]), _capi.strides(gates.stride(0), gates.stride(1)), off, scalar, _dt(u.dtype), _stream())
     _capi.check(code, "based_rglru")
     return out
+
+
+# tokens from which the one-pass kernel is used; below it, the gate products and the recurrence are two launches
+RGLRU_FUSED_MIN_TOKENS = 8
+
+
+def rglru_gated(u, y, gate_weight, r_bias, i_bias, lam, state, *, pos=0, out: torch.Tensor) -> torch.Tensor:
+    """The recurrent unit with its gate products (``gate_weight`` as in :func:`block_gates`): one pass on the tensor cores
+    for bf16 prompts and portions, else :func:`block_gates` and :func:`rglru`."""
+    _need_cuda(u, y, gate_weight, r_bias, i_bias, lam, state, out)
+    B, L, W = u.shape
+    nb, _, n, _ = gate_weight.shape
+    if u.dtype == torch.bfloat16 and L >= RGLRU_FUSED_MIN_TOKENS and B > 0:
+        if (nb * n != W or not gate_weight.is_contiguous() or gate_weight.dtype != u.dtype or lam.dtype != torch.float32
+                or state.dtype != torch.float32 or state.shape[0] < B or state.shape[1] != W or not state.is_contiguous()):
+            raise ValueError("gate_weight must be [blocks, 2, n, n] in u's dtype, state [>= B, W] and lam float32, contiguous")
+        for t, name in ((u, "u"), (y, "y"), (out, "out")):
+            _inner_contig(t, name)
+        off, scalar = _position(pos, u)
+        with torch.cuda.device(u.device):
+            code = _capi.lib().based_rglru_gated(
+                u.data_ptr(), y.data_ptr(), gate_weight.data_ptr(), r_bias.data_ptr(), i_bias.data_ptr(), lam.data_ptr(),
+                state.data_ptr(), out.data_ptr(), B, L, W, n, _capi.strides(*u.stride()[:2]), _capi.strides(*y.stride()[:2]),
+                _capi.strides(*out.stride()[:2]), off, scalar, _dt(u.dtype), _stream())
+        if code != _capi.ERR_IMPL:
+            _capi.check(code, "based_rglru_gated")
+            return out
+    return rglru(u, y, block_gates(u, gate_weight), r_bias, i_bias, lam, state, pos=pos, out=out)

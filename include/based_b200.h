@@ -516,6 +516,15 @@ int based_rglru(const void* u, const void* y, const void* gates, const void* r_b
                 const int64_t y_strides[2], const int64_t out_strides[2], const int64_t gate_strides[2],
                 const int32_t* offsets, int offset, int io_dtype, void* stream);
 
+/*
+ * The same with the gate products inside (tensor cores, bf16): gate_weight [blocks, 2, n, n], r and i matrices stored
+ * [out, in], n = block_width.  BASED_ERR_IMPL for fp32, n not a multiple of 16 or above 256, or unaligned u.
+ */
+int based_rglru_gated(const void* u, const void* y, const void* gate_weight, const void* r_bias, const void* i_bias,
+                      const void* lam, void* state, void* out, int B, int L, int W, int block_width,
+                      const int64_t u_strides[2], const int64_t y_strides[2], const int64_t out_strides[2],
+                      const int32_t* offsets, int offset, int io_dtype, void* stream);
+
 #ifdef __cplusplus
 }
 #endif

@@ -158,7 +158,7 @@ def test_delta_step(H, Hk, d, dv, taps, dtype):
     assert rel_err(got.float().cpu().view(B, L, H, dv), ref) < tol
 
 
-@pytest.mark.parametrize("W,blocks", [(64, 4), (96, 1), (40, 5), (24, 24), (512, 2)])
+@pytest.mark.parametrize("W,blocks", [(64, 4), (96, 1), (40, 5), (24, 24), (512, 2), (320, 2), (128, 1), (144, 1), (384, 1)])
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
 def test_rglru(W, blocks, dtype):
     from based_b200 import ops
@@ -176,7 +176,7 @@ def test_rglru(W, blocks, dtype):
         ref.append(S * R.gelu_tanh(y[i].double()))
         last.append(S[-1])
     ref, last = torch.stack(ref), torch.stack(last)
-    gw = torch.cat([ra.transpose(1, 2), ri.transpose(1, 2)], -1).contiguous().cuda()
+    gw = torch.stack([ra, ri], 1).contiguous().cuda()
     ud, yd = u.cuda(), y.cuda()
     for seed in range(3):
         state = torch.full((B, W), 5.0, device="cuda")
@@ -184,9 +184,10 @@ def test_rglru(W, blocks, dtype):
         at = 0
         for m in ([L] if seed == 0 else [1] * L if seed == 1 else cuts(L, seed)):
             pos = torch.full((B,), at, dtype=torch.int32, device="cuda") if seed == 1 else at
-            ops.rglru(ud[:, at:at + m], yd[:, at:at + m], ops.block_gates(ud[:, at:at + m], gw), rb.reshape(W).cuda(), ib.reshape(W).cuda(),
-                      lam.cuda(), state, pos=pos, out=out[:, at:at + m])
+            ops.rglru_gated(ud[:, at:at + m], yd[:, at:at + m], gw, rb.reshape(W).cuda(), ib.reshape(W).cuda(), lam.cuda(), state,
+                            pos=pos, out=out[:, at:at + m])
             at += m
+        ops.check_status()
         assert rel_err(state.cpu(), last) < 2e-5
         assert rel_err(out.float().cpu(), ref) < (2e-5 if dtype == torch.float32 else 1e-2)
 
