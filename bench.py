@@ -468,7 +468,7 @@ def generation_bench(B=16, L=2048, new_tokens=512, size="360m"):
     res = {"model": f"based-{size} (random init)", "params": nparam, "B_per_gpu": B, "B_total": world * B, "prompt": L,
            "new_tokens": new_tokens, "sharding": "batch-sharded replicas, no communication",
            "prefill_ms": pre_ms, "prefill_tok_per_s": world * B * L / (pre_ms * 1e-3),
-           "decode_ms_per_step": dec_ms / steps, "decode_tok_per_s": world * B * steps / (dec_ms * 1e-3),
+           "steps_ms_per_step": t["steps_ms"] / steps, "decode_ms_per_step": dec_ms / steps, "decode_tok_per_s": world * B * steps / (dec_ms * 1e-3),
            "decode": f"CUDA graph replay of one step ({cfg.n_layer} blocks + lm_head + argmax)"}
     del model
     torch.cuda.empty_cache()
@@ -577,6 +577,194 @@ def tp_bench(dev, world):
     return out
 
 
+def razesun_config(size):
+    """A Razesun stack of the Based model's size and layer mix: RG-LRU layers where that has BaseConv, gated delta where
+    it has LinearAttention, latent attention where it has SlidingAttention (every second one reads the cache of the one
+    before it)."""
+    from based_b200.model import BasedConfig
+    cfg = BasedConfig.based_360m() if size == "360m" else BasedConfig.based_1b()
+    d, ff = cfg.n_embd, 2 * cfg.n_embd
+    heads = d // 128
+    layers, own = [], None
+    for i in range(cfg.n_layer):
+        if i in cfg.alt_mixer_layers:
+            layer = {"type": "delta", "mixer": {"heads": heads, "kv_heads": heads, "dim": 128, "vdim": 128, "conv": 4}}
+        elif i in cfg.alt_mixer_2_layers:
+            m = {"heads": heads, "dim": 128, "rot_dim": 64, "vdim": 128, "q_rank": 512, "kv_rank": 256, "scale": 192 ** -0.5,
+                 "rot": {"base": 1e4, "dims": 64}}
+            if own is None:
+                own = i
+            else:
+                m["kv_from"], own = own, None
+            layer = {"type": "latent_attention", "mixer": m}
+        else:
+            layer = {"type": "rglru", "mixer": {"width": d, "blocks": heads, "conv": 4}}
+        layer["mlp"] = {"kind": "dense", "ff": ff}
+        layers.append(layer)
+    return {"architecture": "Razesun", "vocab": cfg.padded_vocab_size, "width": d, "layers": layers, "norm": {"eps": 1e-6},
+            "residual_mult": 0.5, "logit_scale": 1.0}
+
+
+def random_razesun(size, device="cuda"):
+    from based_b200.registry import build_model
+    torch.manual_seed(0)
+    model = build_model(razesun_config(size), device=device, dtype=torch.bfloat16).eval()
+    with torch.no_grad():
+        for name, p in model.named_parameters():
+            if p.dim() > 1:
+                p.normal_(0, 0.02)
+            elif name.endswith("lam"):
+                p.fill_(-4.0)
+    return model
+
+
+def razesun_generation(B, L, new_tokens, size):
+    """Prompt pass and CUDA-graph decode of a Razesun stack, the same measurement as generation_bench."""
+    model = random_razesun(size)
+    ids = torch.randint(0, model.config.vocab_size, (B, L), device="cuda")
+    model.generate(ids, max_new_tokens=8, cg=True)
+    t = {}
+    model.generate(ids, max_new_tokens=new_tokens, cg=True, timings=t)
+    res = {"model": f"razesun-{size} (random init)", "params": sum({p.data_ptr(): p.numel() for p in model.parameters()}.values()),
+           "B": B, "prompt": L, "new_tokens": new_tokens, "prefill_ms": t["prefill_ms"],
+           "prefill_tok_per_s": B * L / (t["prefill_ms"] * 1e-3), "steps_ms_per_step": t["steps_ms"] / (new_tokens - 1),
+           "decode_tok_per_s": B * (new_tokens - 1) / (t["steps_ms"] * 1e-3)}
+    del model
+    torch.cuda.empty_cache()
+    return res
+
+
+def razesun_kernels(ops, peaks):
+    """Every kernel of the design at layer sizes of a 2048-wide model, and the like kernel of the Based model, as
+    fractions of their rooflines (the slower of algorithmic bytes at the HBM peak and flops at the bf16 peak); L2 is
+    flushed before every call."""
+    from based_b200.mixers import RotaryEmbedding
+    dev = "cuda"
+    flush = torch.empty(256 * 1024 * 1024, dtype=torch.uint8, device=dev)
+    g = torch.Generator(device=dev).manual_seed(0)
+
+    def rnd(*shape, dtype=torch.bfloat16, scale=1.0):
+        return (torch.randn(*shape, device=dev, generator=g) * scale).to(dtype)
+
+    out = {}
+
+    def record(name, what, fn, nbytes, flop=0, iters=10, like=None):
+        t = time_flushed(fn, flush, iters)[0]
+        t_hbm, t_tc = nbytes / (peaks["hbm_gbs"] * 1e9) * 1e3, flop / (peaks["bf16_tflops"] * 1e12) * 1e3
+        out[name] = {"what": what, "ms": t, "roofline_ms": max(t_hbm, t_tc), "frac": max(t_hbm, t_tc) / t,
+                     "bound": "hbm" if t_hbm >= t_tc else "tensor", "like": like}
+
+    with torch.inference_mode():
+        B, L, Hn, d = 8, 8192, 16, 128
+        C, n = 3 * Hn * d, Hn * d
+        y, z = rnd(B, L, C), rnd(B, L, Hn, d)
+        a, b = rnd(B, L, Hn, dtype=torch.float32), rnd(B, L, Hn, dtype=torch.float32)
+        A, dt, w = rnd(Hn, dtype=torch.float32), rnd(Hn, dtype=torch.float32), rnd(d)
+        S, o = torch.zeros(B, Hn, d, d, device=dev), torch.empty(B, L, n, dtype=torch.bfloat16, device=dev)
+        part = [y[..., i * n:(i + 1) * n].unflatten(-1, (Hn, d)) for i in range(3)]
+        record("delta_prefill", "B=8 L=8192 H=16 d=128 dv=128", lambda: ops.delta_prefill(*part, z, a, b, A, dt, w, S, out=o),
+               B * L * Hn * (5 * d * 2 + 8), 6 * d * d * B * L * Hn, like="linattn_prefill")
+        cw, ring = rnd(C, 4), torch.zeros(B, 4, C, dtype=torch.bfloat16, device=dev)
+        record("short_conv", "B=8 L=8192 C=6144 taps=4 silu", lambda: ops.short_conv(y, cw, ring=ring, silu=True), B * L * C * 4,
+               like="gated_conv")
+        del y, z, part, o
+        Bd = 256
+        x, ring = rnd(Bd, C + n), torch.zeros(Bd, 4, C, dtype=torch.bfloat16, device=dev)
+        S, o = torch.zeros(Bd, Hn, d, d, device=dev), torch.empty(Bd, n, dtype=torch.bfloat16, device=dev)
+        a, b = rnd(Bd, Hn, dtype=torch.float32), rnd(Bd, Hn, dtype=torch.float32)
+        pos = torch.full((Bd,), 100, dtype=torch.int32, device=dev)
+        record("delta_step", "B=256 H=16 d=128 dv=128", lambda: ops.delta_step(x, cw, ring, a, b, A, dt, w, S, Hn, pos=pos, out=o),
+               S.numel() * 8 + Bd * (C * 2 * 5 + 2 * n * 2), like="linattn_decode")
+        del S, x
+        W, nb = 2048, 8
+        u, yy = rnd(B, L, W), rnd(B, L, W)
+        gw, lam, st = rnd(nb, 2, W // nb, W // nb, scale=0.05), torch.full((W,), -4.0, device=dev), torch.zeros(B, W, device=dev)
+        rb, o = rnd(W), torch.empty(B, L, W, dtype=torch.bfloat16, device=dev)
+        record("rglru_gated", "B=8 L=8192 W=2048, 8 blocks: gate products and recurrence",
+               lambda: ops.rglru_gated(u, yy, gw, rb, rb, lam, st, out=o), B * L * W * 6, 4 * B * L * W * (W // nb), like="gated_conv")
+        del u, yy, o
+        u1, st1 = rnd(Bd, 1, W), torch.zeros(Bd, W, device=dev)
+        o1, gates = torch.empty_like(u1), rnd(nb, Bd, 2 * W // nb, dtype=torch.float32)
+        record("rglru_step", "B=256 W=2048", lambda: ops.rglru(u1, u1, gates, rb, rb, lam, st1, pos=pos, out=o1), Bd * W * (8 + 8 + 6),
+               like="gated_conv_step")
+        for Bp, Lp in ((4, 8192), (8, 2048)):
+            rd = 64
+            q, kv, kr = rnd(Bp, Lp, Hn, d + rd), rnd(Bp, Lp, Hn * 2 * d), rnd(Bp, Lp, rd)
+            o, gate = torch.empty(Bp, Lp, Hn, d, dtype=torch.bfloat16, device=dev), rnd(Bp, Lp, Hn)
+            k, v = kv[..., :n].unflatten(-1, (Hn, d)), kv[..., n:].unflatten(-1, (Hn, d))
+            record(f"latent_prefill_L{Lp}", f"B={Bp} L={Lp} H=16 d=128+64 dv=128",
+                   lambda: ops.latent_prefill(q[..., :d], q[..., d:], k, kr, v, 192 ** -0.5, gate=gate, out=o),
+                   (q.numel() + kv.numel() + kr.numel() + o.numel()) * 2, Bp * Hn * Lp * Lp * (d + rd + d), like="swa_prefill")
+            del q, kv, o, k, v
+        r, T = 512, 4096
+        for Bp in (64, 16):
+            cache, q = rnd(Bp, T, r + rd), rnd(Bp, 1, Hn, r + rd)
+            o, pos = torch.empty(Bp, 1, Hn, r, dtype=torch.bfloat16, device=dev), torch.full((Bp,), T - 1, dtype=torch.int32, device=dev)
+            record(f"latent_decode_B{Bp}", f"B={Bp} keys=4096 H=16 kv_rank=512 rot=64",
+                   lambda: ops.latent_decode(q[..., :r], q[..., r:], cache, 192 ** -0.5, pos=pos, out=o), cache.numel() * 2,
+                   Bp * T * Hn * 2 * (2 * r + rd), like="swa_decode")
+        M, D = 16 * 2048, 2048
+        res, br, w1 = rnd(M, D, dtype=torch.float32), rnd(M, D), rnd(D)
+        record("stream_norm", "rows=32768 D=2048, two outputs", lambda: ops.stream_norm(res, w1, w1, branch=br, mult=0.5), M * D * 14,
+               like="add_rmsnorm")
+        record("add_rmsnorm", "rows=32768 D=2048 (Based)", lambda: ops.add_rmsnorm(br, w1, residual=res, prenorm=True), M * D * 12)
+        cos, sin = RotaryEmbedding(64).tables_f32(8192, torch.device(dev))
+        q, zc, cache = rnd(4, 8192, Hn, 192), rnd(4, 8192, 576), torch.zeros(4, 8192, 576, dtype=torch.bfloat16, device=dev)
+        wn = rnd(512)
+        record("latent_prepare", "B=4 L=8192 H=16 rot=64 kv_rank=512",
+               lambda: ops.latent_prepare_(q, cos, sin, 128, z=zc, norm_weight=wn, cache=cache, kv_rank=512),
+               zc.numel() * 4 + 4 * 8192 * Hn * 64 * 4, like="rotary_qkv_cache")
+        del q, zc, cache, res, br
+        # the Based model's kernels, same timing
+        q, k, v = rnd(B, Hn, L, 16, scale=0.25), rnd(B, Hn, L, 16, scale=0.25), rnd(B, Hn, L, 64)
+        record("linattn_prefill", "B=8 L=8192 H=16 dv=64 (Based)", lambda: ops.linattn_prefill(q, k, v, state_dtype=torch.float32),
+               B * Hn * L * PREFILL_BYTES_PER_TOKEN_HEAD, B * Hn * L * PREFILL_FLOP_PER_TOKEN_HEAD)
+        qd, kd, vd, kvs, ks = [t.to(dev) for t in decode_inputs(256, 1, "cpu", 0)]
+        yd = torch.empty(256, 1, H * DV, dtype=torch.bfloat16, device=dev)
+        record("linattn_decode", "B=256 H=16 dv=64 (Based)", lambda: ops.linattn_decode(qd[0], kd[0], vd[0], kvs, ks, out=yd),
+               DEC_BYTES_PER_UNIT * 256 * H)
+        qkv = rnd(B, L, 3, Hn, 64)
+        record("swa_prefill", "B=8 L=8192 H=16 hd=64 window 64 (Based)", lambda: ops.swa_prefill(qkv[:, :, 0], qkv[:, :, 1], qkv[:, :, 2], 64),
+               B * Hn * L * SWA_BYTES_PER_TOKEN_HEAD, B * Hn * L * SWA_FLOP_PER_TOKEN_HEAD)
+        kvc, q1 = rnd(64, 2048, 2, Hn, 64), rnd(64, 1, 3, Hn, 64)
+        lens = torch.full((64,), 2000, dtype=torch.int32, device=dev)
+        record("swa_decode", "B=64 H=16 hd=64 window 64 (Based)", lambda: ops.swa_decode(q1[:, :, 0], q1[:, :, 1], q1[:, :, 2], kvc, lens, 64),
+               64 * Hn * 65 * 2 * 64 * 2)
+        u, cw3 = rnd(B, L, 2 * 2048), rnd(2048, 3)
+        record("gated_conv", "B=8 L=8192 d_inner=2048 k=3 (Based)", lambda: ops.gated_conv_prefill(u, cw3), B * L * 2048 * 6)
+        st3 = torch.zeros(Bd, 2048, 3, dtype=torch.bfloat16, device=dev)
+        record("gated_conv_step", "B=256 d_inner=2048 k=3 (Based)", lambda: ops.gated_conv_step(u[0, :Bd], st3, cw3), Bd * 2048 * (6 + 12))
+        tab, qkv = RotaryEmbedding(64), rnd(4, 8192, 3, Hn, 64)
+        tab._update_cos_sin_cache(8192, device=qkv.device, dtype=torch.bfloat16)
+        kvc = torch.zeros(4, 8192, 2, Hn, 64, dtype=torch.bfloat16, device=dev)
+        record("rotary_qkv_cache", "B=4 L=8192 H=16 hd=64 (Based)",
+               lambda: ops.rotary_qkv_cache_(qkv, tab._cos_cached, tab._sin_cached, kvc), 4 * 8192 * Hn * 64 * 2 * 7)
+    for name, e in out.items():
+        if e["like"]:
+            e["distance_ratio"] = out[e["like"]]["frac"] / e["frac"]    # how many times further from its roofline
+    return out
+
+
+def run_razesun(args):
+    """The --razesun option: one JSON line with the design's kernels and generation beside the Based model's."""
+    from based_b200 import build_library, ops
+    build_library()
+    peaks = load_peaks()
+    sampler = ClockSampler(0)
+    sampler.start()
+    line = {"bench": "razesun", "data": "synthetic", "dtype": "bf16", "peaks": peaks, "kernels": razesun_kernels(ops, peaks)}
+    torch.cuda.empty_cache()
+    line["generation"] = []
+    for size, B, L, new in (("360m", 16, 2048, 256), ("1b", 8, 4096, 256)):
+        ours = razesun_generation(B, L, new, size)
+        based = generation_bench(B=B, L=L, new_tokens=new, size=size)
+        line["generation"].append({"razesun": ours, "based": based, "prefill_ratio": ours["prefill_tok_per_s"] / based["prefill_tok_per_s"],
+                                   "decode_ratio": based["steps_ms_per_step"] / ours["steps_ms_per_step"]})
+    line["clocks"] = sampler.stop()
+    line["status"] = ops.check_status()
+    print(json.dumps(line), flush=True)
+
+
 def main():
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
@@ -591,6 +779,8 @@ def main():
     ap.add_argument("--sweep-L", type=int, nargs="*", default=None, help="sequence lengths of the prefill sweep")
     ap.add_argument("--regions", type=int, default=25, help="how many times the K-step region is repeated for the "
                     "median / min / max record (the first one is the headline)")
+    ap.add_argument("--razesun", action="store_true",
+                    help="instead of the headline: kernels and generation of the Razesun design beside the Based model's (one GPU)")
     args = ap.parse_args()
     args.warmup = max(args.warmup, 3)
 
@@ -599,6 +789,10 @@ def main():
     local_rank = int(os.environ.get("LOCAL_RANK", "0"))
     if args.impl == "reference":
         run_reference(args, rank, world)
+        return
+
+    if args.razesun:
+        run_razesun(args)
         return
 
     import torch.distributed as dist
