@@ -8,6 +8,7 @@
 // state at its first token from the thread of the group before (a ring of four mbarriers), hands on the state after its
 // last, and only then writes S_t * gelu(y_t): the serial part is one multiply-add per 16 tokens.
 // Warp 16 loads u by TMA (two stages) and issues the MMAs (two accumulator buffers); the weights stay in shared memory.
+// Warp 17 loads the y tiles and stores the output tiles, which replace y's values in place.
 #include <initializer_list>
 #include <mutex>
 
@@ -25,19 +26,17 @@ using namespace tc;
 using bf16 = __nv_bfloat16;
 
 constexpr int TT = 64, GROUPS = 4, TG = TT / GROUPS;   // tokens per tile, groups, tokens per group
-constexpr int NC = 128 * GROUPS, NT = NC + 32;
+constexpr int NC = 128 * GROUPS, NT = NC + 64;
 constexpr uint32_t kWAtom = 128 * 128, kUAtom = TT * 128;   // bytes of 64 columns x 128 (64) rows
 constexpr float kLog2e = 1.4426950408889634f;
 
 struct Params {
-  CUtensorMap mw, mu;            // weights [blocks][2][n][n], u [B][1][L][W]
-  const bf16 *y, *rb, *ib;
+  CUtensorMap mw, mu, my, mo;    // weights [blocks][2][n][n], u [B][1][L][W], y and out [B][blocks][L][n]
+  const bf16 *rb, *ib;
   const float* lam;
   float* state;
-  bf16* out;
   const int32_t* offsets;
   int offset, L, W, n, slices, atoms;
-  Strides2 sy, so;
   unsigned int* status;
 };
 
@@ -46,20 +45,25 @@ __device__ __forceinline__ float rcp(float x) { float r; asm("rcp.approx.ftz.f32
 __device__ __forceinline__ float sqrt_approx(float x) { float r; asm("sqrt.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(x)); return r; }
 
 __global__ void __launch_bounds__(NT, 1) rglru_tc_kernel(const __grid_constant__ Params p) {
-  extern __shared__ uint8_t smem_raw[];
-  uint8_t* smem = smem_raw + ((1024u - (smem_u32(smem_raw) & 1023u)) & 1023u);
+  extern __shared__ __align__(1024) uint8_t smem[];
   const uint32_t sb = smem_u32(smem);
+  if (sb & 1023u) {   // the swizzled tiles need this alignment; there is no room for slack
+    if (threadIdx.x == 0) atomicOr(p.status, 1u << 25);
+    return;
+  }
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
   const int blk = blockIdx.x / p.slices, c0 = (blockIdx.x % p.slices) * 128, b = blockIdx.y;
   const int nt = (p.L + TT - 1) / TT;
-  // shared memory: W_r, W_i (atoms each), u stages, carries, barriers
-  const uint32_t SM_U = 2u * p.atoms * kWAtom, SM_C = SM_U + 2u * p.atoms * kUAtom, SM_BAR = SM_C + GROUPS * 128 * 4;
-  const uint32_t B_W = sb + SM_BAR, B_FULL = B_W + 8, B_D = B_FULL + 16, B_EMPTY = B_D + 16, B_CARRY = B_EMPTY + 16;
-  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(smem + SM_BAR + 8 * (7 + GROUPS));
+  // shared memory: W_r, W_i (atoms each), u stages, y stages (two 64-channel atoms each), carries, barriers
+  const uint32_t SM_U = 2u * p.atoms * kWAtom, SM_Y = SM_U + 2u * p.atoms * kUAtom, SM_C = SM_Y + 4u * kUAtom,
+                 SM_BAR = SM_C + GROUPS * 128 * 4;
+  const uint32_t B_W = sb + SM_BAR, B_FULL = B_W + 8, B_D = B_FULL + 16, B_EMPTY = B_D + 16, B_Y = B_EMPTY + 16,
+                 B_OUT = B_Y + 16, B_CARRY = B_OUT + 16;
+  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(smem + SM_BAR + 8 * (11 + GROUPS));
   volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_slot + 1);
   if (tid == 0) {
     mbar_init(B_W, 1);
-    for (int i = 0; i < 2; ++i) { mbar_init(B_FULL + 8 * i, 1); mbar_init(B_D + 8 * i, 1); mbar_init(B_EMPTY + 8 * i, NC); }
+    for (int i = 0; i < 2; ++i) { mbar_init(B_FULL + 8 * i, 1); mbar_init(B_D + 8 * i, 1); mbar_init(B_EMPTY + 8 * i, NC); mbar_init(B_Y + 8 * i, 1); mbar_init(B_OUT + 8 * i, NC); }
     for (int i = 0; i < GROUPS; ++i) mbar_init(B_CARRY + 8 * i, 128);
     *abort_flag = 0;
     fence_mbar_init();
@@ -95,16 +99,16 @@ __global__ void __launch_bounds__(NT, 1) rglru_tc_kernel(const __grid_constant__
       const int x = t & 1;
       mbar_wait_bounded(B_FULL + 8 * x, (t >> 1) & 1, abort_flag, p.status, 1u << 19);
       fence_after_sync();
+#pragma unroll
       for (int m = 0; m < 2; ++m) {
-        uint32_t acc = 0;
         for (int a = 0; a < p.atoms; ++a) {
+          // a K step of 16 advances both start addresses by 32 bytes, 2 in descriptor units
+          const uint64_t da = make_smem_desc_sw128(sb + (m * p.atoms + a) * kWAtom, 16, 1024);
+          const uint64_t db = make_smem_desc_sw128(sb + SM_U + (x * p.atoms + a) * kUAtom, 16, 1024);
           const int ks = min(64, p.n - 64 * a) >> 4;
-          for (int k = 0; k < ks; ++k) {
-            const uint64_t da = make_smem_desc_sw128(sb + (m * p.atoms + a) * kWAtom + k * 32, 16, 1024);
-            const uint64_t db = make_smem_desc_sw128(sb + SM_U + (x * p.atoms + a) * kUAtom + k * 32, 16, 1024);
-            if (leader) mma_ss(tmem_u + 128 * x + 64 * m, da, db, idesc, acc);
-            acc = 1;
-          }
+#pragma unroll
+          for (int k = 0; k < 4; ++k)
+            if (k < ks && leader) mma_ss(tmem_u + 128 * x + 64 * m, da + 2 * k, db + 2 * k, idesc, (a > 0 || k > 0) ? 1u : 0u);
         }
       }
       if (leader) mma_commit(B_D + 8 * x);
@@ -114,6 +118,25 @@ __global__ void __launch_bounds__(NT, 1) rglru_tc_kernel(const __grid_constant__
         load(t + 1);
       }
       __syncwarp();
+    }
+  } else if (warp == NC / 32 + 1) {
+    if (lane == 0) {
+      const int na = min(128, p.n - c0) > 64 ? 2 : 1;
+      auto load_y = [&](int t) {
+        tma::mbar_expect_tx(B_Y + 8 * (t & 1), (uint32_t)na * kUAtom);
+        for (int a = 0; a < na; ++a)
+          tma::load_4d(sb + SM_Y + ((t & 1) * 2 + a) * kUAtom, &p.my, B_Y + 8 * (t & 1), c0 + 64 * a, t * TT, blk, b);
+      };
+      load_y(0);
+      if (nt > 1) load_y(1);
+      for (int t = 0; t < nt; ++t) {
+        mbar_wait_bounded<false>(B_OUT + 8 * (t & 1), (t >> 1) & 1, abort_flag, p.status, 1u << 23);
+        for (int a = 0; a < na; ++a) tma::store_4d(&p.mo, sb + SM_Y + ((t & 1) * 2 + a) * kUAtom, c0 + 64 * a, t * TT, blk, b);
+        bulk_commit();
+        bulk_wait_read_all();
+        if (t + 2 < nt) load_y(t + 2);
+      }
+      bulk_wait_all();
     }
   } else {
     const int grp = warp >> 2, ch = tid & 127;
@@ -126,18 +149,14 @@ __global__ void __launch_bounds__(NT, 1) rglru_tc_kernel(const __grid_constant__
     float* carry = reinterpret_cast<float*>(smem + SM_C);
     const uint32_t my_carry = B_CARRY + 8 * grp, from = B_CARRY + 8 * ((grp + GROUPS - 1) % GROUPS);
     const float* carry_in = carry + ((grp + GROUPS - 1) % GROUPS) * 128 + ch;
-    const bf16* y = p.y + b * p.sy.b + chan;
-    bf16* out = p.out + b * p.so.b + chan;
+    uint8_t* ycol = smem + SM_Y + (ch >> 6) * kUAtom + (ch & 7) * 2;
+    const int ychunk = (ch & 63) >> 3;
     const uint8_t* ucol = smem + SM_U + ((c0 + ch) >> 6) * kUAtom + (ch & 7) * 2;   // this channel's column of a stage
     const int chunk = ((c0 + ch) & 63) >> 3;
     float S0 = 0.f;
     if (grp == 0 && live && seq::position0(p.offsets, p.offset, b) > 0) S0 = p.state[(int64_t)b * p.W + chan];
     for (int t = 0; t < nt; ++t) {
       const int x = t & 1, tok0 = t * TT + t0g;
-      bf16 yv[TG];
-#pragma unroll
-      for (int i = 0; i < TG; ++i)
-        if (live && tok0 + i < p.L) yv[i] = y[(int64_t)(tok0 + i) * p.sy.h];
       mbar_wait_bounded(B_D + 8 * x, (t >> 1) & 1, abort_flag, p.status, 1u << 21);
       fence_after_sync();
       uint32_t gr[TG], gi[TG];
@@ -179,13 +198,17 @@ __global__ void __launch_bounds__(NT, 1) rglru_tc_kernel(const __grid_constant__
       const float end = fmaf(pr, S0, sr);
       carry[grp * 128 + ch] = end;
       mbar_arrive(my_carry);
-      if (live) {
+      mbar_wait_bounded(B_Y + 8 * x, (t >> 1) & 1, abort_flag, p.status, 1u << 24);
+      uint8_t* ys = ycol + x * 2 * kUAtom;
 #pragma unroll
-        for (int i = 0; i < TG; ++i)
-          if (tok0 + i < p.L)
-            out[(int64_t)(tok0 + i) * p.so.h] = __float2bfloat16_rn(fmaf(P[i], S0, s[i]) * seq::gelu_tanh_t<bf16>(__bfloat162float(yv[i])));
-        if (grp == GROUPS - 1 && t == nt - 1) p.state[(int64_t)b * p.W + chan] = end;
+      for (int i = 0; i < TG; ++i) {   // rows past the sequence and channels past the block are clipped by the store
+        const int row = t0g + i;
+        bf16* e = reinterpret_cast<bf16*>(ys + row * 128 + ((ychunk ^ (row & 7)) << 4));
+        *e = __float2bfloat16_rn(fmaf(P[i], S0, s[i]) * seq::gelu_tanh_t<bf16>(__bfloat162float(*e)));
       }
+      fence_proxy_async();
+      mbar_arrive(B_OUT + 8 * x);
+      if (live && grp == GROUPS - 1 && t == nt - 1) p.state[(int64_t)b * p.W + chan] = end;
     }
   }
   __syncwarp();
@@ -230,17 +253,21 @@ int launch_rglru_tc(const void* u, const void* y, const void* w, const void* rb,
     cache.put(key, *m);
     return 0;
   };
+  for (const Strides2& st : {sy, so})
+    if (st.h % 8 != 0 || st.h <= 0 || (B > 1 && (st.b % 8 != 0 || st.b <= 0))) return BASED_ERR_IMPL;
+  if (!aligned16(y) || !aligned16(out)) return BASED_ERR_IMPL;
   const int64_t nn = (int64_t)n * n;
   if (get_map(&p.mw, w, n, n, 2, blocks, n, nn, 2 * nn, 128) ||
-      get_map(&p.mu, u, W, L, 1, B, L == 1 ? 8 : su.h, 8, B == 1 ? 8 : su.b, TT))
+      get_map(&p.mu, u, W, L, 1, B, L == 1 ? 8 : su.h, 8, B == 1 ? 8 : su.b, TT) ||
+      get_map(&p.my, y, n, L, blocks, B, L == 1 ? 8 : sy.h, n, B == 1 ? 8 : sy.b, TT) ||
+      get_map(&p.mo, out, n, L, blocks, B, L == 1 ? 8 : so.h, n, B == 1 ? 8 : so.b, TT))
     return BASED_ERR_IMPL;
-  p.y = static_cast<const bf16*>(y);
   p.rb = static_cast<const bf16*>(rb);
   p.ib = static_cast<const bf16*>(ib);
   p.lam = lam; p.state = state;
-  p.out = static_cast<bf16*>(out);
-  p.offsets = offsets; p.offset = offset; p.L = L; p.W = W; p.n = n; p.sy = sy; p.so = so;
-  const int smem = 2 * p.atoms * (int)(kWAtom + kUAtom) + GROUPS * 128 * 4 + 8 * (7 + GROUPS) + 16 + 1024;
+  p.offsets = offsets; p.offset = offset; p.L = L; p.W = W; p.n = n;
+  const int smem = 2 * p.atoms * (int)(kWAtom + kUAtom) + 4 * (int)kUAtom + GROUPS * 128 * 4 + 8 * (11 + GROUPS) + 16;
+  if (smem > 227 * 1024) return BASED_ERR_IMPL;
   {
     constexpr int kMaxDevices = 64;
     static std::mutex mu;
