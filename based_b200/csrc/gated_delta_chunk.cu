@@ -40,7 +40,7 @@ constexpr int LT = C + 8;           // row stride of the [64, 64] operand tiles
 constexpr int LI = 20;              // row stride of the diagonal blocks, stored transposed
 constexpr int kConsumers = 8, kHelpers = 8;
 constexpr int NT = 32 * (kConsumers + kHelpers), HT = 32 * kHelpers;
-constexpr float kUnitEps = 1e-6f;
+constexpr float kUnitEps = 1e-6f, kLog2e = 1.4426950408889634f;
 
 struct Params {
   const bf16 *q, *k, *v, *z, *norm_w;
@@ -70,7 +70,7 @@ struct Layout {                     // byte offsets in shared memory
     total = bars + 64;
   }
 };
-// gates of one chunk, C floats each; chunk c's sit in slot c mod 3
+// gates of one chunk, C floats each (logarithms to base 2); chunk c's sit in slot c mod 3
 enum { G_CUM = 0, G_BETA, G_RK, G_RQ, G_EGK, G_EGQ, G_W, G_COL, G_TOT, G_N };
 
 __device__ __forceinline__ void ldsm4(uint32_t (&r)[4], uint32_t a) {
@@ -95,6 +95,7 @@ __device__ __forceinline__ void split_a(const float (&t0)[4], const float (&t1)[
   split(t1[0], t1[1], hi[2], lo[2]);
   split(t1[2], t1[3], hi[3], lo[3]);
 }
+__device__ __forceinline__ float ex2(float x) { float r; asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(x)); return r; }
 __device__ __forceinline__ void bar_sync(int id, int n) { asm volatile("bar.sync %0, %1;\n" ::"r"(id), "r"(n) : "memory"); }
 template <int R> __device__ __forceinline__ void reg_inc() { asm volatile("setmaxnreg.inc.sync.aligned.u32 %0;\n" ::"n"(R)); }
 template <int R> __device__ __forceinline__ void reg_dec() { asm volatile("setmaxnreg.dec.sync.aligned.u32 %0;\n" ::"n"(R)); }
@@ -139,7 +140,7 @@ __global__ void __launch_bounds__(NT, 1) delta_chunk_kernel(const Params p) {
         const int l = c * C + 2 * lane + e;
         if (l < p.L) {
           const int64_t gi = b * p.sg.b + (int64_t)l * p.sg.h + h;
-          lg[e] = -A * seq::softplus_acc(p.a[gi] + dt);
+          lg[e] = -A * kLog2e * seq::softplus_acc(p.a[gi] + dt);
           be[e] = seq::sigmoid_acc(p.b[gi]);
         }
       }
@@ -214,12 +215,12 @@ __global__ void __launch_bounds__(NT, 1) delta_chunk_kernel(const Params p) {
           if (is_q) {
             const float rq = r * rsqrtf((float)d);
             gt[G_RQ * C + i] = rq;
-            gt[G_EGQ * C + i] = expf(G) * rq;
+            gt[G_EGQ * C + i] = ex2(G) * rq;
           } else {
             gt[G_RK * C + i] = r;
-            gt[G_EGK * C + i] = expf(G) * r;
-            gt[G_W * C + i] = expf(gt[G_TOT * C] - G) * r;
-            gt[G_COL * C + i] = expf(gt[G_CUM * C + (i | 15)] - G) * r;   // decay from here to the end of the 16-block
+            gt[G_EGK * C + i] = ex2(G) * r;
+            gt[G_W * C + i] = ex2(gt[G_TOT * C] - G) * r;
+            gt[G_COL * C + i] = ex2(gt[G_CUM * C + (i | 15)] - G) * r;   // decay from here to the end of the 16-block
           }
         }
       }
@@ -252,7 +253,7 @@ __global__ void __launch_bounds__(NT, 1) delta_chunk_kernel(const Params p) {
           const float Gi = gt[G_CUM * C + i];
           float fk = gt[G_BETA * C + i] * gt[G_RK * C + i], fq = gt[G_RQ * C + i];
           if (!diag) {
-            const float ei = expf(Gi - end);
+            const float ei = ex2(Gi - end);
             fk *= -ei;
             fq *= ei;
           }
@@ -262,7 +263,7 @@ __global__ void __launch_bounds__(NT, 1) delta_chunk_kernel(const Params p) {
             float a0 = kk2[nt][2 * half] * fk, a1 = kk2[nt][2 * half + 1] * fk, p0 = qk2[nt][2 * half] * fq, p1 = qk2[nt][2 * half + 1] * fq;
             if (diag) {
               const float2 gj = *reinterpret_cast<const float2*>(gt + G_CUM * C + j), rk = *reinterpret_cast<const float2*>(gt + G_RK * C + j);
-              const float e0 = jj <= ii ? expf(Gi - gj.x) * rk.x : 0.f, e1 = jj + 1 <= ii ? expf(Gi - gj.y) * rk.y : 0.f;
+              const float e0 = jj <= ii ? ex2(Gi - gj.x) * rk.x : 0.f, e1 = jj + 1 <= ii ? ex2(Gi - gj.y) * rk.y : 0.f;
               inv[(bi * 16 + jj) * LI + ii] = jj < ii ? a0 * e0 : 0.f;
               inv[(bi * 16 + jj + 1) * LI + ii] = jj + 1 < ii ? a1 * e1 : 0.f;
               p0 *= e0;
@@ -462,6 +463,13 @@ __global__ void __launch_bounds__(NT, 1) delta_chunk_kernel(const Params p) {
             o[n][0] *= eq.x; o[n][1] *= eq.y; o[n][2] *= eq.x; o[n][3] *= eq.y;
           }
         }
+        // S <- e^{G_C} S + sum_j (w_j u_j) k_j: decayed here, each block's sum added as soon as its u is known, so that
+        // these products fill the gaps of the block-by-block solution
+        const float gc = ex2(gt[G_TOT * C]);
+#pragma unroll
+        for (int n = 0; n < 2 * DK; ++n)
+#pragma unroll
+          for (int e = 0; e < 4; ++e) s[n][e] *= gc;
         // blocks of 16 tokens: u_b = T_b (residual), then its part in the later residuals and in the read-out
 #pragma unroll
         for (int bb = 0; bb < 4; ++bb) {
@@ -495,29 +503,11 @@ __global__ void __launch_bounds__(NT, 1) delta_chunk_kernel(const Params p) {
             mma(o[2 * np], fh, mh[0], mh[1]);
             mma(o[2 * np + 1], fh, mh[2], mh[3]);
           }
-        }
-        bar_sync(2, 32 * active);   // every consumer is through with T and P: the stage may overwrite them
-        {
-          float* st = reinterpret_cast<float*>(sm + lay.R + buf * lay.region) + 16 * warp + g;
-#pragma unroll
-          for (int n = 0; n < 8; ++n)
-#pragma unroll
-            for (int e = 0; e < 4; ++e) st[(8 * n + 2 * t4 + (e & 1)) * lay.ldo + (e >> 1) * 8] = o[n][e];
-        }
-        // S <- e^{G_C} S + sum_j (w_j u_j) k_j
-        const float gc = expf(gt[G_TOT * C]);
-#pragma unroll
-        for (int n = 0; n < 2 * DK; ++n)
-#pragma unroll
-          for (int e = 0; e < 4; ++e) s[n][e] *= gc;
-#pragma unroll
-        for (int bb = 0; bb < 4; ++bb) {
 #pragma unroll
           for (int q = 0; q < 2; ++q) {
             const float2 w = *reinterpret_cast<const float2*>(gt + G_W * C + 16 * bb + 8 * q + 2 * t4);
             x[2 * bb + q][0] *= w.x; x[2 * bb + q][1] *= w.y; x[2 * bb + q][2] *= w.x; x[2 * bb + q][3] *= w.y;
           }
-          uint32_t fh[4], fl[4];
           split_a(x[2 * bb], x[2 * bb + 1], fh, fl);
 #pragma unroll
           for (int np = 0; np < DK; ++np) {
@@ -528,6 +518,14 @@ __global__ void __launch_bounds__(NT, 1) delta_chunk_kernel(const Params p) {
             mma(s[2 * np], fh, fb[0], fb[1]);
             mma(s[2 * np + 1], fh, fb[2], fb[3]);
           }
+        }
+        bar_sync(2, 32 * active);   // every consumer is through with T and P: the stage may overwrite them
+        {
+          float* st = reinterpret_cast<float*>(sm + lay.R + buf * lay.region) + 16 * warp + g;
+#pragma unroll
+          for (int n = 0; n < 8; ++n)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) st[(8 * n + 2 * t4 + (e & 1)) * lay.ldo + (e >> 1) * 8] = o[n][e];
         }
         mbar_arrive(DONE + 8 * buf);
       }

@@ -622,7 +622,8 @@ def razesun_generation(B, L, new_tokens, size):
     """Prompt pass and CUDA-graph decode of a Razesun stack, the same measurement as generation_bench."""
     model = random_razesun(size)
     ids = torch.randint(0, model.config.vocab_size, (B, L), device="cuda")
-    model.generate(ids, max_new_tokens=8, cg=True)
+    for _ in range(2):   # at full size: allocator, cuBLAS heuristics
+        model.generate(ids, max_new_tokens=new_tokens, cg=True)
     t = {}
     model.generate(ids, max_new_tokens=new_tokens, cg=True, timings=t)
     res = {"model": f"razesun-{size} (random init)", "params": sum({p.data_ptr(): p.numel() for p in model.parameters()}.values()),
