@@ -37,9 +37,9 @@ const char* based_error_string(int code) {
 
 int based_read_status(unsigned int* out, int reset) {
   unsigned int a = 0, b = 0, c = 0, d = 0, e = 0, f = 0;
-  int rc = read_tc_status(&a, reset);
-  if (rc == 0) rc = read_tc_status_swa(&b, reset);
-  if (rc == 0) rc = read_tp_status(&c, reset);
+  int rc = read_tc_status ? read_tc_status(&a, reset) : 0;
+  if (rc == 0 && read_tc_status_swa) rc = read_tc_status_swa(&b, reset);
+  if (rc == 0 && read_tp_status) rc = read_tp_status(&c, reset);
   if (rc == 0) rc = read_tc_status_latent(&d, reset);
   if (rc == 0) rc = read_tc_status_delta(&e, reset);
   if (rc == 0) rc = read_tc_status_rglru(&f, reset);
@@ -95,6 +95,7 @@ int based_linattn_prefill(const void* q, const void* k, const void* v, void* y, 
   if (autosel) impl = (io_dtype == BASED_BF16) ? BASED_IMPL_TCGEN05 : BASED_IMPL_SIMT;
   if (impl == BASED_IMPL_TCGEN05) {
     if (io_dtype != BASED_BF16) return BASED_ERR_IMPL;
+    if (!launch_linattn_prefill_tc) return BASED_ERR_IMPL;
     const int rc = launch_linattn_prefill_tc(q, k, v, y, kv_state, k_state, B, H, L, dv, s3(q_strides),
                                              s3(k_strides), s3(v_strides), s3(y_strides), state_dtype, eps, 1,
                                              nullptr, 0, st);
@@ -102,17 +103,20 @@ int based_linattn_prefill(const void* q, const void* k, const void* v, void* y, 
     impl = BASED_IMPL_SIMT;
   }
   if (impl != BASED_IMPL_SIMT) return BASED_ERR_IMPL;
+  if (!launch_linattn_prefill_simt) return BASED_ERR_IMPL;
   return launch_linattn_prefill_simt(q, k, v, y, kv_state, k_state, B, H, L, dv, s3(q_strides), s3(k_strides),
                                      s3(v_strides), s3(y_strides), io_dtype, state_dtype, eps, st);
 }
 
 int based_linattn_prefill_segments(int B, int H, int L) {
   if (B <= 0 || H <= 0 || L <= 0) return 1;
+  if (!linattn_prefill_tc_auto_segments) return 1;
   return linattn_prefill_tc_auto_segments(B, H, L);
 }
 
 size_t based_linattn_prefill_scratch_bytes(int B, int H, int L, int dv, int nseg) {
   if (B <= 0 || H <= 0 || L <= 0 || dv <= 0 || nseg <= 1) return 0;
+  if (!linattn_prefill_tc_scratch_bytes) return 0;
   return linattn_prefill_tc_scratch_bytes(B, H, L, dv, nseg);
 }
 
@@ -126,6 +130,7 @@ int based_linattn_prefill_split(const void* q, const void* k, const void* v, voi
   const int pre = prefill_preamble(q, k, v, y, kv_state, k_state, B, H, L, d, dv, q_strides, k_strides, v_strides,
                                    y_strides, BASED_BF16, state_dtype, st);
   if (pre != 0) return pre == kDone ? BASED_OK : pre;
+  if (!launch_linattn_prefill_tc) return BASED_ERR_IMPL;
   return launch_linattn_prefill_tc(q, k, v, y, kv_state, k_state, B, H, L, dv, s3(q_strides), s3(k_strides),
                                    s3(v_strides), s3(y_strides), state_dtype, eps, nseg, scratch, scratch_bytes, st);
 }
@@ -140,6 +145,7 @@ int based_linattn_prefill_split_static(const void* q, const void* k, const void*
   const int pre = prefill_preamble(q, k, v, y, kv_state, k_state, B, H, L, d, dv, q_strides, k_strides, v_strides,
                                    y_strides, BASED_BF16, state_dtype, st);
   if (pre != 0) return pre == kDone ? BASED_OK : pre;
+  if (!launch_linattn_prefill_tc_static) return BASED_ERR_IMPL;
   return launch_linattn_prefill_tc_static(q, k, v, y, kv_state, k_state, B, H, L, dv, s3(q_strides), s3(k_strides),
                                           s3(v_strides), s3(y_strides), state_dtype, eps, nseg, st);
 }
@@ -157,6 +163,7 @@ int based_linattn_decode(const void* q, const void* k, const void* v, void* y, v
   if ((int64_t)B * H > 2147483647LL) return BASED_ERR_TOO_LARGE;
   if (!aligned16(kv_state)) return BASED_ERR_ALIGN;
   if (B == 0 || H == 0) return BASED_OK;
+  if (!launch_linattn_decode) return BASED_ERR_IMPL;
   return launch_linattn_decode(q, k, v, y, kv_state, k_state, B, H, dv, s2(q_strides), s2(k_strides),
                                s2(v_strides), s2(y_strides), io_dtype, state_dtype, eps,
                                static_cast<cudaStream_t>(stream));
@@ -176,12 +183,14 @@ int based_swa_prefill(const void* q, const void* k, const void* v, void* o, int 
   if (autosel) impl = (io_dtype == BASED_BF16) ? BASED_IMPL_TCGEN05 : BASED_IMPL_SIMT;
   if (impl == BASED_IMPL_TCGEN05) {
     if (io_dtype != BASED_BF16) return BASED_ERR_IMPL;
+    if (!launch_swa_prefill_tc) return BASED_ERR_IMPL;
     const int rc = launch_swa_prefill_tc(q, k, v, o, B, L, H, hd, s3_blh(q_strides), s3_blh(k_strides), s3_blh(v_strides),
                                          s3_blh(o_strides), window_left, softmax_scale, st);
     if (!(autosel && rc == BASED_ERR_IMPL)) return rc;
     impl = BASED_IMPL_SIMT;
   }
   if (impl != BASED_IMPL_SIMT) return BASED_ERR_IMPL;
+  if (!launch_swa_prefill_simt) return BASED_ERR_IMPL;
   return launch_swa_prefill_simt(q, k, v, o, B, L, H, hd, s3_blh(q_strides), s3_blh(k_strides), s3_blh(v_strides),
                                  s3_blh(o_strides), window_left, softmax_scale, io_dtype, st);
 }
@@ -194,6 +203,7 @@ int based_rotary_apply(void* x, int B, int L, int H, int hd, const int64_t x_str
   if (B < 0 || L < 0 || H < 0 || hd <= 0 || rotary_dim <= 0 || rotary_dim > hd || rotary_dim % 2 != 0 ||
       seqlen_offset_scalar < 0)
     return BASED_ERR_SHAPE;
+  if (!launch_rotary) return BASED_ERR_IMPL;
   return launch_rotary(x, B, L, H, s3_blh(x_strides), rotary_cos, rotary_sin, rotary_dim, seqlen_offsets,
                        seqlen_offset_scalar, io_dtype, static_cast<cudaStream_t>(stream));
 }
@@ -212,6 +222,7 @@ int based_swa_decode(const void* q, const void* k_new, const void* v_new, void* 
   if (rotary_cos && (rotary_dim <= 0 || rotary_dim > hd || rotary_dim % 2 != 0)) return BASED_ERR_SHAPE;
   if (!cache_seqlens && (cache_seqlen_scalar < 0 || cache_seqlen_scalar >= max_seqlen)) return BASED_ERR_SHAPE;
   if (B == 0 || H == 0) return BASED_OK;
+  if (!launch_swa_decode) return BASED_ERR_IMPL;
   return launch_swa_decode(q, k_new, v_new, o, kv_cache, cache_seqlens, cache_seqlen_scalar, rotary_cos, rotary_sin,
                            rotary_dim, B, H, hd, max_seqlen, s2(q_strides), s2(k_strides), s2(v_strides),
                            s2(o_strides), window_left, softmax_scale, io_dtype,
@@ -231,6 +242,7 @@ int based_gated_conv_prefill(const void* u1, const void* u2, void* v, void* stat
     if (state) return (int)cudaMemsetAsync(state, 0, (size_t)B * di * k * dtype_size(io_dtype), st);
     return BASED_OK;
   }
+  if (!launch_gated_conv_prefill) return BASED_ERR_IMPL;
   return launch_gated_conv_prefill(u1, u2, v, state, weight, bias, B, L, di, k, s2(u1_strides), s2(u2_strides),
                                    s2(v_strides), io_dtype, w_dtype, st);
 }
@@ -243,6 +255,7 @@ int based_gated_conv_step(const void* u1, const void* u2, void* y, void* state, 
   if (B < 0 || di <= 0 || k < 1 || k > 4) return BASED_ERR_SHAPE;
   if ((int64_t)B * di > 2147483647LL) return BASED_ERR_TOO_LARGE;
   if (B == 0) return BASED_OK;
+  if (!launch_gated_conv_step) return BASED_ERR_IMPL;
   return launch_gated_conv_step(u1, u2, y, state, weight, bias, B, di, k, u1_batch_stride, u2_batch_stride,
                                 y_batch_stride, io_dtype, w_dtype, static_cast<cudaStream_t>(stream));
 }
@@ -291,12 +304,14 @@ int based_rotary_qkv_cache(void* qkv, int B, int L, int H, int hd, const int64_t
                            const int64_t cache_strides[2], void* stream) {
   if (!qkv || !qkv_strides || !rotary_cos || !rotary_sin || !kv_cache || !cache_strides) return BASED_ERR_NULL;
   if (B < 0 || L < 0 || H < 0 || hd < 16 || hd > 256) return BASED_ERR_SHAPE;
+  if (!launch_rotary_qkv_cache) return BASED_ERR_IMPL;
   return launch_rotary_qkv_cache(qkv, B, L, H, hd, qkv_strides[0], qkv_strides[1], qkv_strides[2], qkv_strides[3],
                                  rotary_cos, rotary_sin, kv_cache, cache_strides[0], cache_strides[1],
                                  static_cast<cudaStream_t>(stream));
 }
 
 size_t based_tp_outproj_workspace_bytes(int world, int max_rows, int N) {
+  if (!tp_outproj_workspace_bytes) return 0;
   return tp_outproj_workspace_bytes(world, max_rows, N);
 }
 
@@ -318,6 +333,7 @@ int based_tp_outproj_allreduce(const void* x, const void* w, const void* bias, v
   const void* xs[1] = {x};
   const void* ws[1] = {w};
   void* os[1] = {out};
+  if (!launch_tp_outproj_allreduce) return BASED_ERR_IMPL;
   return launch_tp_outproj_allreduce(xs, ws, bias, os, workspaces, M, N, K, x_row_stride, out_row_stride, max_rows, rank,
                                      world, 0, static_cast<cudaStream_t>(stream));
 }
@@ -326,6 +342,7 @@ int based_tp_outproj_allreduce_emulated(const void* const* x, const void* const*
                                         int M, int N, int K, int64_t x_row_stride, int64_t out_row_stride,
                                         void* const* workspaces, int max_rows, int world, void* stream) {
   if (!x || !w || !out || !workspaces) return BASED_ERR_NULL;
+  if (!launch_tp_outproj_allreduce) return BASED_ERR_IMPL;
   return launch_tp_outproj_allreduce(x, w, bias, out, workspaces, M, N, K, x_row_stride, out_row_stride, max_rows, 0,
                                      world, 1, static_cast<cudaStream_t>(stream));
 }

@@ -52,29 +52,31 @@ __device__ __forceinline__ float warp_max(float v) {
 inline bool aligned16(const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15u) == 0; }
 
 // Launchers implemented one per .cu file; all return a cudaError_t-compatible int (0 = ok).
-int launch_linattn_decode(const void* q, const void* k, const void* v, void* y, void* kv_state, void* k_state,
+// BASED_WEAK: not in every build of the library (a part without a kernel leaves its launcher null; capi.cu checks).
+#define BASED_WEAK __attribute__((weak))
+BASED_WEAK int launch_linattn_decode(const void* q, const void* k, const void* v, void* y, void* kv_state, void* k_state,
                           int B, int H, int dv, Strides2 sq, Strides2 sk, Strides2 sv, Strides2 sy,
                           int io_dtype, int state_dtype, float eps, cudaStream_t stream);
 
-int launch_linattn_prefill_simt(const void* q, const void* k, const void* v, void* y, void* kv_state, void* k_state,
+BASED_WEAK int launch_linattn_prefill_simt(const void* q, const void* k, const void* v, void* y, void* kv_state, void* k_state,
                                 int B, int H, int L, int dv, Strides3 sq, Strides3 sk, Strides3 sv, Strides3 sy,
                                 int io_dtype, int state_dtype, float eps, cudaStream_t stream);
 
-int launch_linattn_prefill_tc(const void* q, const void* k, const void* v, void* y, void* kv_state, void* k_state,
+BASED_WEAK int launch_linattn_prefill_tc(const void* q, const void* k, const void* v, void* y, void* kv_state, void* k_state,
                               int B, int H, int L, int dv, Strides3 sq, Strides3 sk, Strides3 sv, Strides3 sy,
                               int state_dtype, float eps, int nseg, void* scratch, size_t scratch_bytes,
                               cudaStream_t stream);
-int launch_linattn_prefill_tc_static(const void* q, const void* k, const void* v, void* y, void* kv_state,
+BASED_WEAK int launch_linattn_prefill_tc_static(const void* q, const void* k, const void* v, void* y, void* kv_state,
                                      void* k_state, int B, int H, int L, int dv, Strides3 sq, Strides3 sk,
                                      Strides3 sv, Strides3 sy, int state_dtype, float eps, int nseg,
                                      cudaStream_t stream);
-int linattn_prefill_tc_auto_segments(int B, int H, int L);
-size_t linattn_prefill_tc_scratch_bytes(int B, int H, int L, int dv, int nseg);
+BASED_WEAK int linattn_prefill_tc_auto_segments(int B, int H, int L);
+BASED_WEAK size_t linattn_prefill_tc_scratch_bytes(int B, int H, int L, int dv, int nseg);
 
-int launch_gated_conv_prefill(const void* u1, const void* u2, void* v, void* state, const void* weight,
+BASED_WEAK int launch_gated_conv_prefill(const void* u1, const void* u2, void* v, void* state, const void* weight,
                               const void* bias, int B, int L, int di, int k, Strides2 s1, Strides2 s2, Strides2 sv,
                               int io_dtype, int w_dtype, cudaStream_t stream);
-int launch_gated_conv_step(const void* u1, const void* u2, void* y, void* state, const void* weight, const void* bias,
+BASED_WEAK int launch_gated_conv_step(const void* u1, const void* u2, void* y, void* state, const void* weight, const void* bias,
                            int B, int di, int k, int64_t s1, int64_t s2, int64_t sy, int io_dtype, int w_dtype,
                            cudaStream_t stream);
 
@@ -84,34 +86,34 @@ int launch_add_rmsnorm(const void* x, const void* residual, const void* weight, 
 int launch_gated_act(const void* y, const void* gate, void* out, int64_t M, int F, int64_t sy, int64_t sg, int64_t so,
                      int act, int io_dtype, cudaStream_t stream);
 
-int launch_rotary_qkv_cache(void* qkv, int B, int L, int H, int hd, int64_t sb, int64_t sl, int64_t s3, int64_t sh,
+BASED_WEAK int launch_rotary_qkv_cache(void* qkv, int B, int L, int H, int hd, int64_t sb, int64_t sl, int64_t s3, int64_t sh,
                             const void* rcos, const void* rsin, void* cache, int64_t cb, int64_t cl,
                             cudaStream_t stream);
 int launch_decode_linear(const void* x, const void* w, const void* bias, void* out, int M, int N, int K, int64_t sx,
                          int64_t so, int epilogue, int act, void* conv_state, const void* conv_weight,
                          const void* conv_bias, int conv_k, int conv_w_dtype, cudaStream_t stream);
 
-int launch_tp_outproj_allreduce(const void* const* x, const void* const* w, const void* bias, void* const* out,
+BASED_WEAK int launch_tp_outproj_allreduce(const void* const* x, const void* const* w, const void* bias, void* const* out,
                                 void* const* workspaces, int M, int N, int K, int64_t sx, int64_t so, int Mmax,
                                 int rank, int world, int emulate, cudaStream_t stream);
-size_t tp_outproj_workspace_bytes(int world, int Mmax, int N);
-int read_tp_status(unsigned int* out, int reset);      // fused output projection + all-reduce
+BASED_WEAK size_t tp_outproj_workspace_bytes(int world, int Mmax, int N);
+BASED_WEAK int read_tp_status(unsigned int* out, int reset);      // fused output projection + all-reduce
 
-int read_tc_status(unsigned int* out, int reset);      // linear-attention prefill kernel
-int read_tc_status_swa(unsigned int* out, int reset);  // sliding-window prefill kernel
+BASED_WEAK int read_tc_status(unsigned int* out, int reset);      // linear-attention prefill kernel
+BASED_WEAK int read_tc_status_swa(unsigned int* out, int reset);  // sliding-window prefill kernel
 
-int launch_swa_prefill_simt(const void* q, const void* k, const void* v, void* o, int B, int L, int H, int hd,
+BASED_WEAK int launch_swa_prefill_simt(const void* q, const void* k, const void* v, void* o, int B, int L, int H, int hd,
                             Strides3 sq, Strides3 sk, Strides3 sv, Strides3 so, int window_left, float scale,
                             int io_dtype, cudaStream_t stream);
 
-int launch_swa_prefill_tc(const void* q, const void* k, const void* v, void* o, int B, int L, int H, int hd,
+BASED_WEAK int launch_swa_prefill_tc(const void* q, const void* k, const void* v, void* o, int B, int L, int H, int hd,
                           Strides3 sq, Strides3 sk, Strides3 sv, Strides3 so, int window_left, float scale,
                           cudaStream_t stream);
 
-int launch_rotary(void* x, int B, int L, int H, Strides3 sx, const void* rcos, const void* rsin, int rotary_dim,
+BASED_WEAK int launch_rotary(void* x, int B, int L, int H, Strides3 sx, const void* rcos, const void* rsin, int rotary_dim,
                   const int32_t* offsets, int offset_scalar, int io_dtype, cudaStream_t stream);
 
-int launch_swa_decode(const void* q, const void* k_new, const void* v_new, void* o, void* kv_cache,
+BASED_WEAK int launch_swa_decode(const void* q, const void* k_new, const void* v_new, void* o, void* kv_cache,
                       const int32_t* cache_seqlens, int cache_seqlen_scalar, const void* rotary_cos,
                       const void* rotary_sin, int rotary_dim, int B, int H, int hd, int max_seqlen,
                       Strides2 sq, Strides2 sk, Strides2 sv, Strides2 so, int window_left, float scale,

@@ -13,6 +13,14 @@ _MODELS = {
     "Based": "based_b200.model:BasedLMHeadModel",
     "Razesun": "based_b200.razesun:RazesunLMHeadModel",
 }
+# architectures whose kernels are all in one part of the library (see build.PARTS)
+_PARTS = {"Razesun": "hybrid"}
+
+
+def library_part(folder: str):
+    """The part of the kernel library that the model in ``folder`` needs, None for the whole."""
+    with open(os.path.join(folder, "config.json")) as f:
+        return _PARTS.get(json.load(f).get("architecture"))
 
 
 def architectures():

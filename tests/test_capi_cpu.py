@@ -114,3 +114,47 @@ def test_block_level_entry_points_reject_bad_arguments(lib):
     assert lin(p, p, None, p, 0, 64, 64, 64, 64, 0, 0, None, None, None, 0, 1, None) == 0
     s4 = _capi.strides(8, 8, 8, 8)
     assert lib.based_rotary_qkv_cache(p, 1, 4, 2, 64, s4, p, p, None, s2, None) == -1
+
+
+def test_part_of_the_library(tmp_path):
+    """The library of a part alone: everything declared is exported, kernels it lacks answer ERR_IMPL."""
+    import subprocess
+    import sys
+    code = ("import ctypes, os\n"
+            "from based_b200 import build, _capi\n"
+            f"build.LIBDIR = {str(tmp_path)!r}\n"
+            "path = build.build_library(part='hybrid')\n"
+            "assert os.path.basename(path) == 'libbased_b200_hybrid.so' and path == build.library_path()\n"
+            "lib, p, s3 = _capi.lib(), ctypes.c_void_p(256), _capi.strides(1, 1, 1)\n"
+            "assert all(hasattr(lib, n) for n in _capi.SIGNATURES)\n"
+            "assert lib.based_swa_prefill(p, p, p, p, 1, 8, 1, 64, s3, s3, s3, s3, 64, 0.125, 0, 0, None) == -5\n"
+            "assert lib.based_linattn_prefill_segments(1, 16, 4096) == 1\n"
+            "assert lib.based_latent_decode_scratch_bytes(1, 1, 16, 512, 4096) > 0\n"
+            "built = {f for f in os.listdir(os.path.join(build.LIBDIR, 'obj'))}\n"
+            "assert built == {n[:-3] + '.o' for n in build.HYBRID}\n")
+    subprocess.run([sys.executable, "-c", code], check=True, cwd=ROOT, timeout=600, env={k: v for k, v in os.environ.items() if k != "BASED_B200_LIB"})
+
+
+def test_hybrid_entry_points_reject_bad_arguments(lib):
+    p = ctypes.c_void_p(256)
+    s2, s3 = _capi.strides(8, 8), _capi.strides(8, 8, 8)
+    conv = lib.based_short_conv
+    assert conv(p, p, None, p, None, 1, 4, 8, 4, s2, s2, None, 3, 0, 1, None) == -1     # a later token needs the ring
+    assert conv(p, p, p, p, None, 1, 4, 8, 0, s2, s2, None, 0, 0, 1, None) == -2
+    assert conv(p, p, p, p, None, 1, 0, 8, 4, s2, s2, None, 0, 0, 1, None) == 0
+    norm = lib.based_stream_norm
+    assert norm(None, None, None, 0, p, 8, 1.0, p, p, p, p, None, 4, 8, 1e-6, 1, None) == -1   # w2 without out2
+    assert norm(p, None, None, 0, None, 0, 1.0, p, p, None, p, None, 4, 8, 1e-6, 1, None) == -1  # tokens without a table
+    prep = lib.based_latent_prepare
+    assert prep(p, p, p, p, p, p, 8, 1, 4, 2, 16, 8, 16, 10, s2, s2, s2, None, 5, 1e-6, 1, None) == -2   # past the tables
+    assert prep(p, p, p, p, p, p, 9, 1, 4, 2, 16, 7, 16, 10, s2, s2, s2, None, 0, 1e-6, 1, None) == -2   # odd rotation
+    pre = lib.based_latent_prefill
+    assert pre(p, p, p, p, p, None, p, 1, 4, 4, 1, 16, 16, 16, s3, s3, s3, s2, s3, s3, None, 1, 1.0, 1, 0, None) == -2  # too few keys
+    assert pre(p, p, p, p, p, None, p, 1, 4, 4, 1, 20, 16, 16, s3, s3, s3, s2, s3, s3, None, 0, 1.0, 1, 2, None) == -5  # d1 % 16
+    dec = lib.based_latent_decode
+    assert dec(p, p, p, None, p, None, 0, 1, 1, 1, 16, 16, 4, s3, s3, s2, s3, None, None, 4, 1.0, 1, None) == -2   # past the cache
+    delta = lib.based_delta_prefill
+    assert delta(p, p, p, p, p, p, p, p, p, p, p, 1, 4, 3, 2, 16, 16, s2, s2, s2, s2, s2, s2, None, 0, 1e-6, 1, 0, None, 0, None) == -2
+    assert delta(p, p, p, p, p, p, p, p, p, p, p, 1, 9, 2, 2, 20, 16, s2, s2, s2, s2, s2, s2, None, 0, 1e-6, 1, 2, None, 0, None) == -5
+    assert lib.based_rglru_gated(p, p, p, p, p, p, p, p, 1, 8, 40, 20, s2, s2, s2, None, 0, 1, None) == -5
+    assert lib.based_rglru_gated(p, p, p, p, p, p, p, p, 1, 8, 40, 16, s2, s2, s2, None, 0, 1, None) == -2
