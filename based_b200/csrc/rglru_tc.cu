@@ -168,8 +168,7 @@ __global__ void __launch_bounds__(NT, 1) rglru_tc_kernel(const __grid_constant__
       float pr = 1.f, sr = 0.f;
 #pragma unroll
       for (int i = 0; i < TG; ++i) {
-        const int row = t0g + i;
-        const float u = live ? __bfloat162float(*reinterpret_cast<const bf16*>(us + row * 128 + ((chunk ^ (row & 7)) << 4))) : 0.f;
+        const float u = live ? __bfloat162float(*reinterpret_cast<const bf16*>(us + (t0g + i) * 128 + ((chunk ^ (i & 7)) << 4))) : 0.f;
         const float er = 1.f + ex2(fminf(fmaf(__uint_as_float(gr[i]), -kLog2e, rb), 60.f));
         const float ei = 1.f + ex2(fminf(fmaf(__uint_as_float(gi[i]), -kLog2e, ib), 60.f));
         const float q = rcp(er * ei);                       // both sigmoids from one reciprocal
@@ -200,12 +199,13 @@ __global__ void __launch_bounds__(NT, 1) rglru_tc_kernel(const __grid_constant__
       mbar_arrive(my_carry);
       mbar_wait_bounded(B_Y + 8 * x, (t >> 1) & 1, abort_flag, p.status, 1u << 24);
       uint8_t* ys = ycol + x * 2 * kUAtom;
+      auto at = [&](int i) { return reinterpret_cast<bf16*>(ys + (t0g + i) * 128 + ((ychunk ^ (i & 7)) << 4)); };   // t0g is a multiple of 8
+      bf16 yv[TG];   // all read before the first is replaced
 #pragma unroll
-      for (int i = 0; i < TG; ++i) {   // rows past the sequence and channels past the block are clipped by the store
-        const int row = t0g + i;
-        bf16* e = reinterpret_cast<bf16*>(ys + row * 128 + ((ychunk ^ (row & 7)) << 4));
-        *e = __float2bfloat16_rn(fmaf(P[i], S0, s[i]) * seq::gelu_tanh_t<bf16>(__bfloat162float(*e)));
-      }
+      for (int i = 0; i < TG; ++i) yv[i] = *at(i);
+#pragma unroll
+      for (int i = 0; i < TG; ++i)     // rows past the sequence and channels past the block are clipped by the store
+        *at(i) = __float2bfloat16_rn(fmaf(P[i], S0, s[i]) * seq::gelu_tanh_t<bf16>(__bfloat162float(yv[i])));
       fence_proxy_async();
       mbar_arrive(B_OUT + 8 * x);
       if (live && grp == GROUPS - 1 && t == nt - 1) p.state[(int64_t)b * p.W + chan] = end;
