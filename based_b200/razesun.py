@@ -85,6 +85,8 @@ class ParallelBlock(nn.Module):
         self.mixer.load_tensors(t, prefix + "mix.")
         with torch.no_grad():
             self.norm1.copy_(t.get(prefix + "norm1", (d,)))
+            if self.mlp is None and prefix + "norm2" in t:
+                t.get(prefix + "norm2", (d,))   # the second norm of a layer without an MLP has nothing to feed
             if self.mlp is not None:
                 self.norm2.copy_(t.get(prefix + "norm2", (d,)))
                 self.mlp.fc1.weight[:self.ff].copy_(t.get(prefix + "mlp.up", (self.ff, d)))

@@ -44,7 +44,7 @@ def expect(q1, q2, k1, k2, v, gate, pos, scale):
 
 
 # (d1, d2, dv): a small model's, a large model's, and sizes that are no multiple of 64
-SIZES = [(64, 32, 64), (128, 64, 128), (48, 16, 80), (80, 48, 32), (32, 96, 112)]
+SIZES = [(64, 16, 96), (128, 64, 128), (48, 16, 80), (80, 48, 32), (32, 96, 112)]
 CUTS = [(129, 129, 0), (300, 300, 0), (64, 192, 128), (257, 600, 343), (2, 130, 127), (3, 131, 128), (100, 356, 256), (520, 520, 0),
         (31, 31, 0), (1, 1, 0), (255, 640, 384)]
 
@@ -73,7 +73,7 @@ def test_expanded_form(d1, d2, dv, impl):
 
 def test_expanded_form_fp32_and_odd_sizes():
     from based_b200 import ops
-    for n, (d1, d2, dv, dtype) in enumerate([(64, 32, 64, torch.float32), (33, 6, 21, torch.float32), (20, 10, 30, torch.bfloat16),
+    for n, (d1, d2, dv, dtype) in enumerate([(64, 16, 96, torch.float32), (33, 6, 21, torch.float32), (20, 10, 30, torch.bfloat16),
                                              (128, 64, 200, torch.bfloat16)]):
         L, T, pos, H, scale = 77, 177, 100, 3, (d1 + d2) ** -0.5
         t = [x.to(dtype) for x in aimed(L, T, H, d1, d2, dv, pos, scale, seed=n)]
@@ -86,7 +86,7 @@ def test_expanded_form_fp32_and_odd_sizes():
 def test_long_far_keys():
     """One head, 5000 keys: keys thousands of tokens back, and the running maximum that grows on the way."""
     from based_b200 import ops
-    d1, d2, dv, H, L, T = 64, 32, 64, 2, 5000, 5000
+    d1, d2, dv, H, L, T = 64, 48, 64, 2, 5000, 5000
     scale = (d1 + d2) ** -0.5
     t = [x.bfloat16() for x in aimed(L, T, H, d1, d2, dv, 0, scale, seed=5)]
     # a slope along the keys makes the running maximum of most rows grow tile by tile
@@ -107,8 +107,8 @@ def test_long_far_keys():
         assert rel_err(o[0].float().cpu()[rows], ref) < 1.5e-2
 
 
-@pytest.mark.parametrize("r,rd,H,dtype", [(64, 32, 4, torch.bfloat16), (512, 64, 16, torch.bfloat16), (96, 16, 3, torch.bfloat16),
-                                          (200, 24, 5, torch.bfloat16), (64, 32, 4, torch.float32), (33, 6, 2, torch.float32),
+@pytest.mark.parametrize("r,rd,H,dtype", [(80, 32, 4, torch.bfloat16), (512, 64, 16, torch.bfloat16), (96, 16, 3, torch.bfloat16),
+                                          (200, 24, 5, torch.bfloat16), (80, 32, 4, torch.float32), (33, 6, 2, torch.float32),
                                           (33, 6, 2, torch.bfloat16), (512, 64, 40, torch.bfloat16)])
 def test_absorbed_form(r, rd, H, dtype):
     """Positions at and around tile and split borders, one position per row of the batch, several query tokens."""

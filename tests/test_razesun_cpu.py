@@ -54,6 +54,8 @@ def test_every_tensor_is_loaded_and_has_its_place(name, tmp_path):
             assert torch.equal(layer.out_weight[:, layer.split:], t[f"l{i}.mlp.down"].float())
             assert torch.equal(layer.mlp.fc1.weight, torch.cat([t[f"l{i}.mlp.up"], t[f"l{i}.mlp.gate"]]).float())
         assert bool((layer.out_weight[:, layer.inner:layer.split] == 0).all())
+    bare = [i for i, layer in enumerate(m.layers) if layer.mlp is None]
+    m.load_tensors(weights.TensorDict({**t, **{f"l{i}.norm2": t["final.norm"] for i in bare}}))
     with pytest.raises(ValueError, match="does not have"):
         m.load_tensors(weights.TensorDict({**t, "l0.extra": torch.zeros(1)}))
     del t["final.norm"]

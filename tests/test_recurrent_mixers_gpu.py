@@ -76,7 +76,7 @@ def delta_reference(q, k, v, z, a, b, A_log, dt, w, eps):
     return torch.stack(outs), torch.stack(states)
 
 
-DELTA_SIZES = [(6, 3, 64, 32), (4, 4, 128, 128), (4, 2, 32, 64), (2, 1, 96, 48), (3, 1, 64, 144), (2, 2, 128, 256)]
+DELTA_SIZES = [(6, 2, 64, 48), (4, 4, 128, 128), (4, 2, 32, 64), (2, 1, 96, 48), (3, 1, 64, 144), (2, 2, 128, 256)]
 
 
 @pytest.mark.parametrize("H,Hk,d,dv", DELTA_SIZES)
@@ -104,7 +104,7 @@ def test_delta_chunked(H, Hk, d, dv, strong):
 
 
 @pytest.mark.parametrize("H,Hk,d,dv,dtype", [(4, 2, 64, 32, torch.float32), (3, 1, 20, 12, torch.float32), (2, 2, 33, 300, torch.float32),
-                                             (6, 3, 64, 32, torch.bfloat16), (2, 1, 40, 24, torch.bfloat16), (2, 1, 256, 192, torch.bfloat16)])
+                                             (6, 2, 64, 48, torch.bfloat16), (2, 1, 40, 24, torch.bfloat16), (2, 1, 256, 192, torch.bfloat16)])
 def test_delta_recurrent(H, Hk, d, dv, dtype):
     from based_b200 import ops
     eps, L = 1e-6, 70
@@ -119,7 +119,7 @@ def test_delta_recurrent(H, Hk, d, dv, dtype):
     assert rel_err(out.float().cpu().view(2, L, H, dv), ref) < (1e-5 if dtype == torch.float32 else 1e-2)
 
 
-@pytest.mark.parametrize("H,Hk,d,dv,taps", [(6, 3, 64, 32, 4), (4, 4, 128, 128, 4), (2, 1, 40, 24, 2), (3, 1, 96, 48, 3), (2, 2, 256, 64, 5)])
+@pytest.mark.parametrize("H,Hk,d,dv,taps", [(6, 2, 64, 48, 4), (4, 4, 128, 128, 4), (2, 1, 40, 24, 2), (3, 1, 96, 48, 3), (2, 2, 256, 64, 5)])
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
 def test_delta_step(H, Hk, d, dv, taps, dtype):
     """Token by token from the packed projection, two sequences at different positions, against convolution + oracle."""
