@@ -67,6 +67,19 @@ SIGNATURES = {
     "based_delta_step": (c_int, [c_void_p] * 10 + [c_int] * 6 + [c_int64] * 3 + _POS + [c_float, c_int, c_void_p]),
     "based_rglru_gated": (c_int, [c_void_p] * 8 + [c_int] * 4 + [_I64P] * 3 + _POS + [c_int, c_void_p]),
     "based_rglru": (c_int, [c_void_p] * 8 + [c_int] * 4 + [_I64P] * 4 + _POS + [c_int, c_void_p]),
+    # post-norm stacks
+    "based_stream_embed": (c_int, [c_void_p, c_void_p, c_int64, c_float, c_void_p, c_int64, c_void_p, c_void_p] + [c_int] * 3
+                           + _POS + [c_int, c_void_p]),
+    "based_stream_post_norm": (c_int, [c_void_p, c_int64] + [c_void_p] * 4 + [c_int64, c_int, c_float, c_int, c_void_p]),
+    "based_norm_gate": (c_int, [c_void_p, c_int64, c_void_p, c_void_p, c_int64, c_void_p, c_int64, c_int64, c_int, c_float, c_int,
+                                c_void_p]),
+    "based_token_gate": (c_int, [c_void_p, c_int64, c_void_p, c_void_p] + [c_int64] * 3 + [c_void_p, c_int64, c_int, c_int, c_void_p]),
+    "based_tied_prepare": (c_int, [c_void_p] * 6 + [c_int] * 6 + [_I64P] * 4 + _POS + [c_float] * 3 + [c_int, c_void_p]),
+    "based_tied_attention": (c_int, [c_void_p] * 5 + [c_int] * 6 + [_I64P] * 5 + _POS
+                             + [c_float, c_float, c_int, c_int, c_void_p, ctypes.c_size_t, c_void_p]),
+    "based_lightning": (c_int, [c_void_p] * 6 + [c_int] * 5 + [_I64P] * 4 + _POS + [c_int, c_int, c_void_p]),
+    "based_lightning_step": (c_int, [c_void_p] * 4 + [c_int64] + [c_void_p] * 6 + [c_int64] + [c_int] * 4 + _POS
+                             + [c_float, c_int, c_void_p]),
 }
 
 _lib = None

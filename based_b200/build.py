@@ -9,11 +9,12 @@ ROOT = os.path.dirname(PKG)
 CSRC = os.path.join(PKG, "csrc")
 LIBDIR = os.path.join(PKG, "_lib")
 LIBNAME = "libbased_b200.so"
-# Sources of a library for the hybrid stacks alone.  capi.cu refers to the other kernels weakly: in such a library their
-# entry points answer BASED_ERR_IMPL.
+# Sources of libraries for the hybrid stacks and for the post-norm stacks alone.  capi.cu refers to the other kernels weakly:
+# in such a library their entry points answer BASED_ERR_IMPL.
 HYBRID = ("capi.cu", "norm_act.cu", "decode_linear.cu", "short_conv.cu", "gated_delta.cu", "gated_delta_chunk.cu", "rglru.cu",
           "rglru_tc.cu", "latent_attention.cu", "latent_decode.cu", "latent_prefill_tc.cu")
-PARTS = {"hybrid": ("libbased_b200_hybrid.so", HYBRID)}
+POSTNORM = ("capi.cu", "norm_act.cu", "decode_linear.cu", "latent_attention.cu", "tied_attention.cu", "lightning.cu")
+PARTS = {"hybrid": ("libbased_b200_hybrid.so", HYBRID), "postnorm": ("libbased_b200_postnorm.so", POSTNORM)}
 _chosen = None   # library of the part this process asked for, when that is not the whole one
 
 def library_path() -> str:

@@ -40,9 +40,9 @@ int based_read_status(unsigned int* out, int reset) {
   int rc = read_tc_status ? read_tc_status(&a, reset) : 0;
   if (rc == 0 && read_tc_status_swa) rc = read_tc_status_swa(&b, reset);
   if (rc == 0 && read_tp_status) rc = read_tp_status(&c, reset);
-  if (rc == 0) rc = read_tc_status_latent(&d, reset);
-  if (rc == 0) rc = read_tc_status_delta(&e, reset);
-  if (rc == 0) rc = read_tc_status_rglru(&f, reset);
+  if (rc == 0 && read_tc_status_latent) rc = read_tc_status_latent(&d, reset);
+  if (rc == 0 && read_tc_status_delta) rc = read_tc_status_delta(&e, reset);
+  if (rc == 0 && read_tc_status_rglru) rc = read_tc_status_rglru(&f, reset);
   if (out) *out = a | b | c | d | e | f;
   return rc;
 }
@@ -380,6 +380,7 @@ int based_short_conv(const void* x, void* y, void* ring, const void* weight, con
   if (B < 0 || L < 0 || C <= 0 || taps < 1 || offset < 0) return BASED_ERR_SHAPE;
   if (!ring && (offsets || offset > 0)) return BASED_ERR_NULL;
   if (B == 0 || L == 0) return BASED_OK;
+  if (!launch_short_conv) return BASED_ERR_IMPL;
   return launch_short_conv(x, y, ring, weight, bias, B, L, C, taps, s2(x_strides), s2(y_strides), offsets, offset, silu,
                            io_dtype, static_cast<cudaStream_t>(stream));
 }
@@ -397,6 +398,7 @@ int based_latent_prepare(const void* z, const void* norm_weight, void* cache, vo
   if (B == 0 || L == 0) return BASED_OK;
   const int64_t zero[2] = {0, 0};
   const int64_t *zs = z ? z_strides : zero, *cs = z ? cache_strides : zero, *qs = q ? q_strides : zero;
+  if (!launch_latent_prepare) return BASED_ERR_IMPL;
   return launch_latent_prepare(z, norm_weight, cache, q, static_cast<const float*>(cos_table),
                                static_cast<const float*>(sin_table), table_len, B, L, H, kv_rank, rot_dim, dim, max_len,
                                zs[0], zs[1], cs[0], cs[1], qs[0], qs[1], offsets, offset, eps, io_dtype,
@@ -414,10 +416,11 @@ int based_split_key_attention(const void* q1, const void* q2, const void* k1, co
   if (!dtype_ok(io_dtype)) return BASED_ERR_DTYPE;
   if (B < 0 || L < 0 || H <= 0 || d1 <= 0 || d2 < 0 || dv <= 0 || offset < 0) return BASED_ERR_SHAPE;
   if (B == 0 || L == 0) return BASED_OK;
+  if (!launch_split_key_attention) return BASED_ERR_IMPL;
   return launch_split_key_attention(q1, q2, k1, k2, v, gate, out, B, L, H, d1, d2, dv, s3_blh(q1_strides),
                                     s3_blh(q2_strides), s3_blh(k1_strides), s3_blh(k2_strides), s3_blh(v_strides),
                                     s3_blh(out_strides), gate ? gate_strides[0] : 0, gate ? gate_strides[1] : 0, offsets,
-                                    offset, scale, io_dtype, static_cast<cudaStream_t>(stream));
+                                    offset, scale, AttentionOptions{}, io_dtype, static_cast<cudaStream_t>(stream));
 }
 
 int based_latent_prefill(const void* q1, const void* q2, const void* k1, const void* k2, const void* v, const void* gate,
@@ -435,18 +438,21 @@ int based_latent_prefill(const void* q1, const void* q2, const void* k1, const v
   const int64_t gb = gate ? gate_strides[0] : 0, gl = gate ? gate_strides[1] : 0;
   if (impl == BASED_IMPL_TCGEN05 || (impl == BASED_IMPL_AUTO && io_dtype == BASED_BF16)) {
     if (io_dtype != BASED_BF16) return BASED_ERR_IMPL;
+    if (!launch_latent_prefill_tc) return BASED_ERR_IMPL;
     const int rc = launch_latent_prefill_tc(q1, q2, k1, k2, v, gate, out, B, L, T, H, d1, d2, dv, s3_blh(q1_strides),
                                             s3_blh(q2_strides), s3_blh(k1_strides), sk2, s3_blh(v_strides),
                                             s3_blh(out_strides), gb, gl, nullptr, offset, scale, st);
     if (!(impl == BASED_IMPL_AUTO && rc == BASED_ERR_IMPL)) return rc;
   }
+  if (!launch_split_key_attention) return BASED_ERR_IMPL;
   return launch_split_key_attention(q1, q2, k1, k2, v, gate, out, B, L, H, d1, d2, dv, s3_blh(q1_strides),
                                     s3_blh(q2_strides), s3_blh(k1_strides), sk2, s3_blh(v_strides), s3_blh(out_strides),
-                                    gb, gl, nullptr, offset, scale, io_dtype, st);
+                                    gb, gl, nullptr, offset, scale, AttentionOptions{}, io_dtype, st);
 }
 
 size_t based_latent_decode_scratch_bytes(int B, int L, int H, int kv_rank, int max_len) {
   if (B <= 0 || L <= 0 || H <= 0 || kv_rank <= 0 || max_len <= 0) return 0;
+  if (!latent_decode_scratch_bytes) return 0;
   return latent_decode_scratch_bytes(B, L * H, kv_rank, max_len);
 }
 
@@ -464,6 +470,7 @@ int based_latent_decode(const void* qa, const void* qr, const void* cache, const
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   const int64_t gb = gate ? gate_strides[0] : 0, gl = gate ? gate_strides[1] : 0;
   if (io_dtype == BASED_BF16) {
+    if (!launch_latent_decode) return BASED_ERR_IMPL;
     const int rc = launch_latent_decode(qa, qr, cache, gate, out, scratch, scratch_bytes, B, L, H, kv_rank, rot_dim, max_len,
                                         s3_blh(qa_strides), s3_blh(qr_strides), cache_strides[0], cache_strides[1],
                                         s3_blh(out_strides), gb, gl, offsets, offset, scale, st);
@@ -472,9 +479,10 @@ int based_latent_decode(const void* qa, const void* qr, const void* cache, const
   // fp32 models and other sizes: the cached rows as keys and values of every head
   const Strides3 sc{cache_strides[0], 0, cache_strides[1]};
   const char* rot = static_cast<const char*>(cache) + kv_rank * dtype_size(io_dtype);
+  if (!launch_split_key_attention) return BASED_ERR_IMPL;
   return launch_split_key_attention(qa, qr, cache, rot, cache, gate, out, B, L, H, kv_rank, rot_dim, kv_rank,
                                     s3_blh(qa_strides), s3_blh(qr_strides), sc, sc, sc, s3_blh(out_strides), gb, gl, offsets,
-                                    offset, scale, io_dtype, st);
+                                    offset, scale, AttentionOptions{}, io_dtype, st);
 }
 
 int based_delta_prefill(const void* q, const void* k, const void* v, const void* z, const void* a, const void* b,
@@ -491,6 +499,7 @@ int based_delta_prefill(const void* q, const void* k, const void* v, const void*
   // AUTO: chunks for bf16 from a handful of tokens on, else token by token
   if (impl == BASED_IMPL_TCGEN05 || (impl == BASED_IMPL_AUTO && io_dtype == BASED_BF16 && L >= 8)) {
     if (io_dtype != BASED_BF16) return BASED_ERR_IMPL;
+    if (!launch_delta_chunk) return BASED_ERR_IMPL;
     const int rc = launch_delta_chunk(q, k, v, z, static_cast<const float*>(a), static_cast<const float*>(b),
                                       static_cast<const float*>(A_log), static_cast<const float*>(dt_bias), norm_weight,
                                       static_cast<float*>(state), out, scratch, scratch_bytes, B, L, H, Hk, d, dv,
@@ -498,6 +507,7 @@ int based_delta_prefill(const void* q, const void* k, const void* v, const void*
                                       s2(out_strides), offsets, offset, eps, static_cast<cudaStream_t>(stream));
     if (!(impl == BASED_IMPL_AUTO && rc == BASED_ERR_IMPL)) return rc;
   }
+  if (!launch_delta_recurrent) return BASED_ERR_IMPL;
   return launch_delta_recurrent(q, k, v, z, static_cast<const float*>(a), static_cast<const float*>(b),
                                 static_cast<const float*>(A_log), static_cast<const float*>(dt_bias), norm_weight,
                                 static_cast<float*>(state), out, B, L, H, Hk, d, dv, s2(q_strides), s2(k_strides),
@@ -507,6 +517,7 @@ int based_delta_prefill(const void* q, const void* k, const void* v, const void*
 
 size_t based_delta_prefill_scratch_bytes(int B, int L, int H, int d, int dv) {
   if (B <= 0 || L <= 0 || H <= 0 || d <= 0 || dv <= 0) return 0;
+  if (!delta_chunk_scratch_bytes) return 0;
   return delta_chunk_scratch_bytes(B, L, H, d, dv);
 }
 
@@ -518,6 +529,7 @@ int based_delta_step(const void* x, const void* conv_weight, void* ring, const v
   if (!dtype_ok(io_dtype)) return BASED_ERR_DTYPE;
   if (B < 0 || H <= 0 || Hk <= 0 || H % Hk || d <= 0 || dv <= 0 || taps < 1 || offset < 0) return BASED_ERR_SHAPE;
   if (B == 0) return BASED_OK;
+  if (!launch_delta_step) return BASED_ERR_IMPL;
   return launch_delta_step(x, conv_weight, ring, static_cast<const float*>(a), static_cast<const float*>(b),
                            static_cast<const float*>(A_log), static_cast<const float*>(dt_bias), norm_weight,
                            static_cast<float*>(state), out, B, H, Hk, d, dv, taps, x_stride, gate_stride, out_stride,
@@ -533,6 +545,7 @@ int based_rglru(const void* u, const void* y, const void* gates, const void* r_b
   if (!dtype_ok(io_dtype)) return BASED_ERR_DTYPE;
   if (B < 0 || L < 0 || W <= 0 || block_width <= 0 || W % block_width || offset < 0) return BASED_ERR_SHAPE;
   if (B == 0 || L == 0) return BASED_OK;
+  if (!launch_rglru) return BASED_ERR_IMPL;
   return launch_rglru(u, y, static_cast<const float*>(gates), r_bias, i_bias, static_cast<const float*>(lam),
                       static_cast<float*>(state), out, B, L, W, block_width, s2(u_strides), s2(y_strides),
                       s2(out_strides), gate_strides[0], gate_strides[1], offsets, offset, io_dtype,
@@ -549,9 +562,123 @@ int based_rglru_gated(const void* u, const void* y, const void* gate_weight, con
   if (B < 0 || L < 0 || W <= 0 || block_width <= 0 || W % block_width || offset < 0) return BASED_ERR_SHAPE;
   if (B == 0 || L == 0) return BASED_OK;
   if (io_dtype != BASED_BF16) return BASED_ERR_IMPL;
+  if (!launch_rglru_tc) return BASED_ERR_IMPL;
   return launch_rglru_tc(u, y, gate_weight, r_bias, i_bias, static_cast<const float*>(lam), static_cast<float*>(state), out,
                          B, L, W, block_width, s2(u_strides), s2(y_strides), s2(out_strides), offsets, offset,
                          static_cast<cudaStream_t>(stream));
+}
+
+// ------------------------------------------------------------------ post-norm stacks
+
+int based_stream_embed(const void* tokens, const void* table, int64_t V, float scale, const void* pos_table, int64_t P,
+                       void* residual, void* out, int B, int L, int D, const int32_t* offsets, int offset, int io_dtype,
+                       void* stream) {
+  if (!tokens || !table || !pos_table || !residual) return BASED_ERR_NULL;
+  if (!dtype_ok(io_dtype)) return BASED_ERR_DTYPE;
+  if (B < 0 || L < 0 || D <= 0 || V <= 0 || P <= 0 || offset < 0) return BASED_ERR_SHAPE;
+  if (!offsets && (int64_t)offset + L > P) return BASED_ERR_SHAPE;
+  if (B == 0 || L == 0) return BASED_OK;
+  return launch_stream_embed(static_cast<const int64_t*>(tokens), table, V, scale, pos_table, P, static_cast<float*>(residual),
+                             out, B, L, D, offsets, offset, io_dtype, static_cast<cudaStream_t>(stream));
+}
+
+int based_stream_post_norm(const void* branch, int64_t branch_row_stride, const void* weight, void* residual,
+                           const void* out_weight, void* out, int64_t M, int D, float eps, int io_dtype, void* stream) {
+  if (!branch || !weight || !residual || (out_weight && !out)) return BASED_ERR_NULL;
+  if (!dtype_ok(io_dtype)) return BASED_ERR_DTYPE;
+  if (M < 0 || D <= 0) return BASED_ERR_SHAPE;
+  if (M == 0) return BASED_OK;
+  return launch_stream_post_norm(branch, branch_row_stride, weight, static_cast<float*>(residual), out_weight, out, M, D, eps,
+                                 io_dtype, static_cast<cudaStream_t>(stream));
+}
+
+int based_norm_gate(const void* x, int64_t x_row_stride, const void* weight, const void* gate, int64_t gate_row_stride,
+                    void* out, int64_t out_row_stride, int64_t M, int D, float eps, int io_dtype, void* stream) {
+  if (!x || !weight || !gate || !out) return BASED_ERR_NULL;
+  if (!dtype_ok(io_dtype)) return BASED_ERR_DTYPE;
+  if (M < 0 || D <= 0) return BASED_ERR_SHAPE;
+  if (M == 0) return BASED_OK;
+  return launch_norm_gate(x, x_row_stride, weight, gate, gate_row_stride, out, out_row_stride, M, D, eps, io_dtype,
+                          static_cast<cudaStream_t>(stream));
+}
+
+int based_token_gate(const void* z, int64_t z_row_stride, const void* tokens, const void* table, int64_t V,
+                     int64_t table_row_stride, int64_t column, void* out, int64_t M, int n, int io_dtype, void* stream) {
+  if (!z || !tokens || !table || !out) return BASED_ERR_NULL;
+  if (!dtype_ok(io_dtype)) return BASED_ERR_DTYPE;
+  if (M < 0 || n <= 0 || V <= 0 || column < 0 || column + n > table_row_stride) return BASED_ERR_SHAPE;
+  if (M == 0) return BASED_OK;
+  return launch_token_gate(z, z_row_stride, static_cast<const int64_t*>(tokens), table, V, table_row_stride, column, out, M, n,
+                           io_dtype, static_cast<cudaStream_t>(stream));
+}
+
+int based_tied_prepare(void* q, const void* k, const void* q_weight, const void* k_weight, void* cache, void* factor, int B,
+                       int L, int H, int G, int d, int max_len, const int64_t q_strides[2], const int64_t k_strides[2],
+                       const int64_t cache_strides[2], const int64_t factor_strides[2], const int32_t* offsets, int offset,
+                       float eps, float temp_coef, float temp_every, int io_dtype, void* stream) {
+  if (!q || !k || !q_weight || !k_weight || !cache || !factor) return BASED_ERR_NULL;
+  if (!q_strides || !k_strides || !cache_strides || !factor_strides) return BASED_ERR_NULL;
+  if (!dtype_ok(io_dtype)) return BASED_ERR_DTYPE;
+  if (B < 0 || L < 0 || H <= 0 || G <= 0 || H % G || d <= 0 || d > 512 || offset < 0) return BASED_ERR_SHAPE;
+  if (temp_coef != 0.f && !(temp_every > 0.f)) return BASED_ERR_SHAPE;
+  if (!offsets && (int64_t)offset + L > max_len) return BASED_ERR_SHAPE;
+  if (B == 0 || L == 0) return BASED_OK;
+  if (!launch_tied_prepare) return BASED_ERR_IMPL;
+  return launch_tied_prepare(q, k, q_weight, k_weight, cache, static_cast<float*>(factor), B, L, H, G, d, max_len, q_strides[0],
+                             q_strides[1], k_strides[0], k_strides[1], cache_strides[0], cache_strides[1], factor_strides[0],
+                             factor_strides[1], offsets, offset, eps, temp_coef, temp_every, io_dtype,
+                             static_cast<cudaStream_t>(stream));
+}
+
+int based_tied_attention(const void* q, const void* cache, const void* factor, const void* gate, void* out, int B, int L, int H,
+                         int G, int d, int max_len, const int64_t q_strides[2], const int64_t cache_strides[2],
+                         const int64_t factor_strides[2], const int64_t gate_strides[2], const int64_t out_strides[2],
+                         const int32_t* offsets, int offset, float scale, float sink, int io_dtype, int impl, void* scratch,
+                         size_t scratch_bytes, void* stream) {
+  if (!q || !cache || !factor || !out || (gate && !gate_strides)) return BASED_ERR_NULL;
+  if (!q_strides || !cache_strides || !factor_strides || !out_strides) return BASED_ERR_NULL;
+  if (!dtype_ok(io_dtype)) return BASED_ERR_DTYPE;
+  if (B < 0 || L < 0 || H <= 0 || G <= 0 || H % G || d <= 0 || d > 512 || max_len <= 0 || offset < 0 || sink < 0.f) return BASED_ERR_SHAPE;
+  if (!offsets && (int64_t)offset + L > max_len) return BASED_ERR_SHAPE;
+  if (B == 0 || L == 0) return BASED_OK;
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  AttentionOptions x;
+  x.key_factor = static_cast<const float*>(factor);
+  x.fb = factor_strides[0]; x.fh = factor_strides[1];
+  x.group = H / G;
+  x.sink = sink;
+  x.gate_per_element = 1;
+  const int64_t gb = gate ? gate_strides[0] : 0, gl = gate ? gate_strides[1] : 0;
+  const Strides3 sq{q_strides[0], d, q_strides[1]}, sc{cache_strides[0], d, cache_strides[1]}, so{out_strides[0], d, out_strides[1]};
+  if (!launch_split_key_attention) return BASED_ERR_IMPL;
+  return launch_split_key_attention(q, q, cache, cache, cache, gate, out, B, L, H, d, 0, d, sq, sq, sc, sc, sc, so, gb, gl,
+                                    offsets, offset, scale, x, io_dtype, st);
+}
+
+int based_lightning(const void* q, const void* k, const void* v, const void* decay, void* state, void* out, int B, int L, int H,
+                    int d, int dv, const int64_t q_strides[2], const int64_t k_strides[2], const int64_t v_strides[2],
+                    const int64_t out_strides[2], const int32_t* offsets, int offset, int io_dtype, int impl, void* stream) {
+  if (!q || !k || !v || !decay || !state || !out || !q_strides || !k_strides || !v_strides || !out_strides) return BASED_ERR_NULL;
+  if (!dtype_ok(io_dtype)) return BASED_ERR_DTYPE;
+  if (B < 0 || L < 0 || H <= 0 || d <= 0 || d > 512 || dv <= 0 || offset < 0) return BASED_ERR_SHAPE;
+  if (B == 0 || L == 0) return BASED_OK;
+  if (!launch_lightning_recurrent) return BASED_ERR_IMPL;
+  return launch_lightning_recurrent(q, k, v, static_cast<const float*>(decay), static_cast<float*>(state), out, B, L, H, d, dv,
+                                    s2(q_strides), s2(k_strides), s2(v_strides), s2(out_strides), offsets, offset, io_dtype,
+                                    static_cast<cudaStream_t>(stream));
+}
+
+int based_lightning_step(const void* q, const void* k, const void* v, const void* gate, int64_t x_row_stride, const void* decay,
+                         const void* norm_weight, void* state, void* read, void* count, void* out, int64_t out_row_stride, int B,
+                         int H, int d, int dv, const int32_t* offsets, int offset, float eps, int io_dtype, void* stream) {
+  if (!q || !k || !v || !gate || !decay || !norm_weight || !state || !read || !count || !out) return BASED_ERR_NULL;
+  if (!dtype_ok(io_dtype)) return BASED_ERR_DTYPE;
+  if (B < 0 || H <= 0 || d <= 0 || dv <= 0 || offset < 0) return BASED_ERR_SHAPE;
+  if (B == 0) return BASED_OK;
+  if (!launch_lightning_step) return BASED_ERR_IMPL;
+  return launch_lightning_step(q, k, v, gate, x_row_stride, static_cast<const float*>(decay), norm_weight,
+                               static_cast<float*>(state), static_cast<float*>(read), static_cast<int*>(count), out,
+                               out_row_stride, B, H, d, dv, offsets, offset, eps, io_dtype, static_cast<cudaStream_t>(stream));
 }
 
 }  // extern "C"

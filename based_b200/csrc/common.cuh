@@ -119,59 +119,91 @@ BASED_WEAK int launch_swa_decode(const void* q, const void* k_new, const void* v
                       Strides2 sq, Strides2 sk, Strides2 sv, Strides2 so, int window_left, float scale,
                       int io_dtype, cudaStream_t stream);
 
+// What an attention kernel may do beyond softmax(q k^T) v with a gate per head.
+struct AttentionOptions {
+  const float* key_factor = nullptr;   // [B, key heads, keys]: factor of a key's scores (strides fb, fh, 1)
+  int64_t fb = 0, fh = 0;
+  int group = 1;                       // query heads that share a key head
+  float sink = 0.f;                    // added to the softmax sum as that many scores of 0 without a value
+  int gate_per_element = 0;            // gate [B, L, H * dv] instead of [B, L, H]
+};
+
 // Stateful mixers of the hybrid stacks.  offsets (device, one per batch row) or offset: position of a call's first token.
 int launch_stream_norm(const int64_t* tokens, const void* table, const void* table_norm, int64_t V, const void* branch,
                        int64_t branch_stride, float mult, float* residual, const void* w1, const void* w2, void* out1,
                        void* out2, int64_t M, int D, float eps, int io_dtype, cudaStream_t stream);
 int launch_rmsnorm(const void* x, const void* w, void* out, int64_t M, int D, int64_t sx, int64_t so, float eps,
                    int io_dtype, cudaStream_t stream);
-int launch_short_conv(const void* x, void* y, void* ring, const void* w, const void* bias, int B, int L, int C, int taps,
+BASED_WEAK int launch_short_conv(const void* x, void* y, void* ring, const void* w, const void* bias, int B, int L, int C, int taps,
                       Strides2 sx, Strides2 sy, const int32_t* offsets, int offset, int silu, int io_dtype,
                       cudaStream_t stream);
-int launch_latent_prepare(const void* z, const void* norm_w, void* cache, void* q, const float* cosv, const float* sinv,
+BASED_WEAK int launch_latent_prepare(const void* z, const void* norm_w, void* cache, void* q, const float* cosv, const float* sinv,
                           int table_len, int B, int L, int H, int r, int rd, int d, int max_len, int64_t zb, int64_t zl,
                           int64_t cb, int64_t cl, int64_t qb, int64_t ql, const int32_t* offsets, int offset, float eps,
                           int io_dtype, cudaStream_t stream);
-int launch_split_key_attention(const void* q1, const void* q2, const void* k1, const void* k2, const void* v,
+BASED_WEAK int launch_split_key_attention(const void* q1, const void* q2, const void* k1, const void* k2, const void* v,
                                const void* gate, void* out, int B, int L, int H, int d1, int d2, int dv, Strides3 sq1,
                                Strides3 sq2, Strides3 sk1, Strides3 sk2, Strides3 sv, Strides3 so, int64_t gb, int64_t gl,
-                               const int32_t* offsets, int offset, float scale, int io_dtype, cudaStream_t stream);
-int launch_delta_recurrent(const void* q, const void* k, const void* v, const void* z, const float* a, const float* b,
+                               const int32_t* offsets, int offset, float scale, AttentionOptions x, int io_dtype,
+                               cudaStream_t stream);
+BASED_WEAK int launch_delta_recurrent(const void* q, const void* k, const void* v, const void* z, const float* a, const float* b,
                            const float* A_log, const float* dt_bias, const void* norm_w, float* state, void* out, int B,
                            int L, int H, int Hk, int d, int dv, Strides2 sq, Strides2 sk, Strides2 sv, Strides2 sz,
                            Strides2 sg, Strides2 so, const int32_t* offsets, int offset, float eps, int io_dtype,
                            cudaStream_t stream);
-int launch_delta_step(const void* x, const void* conv_w, void* ring, const float* a, const float* b, const float* A_log,
+BASED_WEAK int launch_delta_step(const void* x, const void* conv_w, void* ring, const float* a, const float* b, const float* A_log,
                       const float* dt_bias, const void* norm_w, float* state, void* out, int B, int H, int Hk, int d,
                       int dv, int taps, int64_t sx, int64_t sg, int64_t so, const int32_t* offsets, int offset, float eps,
                       int io_dtype, cudaStream_t stream);
-int launch_rglru(const void* u, const void* y, const float* gates, const void* rb, const void* ib, const float* lam,
+BASED_WEAK int launch_rglru(const void* u, const void* y, const float* gates, const void* rb, const void* ib, const float* lam,
                  float* state, void* out, int B, int L, int W, int bw, Strides2 su, Strides2 sy, Strides2 so,
                  int64_t g_block, int64_t g_row, const int32_t* offsets, int offset, int io_dtype, cudaStream_t stream);
 
-int launch_latent_prefill_tc(const void* q1, const void* q2, const void* k1, const void* k2, const void* v,
+BASED_WEAK int launch_latent_prefill_tc(const void* q1, const void* q2, const void* k1, const void* k2, const void* v,
                              const void* gate, void* out, int B, int L, int T, int H, int d1, int d2, int dv, Strides3 sq1,
                              Strides3 sq2, Strides3 sk1, Strides3 sk2, Strides3 sv, Strides3 so, int64_t gb, int64_t gl,
                              const int32_t* offsets, int offset, float scale, cudaStream_t stream);
-int read_tc_status_latent(unsigned int* out, int reset);
-int latent_decode_splits(int B, int R, int max_len);
-size_t latent_decode_scratch_bytes(int B, int R, int r, int max_len);
-int launch_latent_decode(const void* q1, const void* q2, const void* cache, const void* gate, void* out, void* scratch,
+BASED_WEAK int read_tc_status_latent(unsigned int* out, int reset);
+BASED_WEAK int latent_decode_splits(int B, int R, int max_len);
+BASED_WEAK size_t latent_decode_scratch_bytes(int B, int R, int r, int max_len);
+BASED_WEAK int launch_latent_decode(const void* q1, const void* q2, const void* cache, const void* gate, void* out, void* scratch,
                          size_t scratch_bytes, int B, int L, int H, int r, int rd, int max_len, Strides3 sq1, Strides3 sq2,
                          int64_t cb, int64_t cl, Strides3 so, int64_t gb, int64_t gl, const int32_t* offsets, int offset,
                          float scale, cudaStream_t stream);
 
-int launch_delta_chunk(const void* q, const void* k, const void* v, const void* z, const float* a, const float* b,
+BASED_WEAK int launch_delta_chunk(const void* q, const void* k, const void* v, const void* z, const float* a, const float* b,
                        const float* A_log, const float* dt_bias, const void* norm_w, float* state, void* out, void* scratch,
                        size_t scratch_bytes, int B, int L, int H, int Hk, int d, int dv, Strides2 sq, Strides2 sk,
                        Strides2 sv, Strides2 sz, Strides2 sg, Strides2 so, const int32_t* offsets, int offset, float eps,
                        cudaStream_t stream);
-size_t delta_chunk_scratch_bytes(int B, int L, int H, int d, int dv);
-int read_tc_status_delta(unsigned int* out, int reset);
+BASED_WEAK size_t delta_chunk_scratch_bytes(int B, int L, int H, int d, int dv);
+BASED_WEAK int read_tc_status_delta(unsigned int* out, int reset);
 
-int launch_rglru_tc(const void* u, const void* y, const void* w, const void* rb, const void* ib, const float* lam,
+BASED_WEAK int launch_rglru_tc(const void* u, const void* y, const void* w, const void* rb, const void* ib, const float* lam,
                     float* state, void* out, int B, int L, int W, int n, Strides2 su, Strides2 sy, Strides2 so,
                     const int32_t* offsets, int offset, cudaStream_t stream);
-int read_tc_status_rglru(unsigned int* out, int reset);
+BASED_WEAK int read_tc_status_rglru(unsigned int* out, int reset);
+
+// Post-norm stream, grouped attention over keys that are the values, linear attention with a constant decay.
+int launch_stream_post_norm(const void* branch, int64_t sb, const void* w, float* residual, const void* w_out, void* out,
+                            int64_t M, int D, float eps, int io_dtype, cudaStream_t stream);
+int launch_stream_embed(const int64_t* tokens, const void* table, int64_t V, float scale, const void* pos, int64_t P,
+                        float* residual, void* out, int B, int L, int D, const int32_t* offsets, int offset, int io_dtype,
+                        cudaStream_t stream);
+int launch_norm_gate(const void* x, int64_t sx, const void* w, const void* gate, int64_t sg, void* out, int64_t so, int64_t M,
+                     int D, float eps, int io_dtype, cudaStream_t stream);
+int launch_token_gate(const void* z, int64_t sz, const int64_t* tokens, const void* table, int64_t V, int64_t st,
+                      int64_t column, void* out, int64_t M, int n, int io_dtype, cudaStream_t stream);
+BASED_WEAK int launch_tied_prepare(void* q, const void* k, const void* wq, const void* wk, void* cache, float* factor, int B,
+                                   int L, int H, int G, int d, int max_len, int64_t qb, int64_t ql, int64_t kb, int64_t kl,
+                                   int64_t cb, int64_t cl, int64_t fb, int64_t fh, const int32_t* offsets, int offset,
+                                   float eps, float coef, float every, int io_dtype, cudaStream_t stream);
+BASED_WEAK int launch_lightning_recurrent(const void* q, const void* k, const void* v, const float* decay, float* state,
+                                          void* out, int B, int L, int H, int d, int dv, Strides2 sq, Strides2 sk, Strides2 sv,
+                                          Strides2 so, const int32_t* offsets, int offset, int io_dtype, cudaStream_t stream);
+BASED_WEAK int launch_lightning_step(const void* q, const void* k, const void* v, const void* gate, int64_t sx,
+                                     const float* decay, const void* norm_w, float* state, float* read, int* count, void* out,
+                                     int64_t so, int B, int H, int d, int dv, const int32_t* offsets, int offset, float eps,
+                                     int io_dtype, cudaStream_t stream);
 
 }  // namespace based

@@ -6,6 +6,8 @@
 //    s = (q1 . k1 + q2 . k2) * scale, on CUDA cores with fp32 arithmetic, any sizes.  With k1 = per-head keys and
 //    k2 = the shared rotated part it is the expanded form; with q1 = W_uk^T q and k1 = v = the cached latent
 //    (head stride 0) it is the absorbed form.  fp32 models and sizes the tensor-core kernels do not take run here.
+//    Options: groups of query heads that share a key head, a factor per key on its scores, a sink (a score of 0 without
+//    a value in the softmax sum), an output gate per head or per element.
 #include <initializer_list>
 
 #include "seq_common.cuh"
@@ -76,8 +78,9 @@ struct AttnP {
   const int32_t* offsets;
   int offset, B, L, H, d1, d2, dv;
   Strides3 sq1, sq2, sk1, sk2, sv, so;  // b, h, l
-  int64_t gb, gl;                       // gate [B, L, H]
+  int64_t gb, gl;                       // gate [B, L, H], or [B, L, H * dv] with x.gate_per_element
   float scale;
+  AttentionOptions x;
 };
 
 // One warp per (query, head).  Lanes own keys for the scores of 32 keys at a time, then output channels for the
@@ -95,10 +98,12 @@ __global__ void __launch_bounds__(kWarps * 32) split_key_attention_kernel(const 
   for (int c = lane; c < dq; c += 32) q[c] = to_float<T>(c < p.d1 ? q1[c] : q2[c - p.d1]);
   __syncwarp();
   const int nk = position0(p.offsets, p.offset, b) + l + 1;
-  const T* k1 = static_cast<const T*>(p.k1) + b * p.sk1.b + h * p.sk1.h;
-  const T* k2 = static_cast<const T*>(p.k2) + b * p.sk2.b + h * p.sk2.h;
-  const T* v = static_cast<const T*>(p.v) + b * p.sv.b + h * p.sv.h;
-  float m = -INFINITY, sum = 0.f, acc[NJ];
+  const int g = h / p.x.group;
+  const T* k1 = static_cast<const T*>(p.k1) + b * p.sk1.b + g * p.sk1.h;
+  const T* k2 = static_cast<const T*>(p.k2) + b * p.sk2.b + g * p.sk2.h;
+  const T* v = static_cast<const T*>(p.v) + b * p.sv.b + g * p.sv.h;
+  const float* kf = p.x.key_factor ? p.x.key_factor + b * p.x.fb + g * p.x.fh : nullptr;
+  float m = p.x.sink > 0.f ? 0.f : -INFINITY, sum = lane == 0 ? p.x.sink : 0.f, acc[NJ];
 #pragma unroll
   for (int j = 0; j < NJ; ++j) acc[j] = 0.f;
   for (int t0 = 0; t0 < nk; t0 += 32) {
@@ -109,7 +114,7 @@ __global__ void __launch_bounds__(kWarps * 32) split_key_attention_kernel(const 
       float x = 0.f;
       for (int c = 0; c < p.d1; ++c) x = fmaf(q[c], to_float<T>(a[c]), x);
       for (int c = 0; c < p.d2; ++c) x = fmaf(q[p.d1 + c], to_float<T>(r[c]), x);
-      s = x * p.scale;
+      s = x * p.scale * (kf ? kf[t] : 1.0f);
     }
     const float mn = fmaxf(m, warp_max(s));
     const float corr = expf(m - mn), pr = expf(s - mn);
@@ -128,11 +133,16 @@ __global__ void __launch_bounds__(kWarps * 32) split_key_attention_kernel(const 
   }
   sum = warp_sum(sum);
   float f = 1.0f / sum;
-  if (p.gate) f *= sigmoid_acc(to_float<T>(static_cast<const T*>(p.gate)[b * p.gb + l * p.gl + h]));
+  const T* gate = p.gate ? static_cast<const T*>(p.gate) + b * p.gb + l * p.gl : nullptr;
+  if (gate && !p.x.gate_per_element) { f *= sigmoid_acc(to_float<T>(gate[h])); gate = nullptr; }
+  if (gate) gate += (int64_t)h * p.dv;
   T* o = static_cast<T*>(p.out) + b * p.so.b + h * p.so.h + l * p.so.l;
 #pragma unroll
   for (int j = 0; j < NJ; ++j)
-    if (lane + 32 * j < p.dv) o[lane + 32 * j] = from_float<T>(acc[j] * f);
+    if (lane + 32 * j < p.dv) {
+      const float gf = gate ? sigmoid_acc(to_float<T>(gate[lane + 32 * j])) : 1.0f;
+      o[lane + 32 * j] = from_float<T>(acc[j] * f * gf);
+    }
 }
 
 template <typename T>
@@ -166,10 +176,11 @@ int launch_latent_prepare(const void* z, const void* norm_w, void* cache, void* 
 int launch_split_key_attention(const void* q1, const void* q2, const void* k1, const void* k2, const void* v,
                                const void* gate, void* out, int B, int L, int H, int d1, int d2, int dv, Strides3 sq1,
                                Strides3 sq2, Strides3 sk1, Strides3 sk2, Strides3 sv, Strides3 so, int64_t gb, int64_t gl,
-                               const int32_t* offsets, int offset, float scale, int io_dtype, cudaStream_t stream) {
+                               const int32_t* offsets, int offset, float scale, AttentionOptions x, int io_dtype,
+                               cudaStream_t stream) {
   if (B > 65535 || H > 65535) return BASED_ERR_TOO_LARGE;
   if (dv > 1024 || d1 + d2 > 2560) return BASED_ERR_SHAPE;
-  const AttnP p{q1, q2, k1, k2, v, gate, out, offsets, offset, B, L, H, d1, d2, dv, sq1, sq2, sk1, sk2, sv, so, gb, gl, scale};
+  const AttnP p{q1, q2, k1, k2, v, gate, out, offsets, offset, B, L, H, d1, d2, dv, sq1, sq2, sk1, sk2, sv, so, gb, gl, scale, x};
   return io_dtype == BASED_BF16 ? launch_attn_t<__nv_bfloat16>(p, stream) : launch_attn_t<float>(p, stream);
 }
 

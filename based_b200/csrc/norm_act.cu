@@ -14,6 +14,11 @@
 //    (the two norms of one x share their root mean square).  With token ids instead of a branch the row is
 //    norm(embedding[token]), so a model's first step is the same launch.
 //
+//  * the norm step of a POST-norm block (x <- x + norm(sublayer(x))): the sublayer's output is normed, added to the fp32
+//    stream, and the new stream is handed on in the activations' dtype, plain or with a norm of its own (a model's last).
+//    stream_embed starts such a stream: scaled token vector plus position vector.
+//  * norm_gate: norm(x) * w * sigmoid(gate).  token_gate: gelu(z) times a slice of the token's own vector.
+//
 // All are HBM-bound; 16-byte vector accesses, fp32 arithmetic, one read of every input.
 #include "seq_common.cuh"
 
@@ -266,6 +271,165 @@ __global__ void __launch_bounds__(NORM_THREADS) stream_norm_kernel(const StreamP
   }
 }
 
+// ---- post-norm block
+struct PostNormParams {
+  const void *branch, *w;      // [M, D] and [D]
+  float* residual;             // [M, D] fp32, updated in place
+  const void* w_out;           // [D] or null: out = norm(residual) * w_out, else out = residual
+  void* out;                   // [M, D] in T; null: nothing but the stream is written
+  int64_t sb;
+  int D;
+  float eps;
+};
+
+template <typename T, int N, int VPT>
+__global__ void __launch_bounds__(NORM_THREADS) stream_post_norm_kernel(const PostNormParams p) {
+  using seq::Pack;
+  const int64_t row = blockIdx.x;
+  const int groups = p.D / N;
+  float* res = p.residual + row * p.D;
+  const T* br = static_cast<const T*>(p.branch) + row * p.sb;
+  float z[VPT][N], r[VPT][N];
+  float ss = 0.f;
+#pragma unroll
+  for (int v = 0; v < VPT; ++v) {
+    const int g = threadIdx.x + v * NORM_THREADS;
+    if (g < groups) {
+      Pack<T, N>::load(br + (int64_t)g * N, z[v]);
+      Pack<float, N>::load(res + (int64_t)g * N, r[v]);
+#pragma unroll
+      for (int i = 0; i < N; ++i) ss = fmaf(z[v][i], z[v][i], ss);
+    }
+  }
+  float rstd = rsqrtf(block_sum(ss) / (float)p.D + p.eps);
+  ss = 0.f;
+#pragma unroll
+  for (int v = 0; v < VPT; ++v) {
+    const int g = threadIdx.x + v * NORM_THREADS;
+    if (g < groups) {
+      float w[N];
+      Pack<T, N>::load(static_cast<const T*>(p.w) + (int64_t)g * N, w);
+#pragma unroll
+      for (int i = 0; i < N; ++i) {
+        r[v][i] = fmaf(z[v][i] * rstd, w[i], r[v][i]);
+        ss = fmaf(r[v][i], r[v][i], ss);
+      }
+      Pack<float, N>::store(res + (int64_t)g * N, r[v]);
+    }
+  }
+  if (!p.out) return;
+  rstd = p.w_out ? rsqrtf(block_sum(ss) / (float)p.D + p.eps) : 1.0f;
+#pragma unroll
+  for (int v = 0; v < VPT; ++v) {
+    const int g = threadIdx.x + v * NORM_THREADS;
+    if (g < groups) {
+      if (p.w_out) {
+        float w[N];
+        Pack<T, N>::load(static_cast<const T*>(p.w_out) + (int64_t)g * N, w);
+#pragma unroll
+        for (int i = 0; i < N; ++i) r[v][i] *= rstd * w[i];
+      }
+      Pack<T, N>::store(static_cast<T*>(p.out) + row * p.D + (int64_t)g * N, r[v]);
+    }
+  }
+}
+
+struct EmbedParams {
+  const int64_t* tokens;        // [B, L]
+  const void *table, *pos;      // [V, D], [P, D]
+  float* residual;              // [B, L, D] fp32
+  void* out;                    // the same in T, or null
+  const int32_t* offsets;
+  int64_t V, P;
+  int offset, L, D;
+  float scale;
+};
+
+template <typename T, int N>
+__global__ void __launch_bounds__(NORM_THREADS) stream_embed_kernel(const EmbedParams p) {
+  using seq::Pack;
+  const int64_t row = (int64_t)blockIdx.y * p.L + blockIdx.x;
+  const int64_t tok = p.tokens[row], at = (int64_t)seq::position0(p.offsets, p.offset, blockIdx.y) + blockIdx.x;
+  const bool known = tok >= 0 && tok < p.V, placed = at >= 0 && at < p.P;   // ids and positions outside a table add nothing
+  const T* e = static_cast<const T*>(p.table) + (known ? tok : 0) * p.D;
+  const T* q = static_cast<const T*>(p.pos) + (placed ? at : 0) * p.D;
+  for (int g = threadIdx.x; g < p.D / N; g += NORM_THREADS) {
+    float a[N], b[N];
+    Pack<T, N>::load(e + (int64_t)g * N, a);
+    Pack<T, N>::load(q + (int64_t)g * N, b);
+#pragma unroll
+    for (int i = 0; i < N; ++i) a[i] = fmaf(known ? a[i] : 0.f, p.scale, placed ? b[i] : 0.f);
+    Pack<float, N>::store(p.residual + row * p.D + (int64_t)g * N, a);
+    if (p.out) Pack<T, N>::store(static_cast<T*>(p.out) + row * p.D + (int64_t)g * N, a);
+  }
+}
+
+struct NormGateParams {
+  const void *x, *w, *gate;     // [M, D] (rows sx apart), [D], [M, D] (rows sg apart)
+  void* out;                    // rows so apart
+  int64_t sx, sg, so;
+  int D;
+  float eps;
+};
+
+template <typename T, int N, int VPT>
+__global__ void __launch_bounds__(NORM_THREADS) norm_gate_kernel(const NormGateParams p) {
+  using seq::Pack;
+  const int64_t row = blockIdx.x;
+  const int groups = p.D / N;
+  const T *x = static_cast<const T*>(p.x) + row * p.sx, *gate = static_cast<const T*>(p.gate) + row * p.sg;
+  float z[VPT][N], h[VPT][N];
+  float ss = 0.f;
+#pragma unroll
+  for (int v = 0; v < VPT; ++v) {
+    const int g = threadIdx.x + v * NORM_THREADS;
+    if (g < groups) {
+      Pack<T, N>::load(x + (int64_t)g * N, z[v]);
+      Pack<T, N>::load(gate + (int64_t)g * N, h[v]);
+#pragma unroll
+      for (int i = 0; i < N; ++i) ss = fmaf(z[v][i], z[v][i], ss);
+    }
+  }
+  const float rstd = rsqrtf(block_sum(ss) / (float)p.D + p.eps);
+#pragma unroll
+  for (int v = 0; v < VPT; ++v) {
+    const int g = threadIdx.x + v * NORM_THREADS;
+    if (g < groups) {
+      float w[N];
+      Pack<T, N>::load(static_cast<const T*>(p.w) + (int64_t)g * N, w);
+#pragma unroll
+      for (int i = 0; i < N; ++i) z[v][i] *= rstd * w[i] * seq::sigmoid_t<T>(h[v][i]);
+      Pack<T, N>::store(static_cast<T*>(p.out) + row * p.so + (int64_t)g * N, z[v]);
+    }
+  }
+}
+
+struct TokenGateParams {
+  const void *z, *table;        // [M, n] (rows sz apart); table rows of st elements, the slice starts at `column`
+  const int64_t* tokens;        // [M]
+  void* out;                    // [M, n] contiguous
+  int64_t M, V, sz, st, column;
+  int n;
+};
+
+template <typename T, int N>
+__global__ void __launch_bounds__(256) token_gate_kernel(const TokenGateParams p) {
+  using seq::Pack;
+  const int per = p.n / N;
+  const int64_t i = (int64_t)blockIdx.x * 256 + threadIdx.x;
+  if (i >= p.M * per) return;
+  const int64_t row = i / per;
+  const int c = (int)(i - row * per) * N;
+  const int64_t tok = p.tokens[row];
+  const bool known = tok >= 0 && tok < p.V;
+  float z[N], e[N];
+  Pack<T, N>::load(static_cast<const T*>(p.z) + row * p.sz + c, z);
+  Pack<T, N>::load(static_cast<const T*>(p.table) + (known ? tok : 0) * p.st + p.column + c, e);
+#pragma unroll
+  for (int k = 0; k < N; ++k) z[k] = known ? seq::gelu_tanh_t<T>(z[k]) * e[k] : 0.f;
+  Pack<T, N>::store(static_cast<T*>(p.out) + row * p.n + c, z);
+}
+
 struct ActParams {
   const void *y, *gate;
   void* out;
@@ -342,7 +506,96 @@ int launch_stream_norm_t(const StreamParams& p, cudaStream_t stream) {
   return (int)cudaGetLastError();
 }
 
+template <typename T>
+int launch_post_norm_t(const PostNormParams& p, int64_t M, cudaStream_t stream) {
+  const bool vec = p.D % 8 == 0 && p.sb % 8 == 0 && aligned16(p.branch) && aligned16(p.w) && aligned16(p.residual) &&
+                   aligned16(p.w_out) && aligned16(p.out);
+  const int vpt = (p.D / (vec ? 8 : 1) + NORM_THREADS - 1) / NORM_THREADS;
+  const unsigned grid = (unsigned)M;
+  if (vec) {
+    if (vpt <= 1) stream_post_norm_kernel<T, 8, 1><<<grid, NORM_THREADS, 0, stream>>>(p);
+    else if (vpt <= 2) stream_post_norm_kernel<T, 8, 2><<<grid, NORM_THREADS, 0, stream>>>(p);
+    else if (vpt <= 4) stream_post_norm_kernel<T, 8, 4><<<grid, NORM_THREADS, 0, stream>>>(p);
+    else if (vpt <= 8) stream_post_norm_kernel<T, 8, 8><<<grid, NORM_THREADS, 0, stream>>>(p);
+    else return BASED_ERR_SHAPE;   // rows up to 8192 wide
+  } else {
+    if (vpt <= 4) stream_post_norm_kernel<T, 1, 4><<<grid, NORM_THREADS, 0, stream>>>(p);
+    else if (vpt <= 32) stream_post_norm_kernel<T, 1, 32><<<grid, NORM_THREADS, 0, stream>>>(p);
+    else return BASED_ERR_SHAPE;   // rows up to 4096 wide
+  }
+  return (int)cudaGetLastError();
+}
+
+template <typename T>
+int launch_embed_t(const EmbedParams& p, int B, cudaStream_t stream) {
+  const dim3 grid((unsigned)p.L, (unsigned)B);
+  if (p.D % 8 == 0 && aligned16(p.table) && aligned16(p.pos) && aligned16(p.residual) && aligned16(p.out))
+    stream_embed_kernel<T, 8><<<grid, NORM_THREADS, 0, stream>>>(p);
+  else
+    stream_embed_kernel<T, 1><<<grid, NORM_THREADS, 0, stream>>>(p);
+  return (int)cudaGetLastError();
+}
+
+template <typename T>
+int launch_norm_gate_t(const NormGateParams& p, int64_t M, cudaStream_t stream) {
+  const bool vec = p.D % 8 == 0 && p.sx % 8 == 0 && p.sg % 8 == 0 && p.so % 8 == 0 && aligned16(p.x) && aligned16(p.w) &&
+                   aligned16(p.gate) && aligned16(p.out);
+  const int vpt = (p.D / (vec ? 8 : 1) + NORM_THREADS - 1) / NORM_THREADS;
+  const unsigned grid = (unsigned)M;
+  if (vec) {
+    if (vpt <= 1) norm_gate_kernel<T, 8, 1><<<grid, NORM_THREADS, 0, stream>>>(p);
+    else if (vpt <= 2) norm_gate_kernel<T, 8, 2><<<grid, NORM_THREADS, 0, stream>>>(p);
+    else if (vpt <= 4) norm_gate_kernel<T, 8, 4><<<grid, NORM_THREADS, 0, stream>>>(p);
+    else if (vpt <= 8) norm_gate_kernel<T, 8, 8><<<grid, NORM_THREADS, 0, stream>>>(p);
+    else return BASED_ERR_SHAPE;
+  } else {
+    if (vpt <= 4) norm_gate_kernel<T, 1, 4><<<grid, NORM_THREADS, 0, stream>>>(p);
+    else if (vpt <= 32) norm_gate_kernel<T, 1, 32><<<grid, NORM_THREADS, 0, stream>>>(p);
+    else return BASED_ERR_SHAPE;
+  }
+  return (int)cudaGetLastError();
+}
+
+template <typename T>
+int launch_token_gate_t(const TokenGateParams& p, cudaStream_t stream) {
+  const bool vec = p.n % 8 == 0 && p.sz % 8 == 0 && p.st % 8 == 0 && p.column % 8 == 0 && aligned16(p.z) && aligned16(p.table) &&
+                   aligned16(p.out);
+  const int64_t work = p.M * (p.n / (vec ? 8 : 1)), blocks = (work + 255) / 256;
+  if (blocks > 2147483647LL) return BASED_ERR_TOO_LARGE;
+  if (vec) token_gate_kernel<T, 8><<<(unsigned)blocks, 256, 0, stream>>>(p);
+  else token_gate_kernel<T, 1><<<(unsigned)blocks, 256, 0, stream>>>(p);
+  return (int)cudaGetLastError();
+}
+
 }  // namespace
+
+int launch_stream_post_norm(const void* branch, int64_t sb, const void* w, float* residual, const void* w_out, void* out,
+                            int64_t M, int D, float eps, int io_dtype, cudaStream_t stream) {
+  if (M > 2147483647LL) return BASED_ERR_TOO_LARGE;
+  const PostNormParams p{branch, w, residual, w_out, out, sb, D, eps};
+  return io_dtype == BASED_BF16 ? launch_post_norm_t<__nv_bfloat16>(p, M, stream) : launch_post_norm_t<float>(p, M, stream);
+}
+
+int launch_stream_embed(const int64_t* tokens, const void* table, int64_t V, float scale, const void* pos, int64_t P,
+                        float* residual, void* out, int B, int L, int D, const int32_t* offsets, int offset, int io_dtype,
+                        cudaStream_t stream) {
+  if (B > 65535) return BASED_ERR_TOO_LARGE;
+  const EmbedParams p{tokens, table, pos, residual, out, offsets, V, P, offset, L, D, scale};
+  return io_dtype == BASED_BF16 ? launch_embed_t<__nv_bfloat16>(p, B, stream) : launch_embed_t<float>(p, B, stream);
+}
+
+int launch_norm_gate(const void* x, int64_t sx, const void* w, const void* gate, int64_t sg, void* out, int64_t so, int64_t M,
+                     int D, float eps, int io_dtype, cudaStream_t stream) {
+  if (M > 2147483647LL) return BASED_ERR_TOO_LARGE;
+  const NormGateParams p{x, w, gate, out, sx, sg, so, D, eps};
+  return io_dtype == BASED_BF16 ? launch_norm_gate_t<__nv_bfloat16>(p, M, stream) : launch_norm_gate_t<float>(p, M, stream);
+}
+
+int launch_token_gate(const void* z, int64_t sz, const int64_t* tokens, const void* table, int64_t V, int64_t st,
+                      int64_t column, void* out, int64_t M, int n, int io_dtype, cudaStream_t stream) {
+  const TokenGateParams p{z, table, tokens, out, M, V, sz, st, column, n};
+  return io_dtype == BASED_BF16 ? launch_token_gate_t<__nv_bfloat16>(p, stream) : launch_token_gate_t<float>(p, stream);
+}
 
 int launch_stream_norm(const int64_t* tokens, const void* table, const void* table_norm, int64_t V, const void* branch,
                        int64_t branch_stride, float mult, float* residual, const void* w1, const void* w2, void* out1,

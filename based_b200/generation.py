@@ -87,6 +87,8 @@ class GenerationMixin:
 
     # whether a call with seqlen_offset > 0 may bring more than one token (a later portion of a prompt)
     supports_portions = False
+    # positions a model has learned vectors for; None: no limit
+    max_positions = None
 
     def new_inference_params(self, batch_size: int, max_seqlen: int) -> InferenceParams:
         w = self.lm_head.weight
@@ -118,6 +120,8 @@ class GenerationMixin:
         capture), ``steps_ms`` (the steps alone).
         ``portion`` > 0 feeds the prompt that many tokens at a time (models that support portions)."""
         B, L = input_ids.shape
+        if self.max_positions is not None and L + max(max_new_tokens - 1, 0) > self.max_positions:
+            raise ValueError(f"{L} + {max_new_tokens} tokens are more than the model's {self.max_positions} positions")
         ip = self.new_inference_params(B, L + max_new_tokens)
         ev = [torch.cuda.Event(enable_timing=True) for _ in range(4)]
         out = torch.empty(B, L + max_new_tokens, dtype=input_ids.dtype, device=input_ids.device)

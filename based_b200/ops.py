@@ -928,3 +928,212 @@ def rglru_gated(u, y, gate_weight, r_bias, i_bias, lam, state, *, pos=0, out: to
             _capi.check(code, "based_rglru_gated")
             return out
     return rglru(u, y, block_gates(u, gate_weight), r_bias, i_bias, lam, state, pos=pos, out=out)
+
+
+# --------------------------------------------------------------------------- post-norm stacks
+
+def _strides_bl(t):
+    return _capi.strides(*t.stride()[:2])
+
+
+def _same_dtype(like, **tensors):
+    for name, t in tensors.items():
+        if t is not None and (t.dtype != like.dtype or t.stride(-1) != 1):
+            raise TypeError(f"{name} must be in the inputs' dtype with an innermost stride of 1")
+
+
+def stream_embed(residual: torch.Tensor, tokens: torch.Tensor, table: torch.Tensor, scale: float, pos_table: torch.Tensor,
+                 pos=0) -> torch.Tensor:
+    """Start of a stream: the fp32 ``residual [B, L, D]`` becomes ``table[token] * scale + pos_table[position]`` IN PLACE;
+    returns it in the table's dtype (fp32: the stream itself)."""
+    _need_cuda(residual, tokens, table, pos_table)
+    B, L, D = residual.shape
+    if residual.dtype != torch.float32 or not residual.is_contiguous():
+        raise TypeError("residual must be a contiguous float32 tensor")
+    if tokens.dtype != torch.int64 or tokens.shape != (B, L):
+        raise TypeError("tokens must be int64 [B, L]")
+    if table.dtype != pos_table.dtype or not (table.is_contiguous() and pos_table.is_contiguous()) or table.shape[1] != D or pos_table.shape[1] != D:
+        raise ValueError("table and pos_table must be contiguous [rows, D] of one dtype")
+    out = residual if table.dtype == torch.float32 else torch.empty(B, L, D, dtype=table.dtype, device=residual.device)
+    off, scalar = _position(pos, residual)
+    if residual.numel() > 0:
+        tokens = tokens.contiguous()
+        with torch.cuda.device(residual.device):
+            code = _capi.lib().based_stream_embed(
+                tokens.data_ptr(), table.data_ptr(), table.shape[0], float(scale), pos_table.data_ptr(), pos_table.shape[0],
+                residual.data_ptr(), None if out is residual else out.data_ptr(), B, L, D, off, scalar, _dt(table.dtype), _stream())
+        _capi.check(code, "based_stream_embed")
+    return out
+
+
+def stream_post_norm(residual: torch.Tensor, branch: torch.Tensor, weight: torch.Tensor, *,
+                     out_weight: Optional[torch.Tensor] = None, eps: float = 1e-6) -> torch.Tensor:
+    """The norm step of a post-norm block: the fp32 stream ``residual [..., D]`` becomes ``residual + rmsnorm(branch) * weight``
+    IN PLACE; returns it in the branch's dtype (fp32: the stream itself), or its RMSNorm scaled by ``out_weight``."""
+    _need_cuda(residual, branch, weight, out_weight)
+    D = residual.shape[-1]
+    if residual.dtype != torch.float32 or not residual.is_contiguous():
+        raise TypeError("residual must be a contiguous float32 tensor")
+    b2 = flat_rows(branch)
+    _same_dtype(branch, branch=branch, weight=weight, out_weight=out_weight)
+    M = residual.numel() // D if D else 0
+    if b2.shape != (M, D) or weight.shape != (D,) or (out_weight is not None and out_weight.shape != (D,)):
+        raise ValueError("branch must have the stream's shape and the weights its width")
+    alias = out_weight is None and branch.dtype == torch.float32
+    out = residual if alias else torch.empty(residual.shape, dtype=branch.dtype, device=residual.device)
+    if M > 0:
+        with torch.cuda.device(residual.device):
+            code = _capi.lib().based_stream_post_norm(b2.data_ptr(), b2.stride(0), weight.data_ptr(), residual.data_ptr(), _ptr(out_weight),
+                                                      None if alias else out.data_ptr(), M, D, float(eps), _dt(branch.dtype), _stream())
+        _capi.check(code, "based_stream_post_norm")
+    return out
+
+
+def norm_gate(x: torch.Tensor, weight: torch.Tensor, gate: torch.Tensor, eps: float, out: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """``rmsnorm(x) * weight * sigmoid(gate)`` over the last dim; column slices are fine for all but the weight."""
+    _need_cuda(x, weight, gate, out)
+    D = x.shape[-1]
+    out = torch.empty(x.shape, dtype=x.dtype, device=x.device) if out is None else out
+    _same_dtype(x, x=x, weight=weight, gate=gate, out=out)
+    x2, g2, o2 = flat_rows(x), flat_rows(gate), flat_rows(out)
+    if g2.shape != x2.shape or o2.shape != x2.shape or weight.shape != (D,):
+        raise ValueError("gate and out must have x's shape and the weight its width")
+    if x2.numel() > 0:
+        with torch.cuda.device(x.device):
+            code = _capi.lib().based_norm_gate(x2.data_ptr(), x2.stride(0), weight.data_ptr(), g2.data_ptr(), g2.stride(0), o2.data_ptr(),
+                                               o2.stride(0), x2.shape[0], D, float(eps), _dt(x.dtype), _stream())
+        _capi.check(code, "based_norm_gate")
+    return out
+
+
+def token_gate(z: torch.Tensor, tokens: torch.Tensor, table: torch.Tensor, column: int) -> torch.Tensor:
+    """``gelu_tanh(z) * table[token, column : column + n]`` for ``z [..., n]``, contiguous."""
+    _need_cuda(z, tokens, table)
+    n = z.shape[-1]
+    z2 = flat_rows(z)
+    _same_dtype(z, z=z, table=table)
+    if tokens.dtype != torch.int64 or tokens.numel() != z2.shape[0] or not 0 <= column <= table.shape[1] - n:
+        raise ValueError("tokens must be int64, one per row, and the slice inside the table")
+    out = torch.empty(z.shape, dtype=z.dtype, device=z.device)
+    if out.numel() > 0:
+        tokens = tokens.contiguous()
+        with torch.cuda.device(z.device):
+            code = _capi.lib().based_token_gate(z2.data_ptr(), z2.stride(0), tokens.data_ptr(), table.data_ptr(), table.shape[0],
+                                                table.stride(0), int(column), out.data_ptr(), z2.shape[0], n, _dt(z.dtype), _stream())
+        _capi.check(code, "based_token_gate")
+    return out
+
+
+def _check_tied(q, cache, factor, B, H, G, d):
+    if H % G or q.shape[2] != H * d or cache.shape[0] < B or cache.shape[2] != G * d or cache.dtype != q.dtype or cache.stride(2) != 1:
+        raise ValueError("q must be [B, L, H d] and cache [>= B, max_len, G d] in its dtype, H a multiple of G")
+    if factor.dtype != torch.float32 or factor.shape[0] < B or factor.shape[1:] != (G, cache.shape[1]) or factor.stride(2) != 1:
+        raise ValueError("factor must be float32 [>= B, G, max_len]")
+
+
+def tied_prepare_(q: torch.Tensor, k: torch.Tensor, q_weight: torch.Tensor, k_weight: torch.Tensor, cache: torch.Tensor,
+                  factor: torch.Tensor, *, pos=0, eps: float = 1e-6, temp_coef: float = 0.0, temp_every: float = 1.0) -> torch.Tensor:
+    """Queries ``q [B, L, H d]`` normed per head, times both norm weights and ``1 + temp_coef ln(floor((p + 1) / temp_every) +
+    1)`` IN PLACE; keys ``k [B, L, G d]`` appended to ``cache [B, max_len, G d]`` as they are, their inverse root mean squares to
+    ``factor [B, G, max_len]``."""
+    _need_cuda(q, k, q_weight, k_weight, cache, factor)
+    B, L, _ = q.shape
+    d = q_weight.shape[0]
+    H, G = q.shape[2] // d, k.shape[2] // d
+    _same_dtype(q, q=q, k=k, q_weight=q_weight, k_weight=k_weight)
+    _check_tied(q, cache, factor, B, H, G, d)
+    if k.shape != (B, L, G * d) or k_weight.shape != (d,):
+        raise ValueError("k must be [B, L, G d]")
+    off, scalar = _position(pos, q)
+    if q.numel() > 0:
+        with torch.cuda.device(q.device):
+            code = _capi.lib().based_tied_prepare(
+                q.data_ptr(), k.data_ptr(), q_weight.data_ptr(), k_weight.data_ptr(), cache.data_ptr(), factor.data_ptr(), B, L, H, G, d,
+                cache.shape[1], _strides_bl(q), _strides_bl(k), _strides_bl(cache), _strides_bl(factor), off, scalar, float(eps),
+                float(temp_coef), float(temp_every), _dt(q.dtype), _stream())
+        _capi.check(code, "based_tied_prepare")
+    return q
+
+
+def tied_attention(q: torch.Tensor, cache: torch.Tensor, factor: torch.Tensor, heads: int, scale: float, *,
+                   gate: Optional[torch.Tensor] = None, pos=0, sink: float = 0.0, out: torch.Tensor, impl: str = "auto") -> torch.Tensor:
+    """Causal attention of prepared queries ``q [B, L, H d]`` at positions ``pos ..`` over ``cache [B, max_len, G d]``, whose rows
+    are keys (scores times ``factor``) and values; ``sink`` scores of 0 without a value in each softmax sum; ``out [B, L, H d]``
+    times ``sigmoid(gate [B, L, H d])``."""
+    _need_cuda(q, cache, factor, gate, out)
+    B, L, W = q.shape
+    d = W // heads
+    G = cache.shape[2] // d
+    _same_dtype(q, q=q, gate=gate, out=out)
+    _check_tied(q, cache, factor, B, heads, G, d)
+    if out.shape != q.shape or (gate is not None and gate.shape != q.shape):
+        raise ValueError("gate and out must have q's shape")
+    off, scalar = _position(pos, q)
+    if out.numel() == 0:
+        return out
+    with torch.cuda.device(q.device):
+        code = _capi.lib().based_tied_attention(
+            q.data_ptr(), cache.data_ptr(), factor.data_ptr(), _ptr(gate), out.data_ptr(), B, L, heads, G, d, cache.shape[1],
+            _strides_bl(q), _strides_bl(cache), _strides_bl(factor), _strides_bl(gate) if gate is not None else None, _strides_bl(out),
+            off, scalar, float(scale), float(sink), _dt(q.dtype), _IMPLS[impl], None, 0, _stream())
+    _capi.check(code, "based_tied_attention")
+    return out
+
+
+def _check_lightning(state, decay, B, H, d, dv):
+    if state.shape[0] < B or state.shape[1:] != (H, d, dv) or state.dtype != torch.float32 or not state.is_contiguous():
+        raise ValueError("state must be a contiguous float32 [>= B, H, d, dv] tensor")
+    if decay.shape != (H,) or decay.dtype != torch.float32 or not decay.is_contiguous():
+        raise ValueError("decay must be float32, one per head")
+
+
+def lightning(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay: torch.Tensor, state: torch.Tensor, *, pos=0,
+              out: Optional[torch.Tensor] = None, impl: str = "auto") -> torch.Tensor:
+    """Linear attention with a constant decay per head: q, k ``[B, L, H d]``, v ``[B, L, H dv]`` before silu, ``state [B, H, d,
+    dv]`` fp32 updated IN PLACE; the read-out ``[B, L, H dv]``."""
+    _need_cuda(q, k, v, decay, state, out)
+    B, L, _ = q.shape
+    _, H, d, dv = state.shape
+    _check_lightning(state, decay, B, H, d, dv)
+    out = torch.empty(B, L, H * dv, dtype=q.dtype, device=q.device) if out is None else out
+    _same_dtype(q, q=q, k=k, v=v, out=out)
+    if q.shape[2] != H * d or k.shape != q.shape or v.shape != (B, L, H * dv) or out.shape != v.shape:
+        raise ValueError("q, k must be [B, L, H d] and v, out [B, L, H dv]")
+    off, scalar = _position(pos, q)
+    if out.numel() == 0:
+        return out
+    with torch.cuda.device(q.device):
+        code = _capi.lib().based_lightning(q.data_ptr(), k.data_ptr(), v.data_ptr(), decay.data_ptr(), state.data_ptr(), out.data_ptr(), B, L,
+                                           H, d, dv, _strides_bl(q), _strides_bl(k), _strides_bl(v), _strides_bl(out), off, scalar,
+                                           _dt(q.dtype), _IMPLS[impl], _stream())
+    _capi.check(code, "based_lightning")
+    return out
+
+
+def lightning_step(q, k, v, gate, decay, norm_weight, state, read, count, *, pos, eps: float, out: torch.Tensor) -> bool:
+    """One token per row in one launch: q, k, v, gate are column slices ``[B, .]`` of one packed projection, ``state`` is updated
+    IN PLACE, ``read [B, H dv]`` fp32 and ``count [B]`` int32 (zeros) are workspace; ``out [B, H dv]`` normed over all heads and
+    gated.  Returns False, nothing launched, for sizes it does not take."""
+    _need_cuda(q, k, v, gate, decay, norm_weight, state, read, count, out)
+    B = q.shape[0]
+    _, H, d, dv = state.shape
+    _check_lightning(state, decay, B, H, d, dv)
+    _same_dtype(q, q=q, k=k, v=v, gate=gate, norm_weight=norm_weight, out=out)
+    if q.shape[1] != H * d or k.shape != q.shape or v.shape != (B, H * dv) or gate.shape != v.shape or out.shape != v.shape or norm_weight.shape != (H * dv,):
+        raise ValueError("q, k must be [B, H d] and v, gate, out [B, H dv]")
+    if len({t.stride(0) for t in (q, k, v, gate)}) > 1 and B > 1:
+        raise ValueError("q, k, v and gate must be slices of one tensor")
+    if read.dtype != torch.float32 or read.shape[0] < B or read.shape[1] != H * dv or not read.is_contiguous() or count.dtype != torch.int32 or count.numel() < B:
+        raise ValueError("read must be contiguous float32 [>= B, H dv] and count int32 [>= B]")
+    off, scalar = _position(pos, q)
+    if B == 0:
+        return True
+    with torch.cuda.device(q.device):
+        code = _capi.lib().based_lightning_step(
+            q.data_ptr(), k.data_ptr(), v.data_ptr(), gate.data_ptr(), q.stride(0), decay.data_ptr(), norm_weight.data_ptr(),
+            state.data_ptr(), read.data_ptr(), count.data_ptr(), out.data_ptr(), out.stride(0), B, H, d, dv, off, scalar, float(eps),
+            _dt(q.dtype), _stream())
+    if code == _capi.ERR_IMPL:
+        return False
+    _capi.check(code, "based_lightning_step")
+    return True

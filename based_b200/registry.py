@@ -12,9 +12,10 @@ from .weights import SafeTensors
 _MODELS = {
     "Based": "based_b200.model:BasedLMHeadModel",
     "Razesun": "based_b200.razesun:RazesunLMHeadModel",
+    "Vubenex": "based_b200.vubenex:VubenexLMHeadModel",
 }
 # architectures whose kernels are all in one part of the library (see build.PARTS)
-_PARTS = {"Razesun": "hybrid"}
+_PARTS = {"Razesun": "hybrid", "Vubenex": "postnorm"}
 
 
 def library_part(folder: str):

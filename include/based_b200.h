@@ -525,6 +525,76 @@ int based_rglru_gated(const void* u, const void* y, const void* gate_weight, con
                       const int64_t u_strides[2], const int64_t y_strides[2], const int64_t out_strides[2],
                       const int32_t* offsets, int offset, int io_dtype, void* stream);
 
+/*
+ * ---------------------------------------------------------------------------------------------------------------
+ * Post-norm stacks (x <- x + norm(sublayer(x))) with grouped attention over keys that are the values and linear attention
+ * with a constant decay per head.  No counterpart in the reference.  Conventions as above: positions, fp32 parts, state.
+ */
+
+/*
+ * residual[b, l] = table[token] * scale + pos_table[position] (fp32, contiguous [B, L, D]), and the same in io_dtype to out
+ * (NULL: not written).  Token ids and positions outside their table add nothing.
+ */
+int based_stream_embed(const void* tokens, const void* table, int64_t V, float scale, const void* pos_table, int64_t P,
+                       void* residual, void* out, int B, int L, int D, const int32_t* offsets, int offset, int io_dtype,
+                       void* stream);
+
+/*
+ * residual += norm(branch) * weight (fp32, contiguous [M, D], in place); out (contiguous, io_dtype, may be NULL) = the new
+ * residual, or norm(residual) * out_weight when out_weight is given.
+ */
+int based_stream_post_norm(const void* branch, int64_t branch_row_stride, const void* weight, void* residual,
+                           const void* out_weight, void* out, int64_t M, int D, float eps, int io_dtype, void* stream);
+
+/* out = x / sqrt(mean(x^2) + eps) * weight * sigmoid(gate), rows of D. */
+int based_norm_gate(const void* x, int64_t x_row_stride, const void* weight, const void* gate, int64_t gate_row_stride,
+                    void* out, int64_t out_row_stride, int64_t M, int D, float eps, int io_dtype, void* stream);
+
+/* out[row] = gelu_tanh(z[row]) * table[tokens[row], column .. column + n), out contiguous [M, n]; unknown ids give zero. */
+int based_token_gate(const void* z, int64_t z_row_stride, const void* tokens, const void* table, int64_t V,
+                     int64_t table_row_stride, int64_t column, void* out, int64_t M, int n, int io_dtype, void* stream);
+
+/*
+ * Between the projections and the attention of a layer whose values are its keys before their norm: q [B, L, H d] becomes
+ * q / rms(q) * q_weight * k_weight * (1 + temp_coef ln(floor((p + 1) / temp_every) + 1)) in place; k [B, L, G d] is copied to
+ * the cache rows of its positions and 1 / rms(k) (eps inside the root) to factor [B, G, max_len] fp32.  Strides are
+ * (batch, token), factor's (batch, key head); heads of d contiguous.  Positions past max_len are skipped (device offsets)
+ * or rejected (scalar).  d <= 512.
+ */
+int based_tied_prepare(void* q, const void* k, const void* q_weight, const void* k_weight, void* cache, void* factor, int B,
+                       int L, int H, int G, int d, int max_len, const int64_t q_strides[2], const int64_t k_strides[2],
+                       const int64_t cache_strides[2], const int64_t factor_strides[2], const int32_t* offsets, int offset,
+                       float eps, float temp_coef, float temp_every, int io_dtype, void* stream);
+
+/*
+ * Causal attention of prepared queries over that cache: score = (q . k) * factor * scale, values = k, query head h reads key
+ * head h / (H / G), `sink` scores of 0 without a value in every softmax sum; out [B, L, H d], times sigmoid(gate) element by
+ * element when gate [B, L, H d] is given.  Query l sees keys 0 .. offset + l.  AUTO picks by dtype, sizes and the number of
+ * query rows.  scratch: based_tied_attention_scratch_bytes bytes, 16-byte aligned (NULL when that is 0).
+ */
+int based_tied_attention(const void* q, const void* cache, const void* factor, const void* gate, void* out, int B, int L, int H,
+                         int G, int d, int max_len, const int64_t q_strides[2], const int64_t cache_strides[2],
+                         const int64_t factor_strides[2], const int64_t gate_strides[2], const int64_t out_strides[2],
+                         const int32_t* offsets, int offset, float scale, float sink, int io_dtype, int impl, void* scratch,
+                         size_t scratch_bytes, void* stream);
+
+/*
+ * S <- decay S + silu(k) silu(v)^T, out = S^T silu(q) over the tokens of a call: q, k [B, L, H d], v [B, L, H dv] before silu
+ * (strides batch, token; heads contiguous), decay [H] fp32, state [B, H, d, dv] fp32 updated, out [B, L, H dv].  d <= 512.
+ */
+int based_lightning(const void* q, const void* k, const void* v, const void* decay, void* state, void* out, int B, int L, int H,
+                    int d, int dv, const int64_t q_strides[2], const int64_t k_strides[2], const int64_t v_strides[2],
+                    const int64_t out_strides[2], const int32_t* offsets, int offset, int io_dtype, int impl, void* stream);
+
+/*
+ * One token per row, from slices of the packed projection (q, k, v, gate: rows x_row_stride apart) to the gated output in one
+ * launch: out = norm over all heads of the read-out * norm_weight * sigmoid(gate).  read [B, H dv] fp32 is workspace, count
+ * [B] int32 is zero before the first call and zero again after every call.  BASED_ERR_IMPL for dv % 4 or d above 1024.
+ */
+int based_lightning_step(const void* q, const void* k, const void* v, const void* gate, int64_t x_row_stride, const void* decay,
+                         const void* norm_weight, void* state, void* read, void* count, void* out, int64_t out_row_stride, int B,
+                         int H, int d, int dv, const int32_t* offsets, int offset, float eps, int io_dtype, void* stream);
+
 #ifdef __cplusplus
 }
 #endif
