@@ -14,6 +14,8 @@ BASED_BF16 = 1
 IMPL_AUTO = 0
 IMPL_SIMT = 1
 IMPL_TCGEN05 = 2
+IMPL_DECODE = 3
+TIED_DECODE_ROWS = 64
 ERR_IMPL = -5
 
 _I64P = POINTER(c_int64)
@@ -76,7 +78,8 @@ SIGNATURES = {
     "based_token_gate": (c_int, [c_void_p, c_int64, c_void_p, c_void_p] + [c_int64] * 3 + [c_void_p, c_int64, c_int, c_int, c_void_p]),
     "based_tied_prepare": (c_int, [c_void_p] * 6 + [c_int] * 6 + [_I64P] * 4 + _POS + [c_float] * 3 + [c_int, c_void_p]),
     "based_tied_attention": (c_int, [c_void_p] * 5 + [c_int] * 6 + [_I64P] * 5 + _POS
-                             + [c_float, c_float, c_int, c_int, c_void_p, ctypes.c_size_t, c_void_p]),
+                             + [c_float, c_float, c_int, c_int, c_void_p, ctypes.c_size_t, c_void_p, c_int, c_void_p]),
+    "based_tied_attention_scratch_bytes": (ctypes.c_size_t, [c_int] * 6),
     "based_lightning": (c_int, [c_void_p] * 6 + [c_int] * 5 + [_I64P] * 4 + _POS + [c_int, c_int, c_void_p]),
     "based_lightning_step": (c_int, [c_void_p] * 4 + [c_int64] + [c_void_p] * 6 + [c_int64] + [c_int] * 4 + _POS
                              + [c_float, c_int, c_void_p]),

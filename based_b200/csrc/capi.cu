@@ -36,14 +36,16 @@ const char* based_error_string(int code) {
 }
 
 int based_read_status(unsigned int* out, int reset) {
-  unsigned int a = 0, b = 0, c = 0, d = 0, e = 0, f = 0;
+  unsigned int a = 0, b = 0, c = 0, d = 0, e = 0, f = 0, g = 0, h = 0;
   int rc = read_tc_status ? read_tc_status(&a, reset) : 0;
   if (rc == 0 && read_tc_status_swa) rc = read_tc_status_swa(&b, reset);
   if (rc == 0 && read_tp_status) rc = read_tp_status(&c, reset);
   if (rc == 0 && read_tc_status_latent) rc = read_tc_status_latent(&d, reset);
   if (rc == 0 && read_tc_status_delta) rc = read_tc_status_delta(&e, reset);
   if (rc == 0 && read_tc_status_rglru) rc = read_tc_status_rglru(&f, reset);
-  if (out) *out = a | b | c | d | e | f;
+  if (rc == 0 && read_tc_status_tied) rc = read_tc_status_tied(&g, reset);
+  if (rc == 0 && read_tc_status_lightning) rc = read_tc_status_lightning(&h, reset);
+  if (out) *out = a | b | c | d | e | f | g | h;
   return rc;
 }
 
@@ -634,7 +636,7 @@ int based_tied_attention(const void* q, const void* cache, const void* factor, c
                          int G, int d, int max_len, const int64_t q_strides[2], const int64_t cache_strides[2],
                          const int64_t factor_strides[2], const int64_t gate_strides[2], const int64_t out_strides[2],
                          const int32_t* offsets, int offset, float scale, float sink, int io_dtype, int impl, void* scratch,
-                         size_t scratch_bytes, void* stream) {
+                         size_t scratch_bytes, void* count, int count_len, void* stream) {
   if (!q || !cache || !factor || !out || (gate && !gate_strides)) return BASED_ERR_NULL;
   if (!q_strides || !cache_strides || !factor_strides || !out_strides) return BASED_ERR_NULL;
   if (!dtype_ok(io_dtype)) return BASED_ERR_DTYPE;
@@ -649,10 +651,32 @@ int based_tied_attention(const void* q, const void* cache, const void* factor, c
   x.sink = sink;
   x.gate_per_element = 1;
   const int64_t gb = gate ? gate_strides[0] : 0, gl = gate ? gate_strides[1] : 0;
+  const bool autosel = impl == BASED_IMPL_AUTO;
+  if (io_dtype != BASED_BF16 && !autosel && impl != BASED_IMPL_SIMT) return BASED_ERR_IMPL;
+  if (io_dtype == BASED_BF16 && (impl == BASED_IMPL_DECODE || (autosel && (offsets || L * (H / G) <= BASED_TIED_DECODE_ROWS)))) {
+    if (!launch_tied_decode) return BASED_ERR_IMPL;
+    const int rc = launch_tied_decode(q, cache, x.key_factor, gate, out, scratch, scratch_bytes, static_cast<int*>(count), count_len, B,
+                                      L, H, G, d, max_len, q_strides[0], q_strides[1], cache_strides[0], cache_strides[1], x.fb,
+                                      x.fh, gb, gl, out_strides[0], out_strides[1], offsets, offset, scale, sink, st);
+    if (!(autosel && rc == BASED_ERR_IMPL)) return rc;
+  }
+  if (io_dtype == BASED_BF16 && !offsets && (impl == BASED_IMPL_TCGEN05 || autosel)) {
+    if (!launch_tied_prefill_tc) return BASED_ERR_IMPL;
+    const int rc = launch_tied_prefill_tc(q, cache, x.key_factor, gate, out, B, L, H, G, d, q_strides[0], q_strides[1],
+                                          cache_strides[0], cache_strides[1], x.fb, x.fh, gb, gl, out_strides[0],
+                                          out_strides[1], offset, scale, sink, st);
+    if (!(autosel && rc == BASED_ERR_IMPL)) return rc;
+  }
+  if (!autosel && impl != BASED_IMPL_SIMT) return BASED_ERR_IMPL;
   const Strides3 sq{q_strides[0], d, q_strides[1]}, sc{cache_strides[0], d, cache_strides[1]}, so{out_strides[0], d, out_strides[1]};
   if (!launch_split_key_attention) return BASED_ERR_IMPL;
   return launch_split_key_attention(q, q, cache, cache, cache, gate, out, B, L, H, d, 0, d, sq, sq, sc, sc, sc, so, gb, gl,
                                     offsets, offset, scale, x, io_dtype, st);
+}
+
+size_t based_tied_attention_scratch_bytes(int B, int L, int H, int G, int d, int max_len) {
+  if (B <= 0 || L <= 0 || H <= 0 || G <= 0 || H % G || d <= 0 || max_len <= 0 || !tied_decode_scratch_bytes) return 0;
+  return tied_decode_scratch_bytes(B, L * (H / G), G, d, max_len);
 }
 
 int based_lightning(const void* q, const void* k, const void* v, const void* decay, void* state, void* out, int B, int L, int H,
@@ -662,6 +686,15 @@ int based_lightning(const void* q, const void* k, const void* v, const void* dec
   if (!dtype_ok(io_dtype)) return BASED_ERR_DTYPE;
   if (B < 0 || L < 0 || H <= 0 || d <= 0 || d > 512 || dv <= 0 || offset < 0) return BASED_ERR_SHAPE;
   if (B == 0 || L == 0) return BASED_OK;
+  // AUTO: chunks for bf16 from a handful of tokens on, else token by token
+  const bool autosel = impl == BASED_IMPL_AUTO;
+  if (impl == BASED_IMPL_TCGEN05 || (autosel && io_dtype == BASED_BF16 && L >= 16)) {
+    if (io_dtype != BASED_BF16 || !launch_lightning_tc) return BASED_ERR_IMPL;
+    const int rc = launch_lightning_tc(q, k, v, static_cast<const float*>(decay), static_cast<float*>(state), out, B, L, H, d, dv,
+                                       s2(q_strides), s2(k_strides), s2(v_strides), s2(out_strides), offsets, offset,
+                                       static_cast<cudaStream_t>(stream));
+    if (!(autosel && rc == BASED_ERR_IMPL)) return rc;
+  }
   if (!launch_lightning_recurrent) return BASED_ERR_IMPL;
   return launch_lightning_recurrent(q, k, v, static_cast<const float*>(decay), static_cast<float*>(state), out, B, L, H, d, dv,
                                     s2(q_strides), s2(k_strides), s2(v_strides), s2(out_strides), offsets, offset, io_dtype,

@@ -198,9 +198,24 @@ BASED_WEAK int launch_tied_prepare(void* q, const void* k, const void* wq, const
                                    int L, int H, int G, int d, int max_len, int64_t qb, int64_t ql, int64_t kb, int64_t kl,
                                    int64_t cb, int64_t cl, int64_t fb, int64_t fh, const int32_t* offsets, int offset,
                                    float eps, float coef, float every, int io_dtype, cudaStream_t stream);
+BASED_WEAK int launch_tied_prefill_tc(const void* q, const void* cache, const float* factor, const void* gate, void* out, int B,
+                                      int L, int H, int G, int d, int64_t qb, int64_t ql, int64_t cb, int64_t cl, int64_t fb,
+                                      int64_t fh, int64_t gb, int64_t gl, int64_t ob, int64_t ol, int offset, float scale,
+                                      float sink, cudaStream_t stream);
+BASED_WEAK int read_tc_status_tied(unsigned int* out, int reset);
+BASED_WEAK size_t tied_decode_scratch_bytes(int B, int R, int G, int d, int max_len);
+BASED_WEAK int launch_tied_decode(const void* q, const void* cache, const float* factor, const void* gate, void* out,
+                                  void* scratch, size_t scratch_bytes, int* count, int count_len, int B, int L, int H, int G,
+                                  int d, int max_len, int64_t qb, int64_t ql, int64_t cb, int64_t cl, int64_t fb, int64_t fh,
+                                  int64_t gb, int64_t gl, int64_t ob, int64_t ol, const int32_t* offsets, int offset,
+                                  float scale, float sink, cudaStream_t stream);
 BASED_WEAK int launch_lightning_recurrent(const void* q, const void* k, const void* v, const float* decay, float* state,
                                           void* out, int B, int L, int H, int d, int dv, Strides2 sq, Strides2 sk, Strides2 sv,
                                           Strides2 so, const int32_t* offsets, int offset, int io_dtype, cudaStream_t stream);
+BASED_WEAK int launch_lightning_tc(const void* q, const void* k, const void* v, const float* decay, float* state, void* out, int B,
+                                   int L, int H, int d, int dv, Strides2 sq, Strides2 sk, Strides2 sv, Strides2 so,
+                                   const int32_t* offsets, int offset, cudaStream_t stream);
+BASED_WEAK int read_tc_status_lightning(unsigned int* out, int reset);
 BASED_WEAK int launch_lightning_step(const void* q, const void* k, const void* v, const void* gate, int64_t sx,
                                      const float* decay, const void* norm_w, float* state, float* read, int* count, void* out,
                                      int64_t so, int B, int H, int d, int dv, const int32_t* offsets, int offset, float eps,

@@ -1,0 +1,382 @@
+// Linear attention with one constant decay g per head over prompts and portions, in chunks of 128 tokens on the sm_100a
+// tensor cores.  With q, k, v = silu of the projections, i, j places in a chunk of n tokens, S0 the state before it:
+//   o_i = g^(i+1) S0^T q_i + sum_{j <= i} g^(i-j) (q_i . k_j) v_j
+//   S   = g^n S0 + sum_j k_j (g^(n-1-j) v_j)^T
+// One CTA walks the chunks of one (batch, head) (or of a slice of its value columns) with the state as a TMEM accumulator:
+//   warps 0-3    scores: (Q K^T)_ij times g^(i-j) to P (bf16, in the scores' columns); read-out: O = P V + g^(i+1) Q S0
+//   warps 4-7    state: S0 (TMEM) to the bf16 operand of Q S0, and g^n S0 back to TMEM
+//   warp 8       MMA issue
+//   warps 9-24   loads: raw projections of the next chunk to registers, silu there, then to shared memory when the chunk
+//                before is done - the registers are the second buffer, shared memory holds one chunk
+// 32-bit in the recurrence: the state is the fp32 accumulator and is scaled in fp32; g^(n-1-j) v_j enters as a bf16 pair
+// hi + lo (16 mantissa bits) against k as the activation stored it.  Scores and decays are fp32 until P, and nothing feeds
+// the read-out back.
+#include <initializer_list>
+#include <mutex>
+
+#include "seq_common.cuh"
+#include "tcgen05.cuh"
+#include "tma.cuh"
+
+namespace based {
+
+__device__ unsigned int g_tc_status_lightning = 0;
+
+namespace {
+
+using namespace tc;
+using bf16 = __nv_bfloat16;
+
+constexpr int C = 128;                      // tokens per chunk
+constexpr int kLoaders = 512, NT = 9 * 32 + kLoaders;
+constexpr int kItems = C * 16 / kLoaders;   // 16-byte pieces per thread and tensor at 128 columns
+constexpr uint32_t kAtom = 128 * 128;       // bytes of 128 rows x 64 columns
+
+struct Params {
+  const bf16 *q, *k, *v;
+  const float* decay;
+  float* state;
+  bf16* out;
+  const int32_t* offsets;
+  int64_t qb, ql, kb, kl, vb, vl, ob, ol;
+  int offset, L, H, d, dv, cols;            // cols: value columns per CTA
+  unsigned int* status;
+};
+
+__device__ __forceinline__ float ex2(float x) { float r; asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(x)); return r; }
+__device__ __forceinline__ float rcp(float x) { float r; asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(x)); return r; }
+
+// silu of two packed values; both sigmoids from one reciprocal
+__device__ __forceinline__ uint32_t silu2(uint32_t w) {
+  const float a = seq::bf16_lo(w), b = seq::bf16_hi(w);
+  const float ea = 1.f + ex2(fminf(a * -1.4426950408889634f, 60.f)), eb = 1.f + ex2(fminf(b * -1.4426950408889634f, 60.f));
+  const float r = rcp(ea * eb);
+  return pack_bf16(a * (r * eb), b * (r * ea));
+}
+
+__global__ void __launch_bounds__(NT, 1) lightning_tc_kernel(const __grid_constant__ Params p) {
+  extern __shared__ uint8_t smem_raw[];
+  uint8_t* smem = smem_raw + ((1024u - (smem_u32(smem_raw) & 1023u)) & 1023u);
+  const uint32_t sb = smem_u32(smem);
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  const int h = blockIdx.x, b = blockIdx.y, col0 = blockIdx.z * p.cols;
+  const int cols = min(p.cols, p.dv - col0);
+  const int nc = (p.L + C - 1) / C;
+  const int aq = (p.d + 63) / 64, av = (p.cols + 63) / 64;
+  // shared memory: Q, K (always two atoms: its transpose is a 128-row operand), V, hi and lo of the decayed V, S0
+  const uint32_t SM_K = aq * kAtom, SM_V = SM_K + 2 * kAtom, SM_W = SM_V + av * kAtom, SM_S = SM_W + 2 * av * kAtom,
+                 SM_POW = SM_S + av * kAtom, SM_BAR = SM_POW + 132 * 4;
+  float* pw = reinterpret_cast<float*>(smem + SM_POW);   // g^0 .. g^128
+  const uint32_t B_FULL = sb + SM_BAR, B_A = B_FULL + 8, B_P = B_FULL + 16, B_S0 = B_FULL + 24, B_S = B_FULL + 32,
+                 B_O = B_FULL + 40, B_OF = B_FULL + 48;
+  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(smem + SM_BAR + 56);
+  volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_slot + 1);
+  if (tid == 0) {
+    mbar_init(B_FULL, kLoaders); mbar_init(B_A, 1); mbar_init(B_P, 128); mbar_init(B_S0, 128); mbar_init(B_S, 1);
+    mbar_init(B_O, 1); mbar_init(B_OF, 128);
+    *abort_flag = 0;
+    fence_mbar_init();
+  }
+  if (tid <= C) {   // powers by squaring
+    float r = 1.f, x = p.decay[h];
+    for (int e = tid; e > 0; e >>= 1) { if (e & 1) r *= x; x *= x; }
+    pw[tid] = r;
+  }
+  for (uint32_t i = tid * 16; i < 2 * kAtom; i += NT * 16) *reinterpret_cast<uint4*>(smem + SM_K + i) = make_uint4(0, 0, 0, 0);
+  fence_proxy_async();
+  if (warp == 8) tmem_alloc(smem_u32(tmem_slot), 512);
+  fence_before_sync();
+  __syncthreads();
+  fence_after_sync();
+  const uint32_t tmem = *tmem_slot;
+  constexpr uint32_t TM_A = 0, TM_S = 128, TM_O = 256, TM_I = 384;
+
+  if (warp >= 9) {
+    // ---------------- loads, silu, operands
+    const int t = tid - 9 * 32;
+    const int cq = p.d / 8, cv = cols / 8;
+    const uint32_t iq = ((1u << 20) + cq - 1) / cq, iv = ((1u << 20) + cv - 1) / cv;   // exact quotients for the indices used
+    const bf16* q = p.q + b * p.qb + (int64_t)h * p.d;
+    const bf16* k = p.k + b * p.kb + (int64_t)h * p.d;
+    const bf16* v = p.v + b * p.vb + (int64_t)h * p.dv + col0;
+    uint4 rq[kItems], rk[kItems], rv[kItems];
+    auto fetch = [&](int c) {
+      const int l0 = c * C;
+#pragma unroll
+      for (int i = 0; i < kItems; ++i) {
+        const int e = t + i * kLoaders, row = (int)((e * iq) >> 20), cc = (e - row * cq) * 8, l = l0 + row;
+        const bool ok = row < C && l < p.L;
+        rq[i] = ok ? __ldg(reinterpret_cast<const uint4*>(q + (int64_t)l * p.ql + cc)) : make_uint4(0, 0, 0, 0);
+        rk[i] = ok ? __ldg(reinterpret_cast<const uint4*>(k + (int64_t)l * p.kl + cc)) : make_uint4(0, 0, 0, 0);
+      }
+#pragma unroll
+      for (int i = 0; i < kItems; ++i) {
+        const int e = t + i * kLoaders, row = (int)((e * iv) >> 20), cc = (e - row * cv) * 8, l = l0 + row;
+        rv[i] = row < C && l < p.L ? __ldg(reinterpret_cast<const uint4*>(v + (int64_t)l * p.vl + cc)) : make_uint4(0, 0, 0, 0);
+      }
+    };
+    auto act = [&](uint4& x) { x.x = silu2(x.x); x.y = silu2(x.y); x.z = silu2(x.z); x.w = silu2(x.w); };
+    fetch(0);
+    for (int c = 0; c < nc; ++c) {
+#pragma unroll
+      for (int i = 0; i < kItems; ++i) act(rq[i]);
+#pragma unroll
+      for (int i = 0; i < kItems; ++i) act(rk[i]);
+#pragma unroll
+      for (int i = 0; i < kItems; ++i) act(rv[i]);
+      if (c > 0) mbar_wait_bounded(B_O, (c - 1) & 1, abort_flag, p.status, 1u << 0);
+      const int n = min(C, p.L - c * C);
+#pragma unroll
+      for (int i = 0; i < kItems; ++i) {
+        const int e = t + i * kLoaders, row = (int)((e * iq) >> 20), cc = e - row * cq;
+        if (row < C) {
+          const uint32_t at = (cc >> 3) * kAtom + tma::sw128_offset(row, cc & 7);
+          *reinterpret_cast<uint4*>(smem + at) = rq[i];
+          *reinterpret_cast<uint4*>(smem + SM_K + at) = rk[i];
+        }
+      }
+#pragma unroll
+      for (int i = 0; i < kItems; ++i) {
+        const int e = t + i * kLoaders, row = (int)((e * iv) >> 20), cc = e - row * cv;
+        if (row < C) {
+          const uint32_t at = (cc >> 3) * kAtom + tma::sw128_offset(row, cc & 7);
+          *reinterpret_cast<uint4*>(smem + SM_V + at) = rv[i];
+          const float f = row < n ? pw[n - 1 - row] : 0.f;
+          uint32_t hi[4], lo[4];
+          const uint32_t w[4] = {rv[i].x, rv[i].y, rv[i].z, rv[i].w};
+#pragma unroll
+          for (int m = 0; m < 4; ++m) {
+            const float x = seq::bf16_lo(w[m]) * f, y = seq::bf16_hi(w[m]) * f;
+            hi[m] = pack_bf16(x, y);
+            lo[m] = pack_bf16(x - seq::bf16_lo(hi[m]), y - seq::bf16_hi(hi[m]));
+          }
+          *reinterpret_cast<uint4*>(smem + SM_W + at) = make_uint4(hi[0], hi[1], hi[2], hi[3]);
+          *reinterpret_cast<uint4*>(smem + SM_W + av * kAtom + at) = make_uint4(lo[0], lo[1], lo[2], lo[3]);
+        }
+      }
+      fence_proxy_async();
+      mbar_arrive(B_FULL);
+      if (c + 1 < nc) fetch(c + 1);
+    }
+  } else if (warp == 8) {
+    // ---------------- MMA issue (converged warp, one elected lane)
+    const uint32_t tm = __shfl_sync(0xffffffffu, tmem, 0);
+    const bool leader = elect_one_sync();
+    const uint32_t id_a = make_idesc_bf16(128, C, 0, 0), id_i = make_idesc_bf16(128, cols, 0, 1), id_s = make_idesc_bf16(128, cols, 1, 1);
+    const uint64_t dk_t = make_smem_desc_sw128(sb + SM_K, kAtom, 1024), dv_ = make_smem_desc_sw128(sb + SM_V, kAtom, 1024);
+    const uint64_t dw0 = make_smem_desc_sw128(sb + SM_W, kAtom, 1024), dw1 = make_smem_desc_sw128(sb + SM_W + av * kAtom, kAtom, 1024);
+    const uint64_t ds = make_smem_desc_sw128(sb + SM_S, kAtom, 1024);
+    const int ks = p.d / 16;
+    for (int c = 0; c < nc; ++c) {
+      const uint32_t ph = c & 1;
+      mbar_wait_bounded(B_FULL, ph, abort_flag, p.status, 1u << 1);
+      fence_after_sync();
+      for (int k = 0; k < ks; ++k) {   // 16 columns are 32 bytes of a row, four to an atom
+        const uint32_t at = (k >> 2) * kAtom + (k & 3) * 32;
+        const uint64_t da = make_smem_desc_sw128(sb + at, 16, 1024), db = make_smem_desc_sw128(sb + SM_K + at, 16, 1024);
+        if (leader) mma_ss(tm + TM_A, da, db, id_a, k > 0 ? 1u : 0u);
+      }
+      if (leader) mma_commit(B_A);
+      __syncwarp();
+      mbar_wait_bounded(B_S0, ph, abort_flag, p.status, 1u << 2);
+      if (c > 0) mbar_wait_bounded(B_OF, ph ^ 1, abort_flag, p.status, 1u << 3);
+      fence_after_sync();
+      for (int k = 0; k < ks; ++k) {   // 16 rows of S0 are 2048 bytes
+        const uint64_t da = make_smem_desc_sw128(sb + (k >> 2) * kAtom + (k & 3) * 32, 16, 1024);
+        if (leader) mma_ss(tm + TM_I, da, ds + 128 * k, id_i, k > 0 ? 1u : 0u);
+      }
+#pragma unroll
+      for (int k = 0; k < C / 16; ++k) {
+        if (leader) mma_ss(tm + TM_S, dk_t + 128 * k, dw0 + 128 * k, id_s, 1u);
+        if (leader) mma_ss(tm + TM_S, dk_t + 128 * k, dw1 + 128 * k, id_s, 1u);
+      }
+      if (leader) mma_commit(B_S);
+      __syncwarp();
+      mbar_wait_bounded(B_P, ph, abort_flag, p.status, 1u << 4);
+      fence_after_sync();
+#pragma unroll
+      for (int k = 0; k < C / 16; ++k)
+        if (leader) mma_ts(tm + TM_O, tm + TM_A + 8 * k, dv_ + 128 * k, id_i, k > 0 ? 1u : 0u);
+      if (leader) mma_commit(B_O);     // read-out complete, and every operand of this chunk read
+      __syncwarp();
+    }
+  } else if (warp >= 4) {
+    // ---------------- state: one row (key dimension) per thread
+    const int row = tid - 128;
+    const uint32_t ts = tmem + ((uint32_t)((warp & 3) * 32) << 16) + TM_S;
+    const bool live = row < p.d, fresh = seq::position0(p.offsets, p.offset, b) == 0;
+    float* st = p.state + (((int64_t)b * p.H + h) * p.d + (live ? row : 0)) * p.dv + col0;
+    for (int c = 0; c <= nc; ++c) {
+      const float g = c < nc ? pw[min(C, p.L - c * C)] : 0.f;
+      if (c > 0) {
+        mbar_wait_bounded(B_S, (c - 1) & 1, abort_flag, p.status, 1u << 5);
+        fence_after_sync();
+      }
+      for (int x = 0; x < cols; x += 16) {
+        uint32_t s[16];
+        if (c > 0) {
+          tmem_ld16(ts + x, s);
+          tmem_ld_wait();
+        } else {
+#pragma unroll
+          for (int i = 0; i < 16; i += 4) {
+            float4 f = make_float4(0.f, 0.f, 0.f, 0.f);
+            if (live && !fresh) f = *reinterpret_cast<const float4*>(st + x + i);
+            s[i] = __float_as_uint(f.x); s[i + 1] = __float_as_uint(f.y); s[i + 2] = __float_as_uint(f.z); s[i + 3] = __float_as_uint(f.w);
+          }
+        }
+        if (c == nc) {
+          if (live) {
+#pragma unroll
+            for (int i = 0; i < 16; i += 4)
+              *reinterpret_cast<float4*>(st + x + i) = make_float4(__uint_as_float(s[i]), __uint_as_float(s[i + 1]), __uint_as_float(s[i + 2]), __uint_as_float(s[i + 3]));
+          }
+        } else {
+#pragma unroll
+          for (int i = 0; i < 16; i += 8) {
+            uint32_t w[4];
+#pragma unroll
+            for (int m = 0; m < 4; ++m) w[m] = pack_bf16(__uint_as_float(s[i + 2 * m]), __uint_as_float(s[i + 2 * m + 1]));
+            const int cc = (x + i) >> 3;
+            *reinterpret_cast<uint4*>(smem + SM_S + (cc >> 3) * kAtom + tma::sw128_offset(row, cc & 7)) = make_uint4(w[0], w[1], w[2], w[3]);
+          }
+#pragma unroll
+          for (int i = 0; i < 16; ++i) s[i] = __float_as_uint(__uint_as_float(s[i]) * g);
+          tmem_st16(ts + x, s);
+        }
+      }
+      if (c < nc) {
+        tmem_st_wait();
+        fence_proxy_async();
+        fence_before_sync();
+        mbar_arrive(B_S0);
+      }
+    }
+  } else {
+    // ---------------- scores and read-out: one token per thread
+    const int i = tid;
+    const uint32_t tl = tmem + ((uint32_t)(warp * 32) << 16);
+    bf16* out = p.out + b * p.ob + (int64_t)h * p.dv + col0;
+    for (int c = 0; c < nc; ++c) {
+      mbar_wait_bounded(B_A, c & 1, abort_flag, p.status, 1u << 6);
+      fence_after_sync();
+#pragma unroll
+      for (int x = 0; x < 4; ++x) {   // 32 columns at a time: before, on and after this warp's diagonal block
+        uint32_t w[16];
+        if (x <= warp) {
+          uint32_t r[32];
+          tmem_ld32(tl + TM_A + 32 * x, r);
+          tmem_ld_wait();
+          if (x < warp) {             // g^(i-j) = g^(i-last column) g^(last column-j): no power of it is negative
+            const float f = pw[i - 32 * x - 31];
+#pragma unroll
+            for (int j = 0; j < 16; ++j)
+              w[j] = pack_bf16(__uint_as_float(r[2 * j]) * (f * pw[31 - 2 * j]), __uint_as_float(r[2 * j + 1]) * (f * pw[30 - 2 * j]));
+          } else {
+#pragma unroll
+            for (int j = 0; j < 16; ++j) {
+              const int u = lane - 2 * j;
+              const float f0 = u >= 0 ? pw[u] : 0.f, f1 = u >= 1 ? pw[u - 1] : 0.f;
+              w[j] = pack_bf16(u >= 0 ? __uint_as_float(r[2 * j]) * f0 : 0.f, u >= 1 ? __uint_as_float(r[2 * j + 1]) * f1 : 0.f);
+            }
+          }
+        } else {
+#pragma unroll
+          for (int j = 0; j < 16; ++j) w[j] = 0u;
+        }
+        // P of columns 32 x .. goes to columns 16 x ..: already read by this thread
+        tmem_st16(tl + TM_A + 16 * x, w);
+      }
+      tmem_st_wait();
+      fence_before_sync();
+      mbar_arrive(B_P);
+      mbar_wait_bounded(B_O, c & 1, abort_flag, p.status, 1u << 7);
+      fence_after_sync();
+      const float g = pw[i + 1];
+      const bool live = c * C + i < p.L;
+      bf16* o = out + (int64_t)(c * C + i) * p.ol;
+      for (int x = 0; x < cols; x += 16) {
+        uint32_t r0[16], r1[16];
+        tmem_ld16(tl + TM_O + x, r0);
+        tmem_ld16(tl + TM_I + x, r1);
+        tmem_ld_wait();
+        if (live) {
+          uint32_t w[8];
+#pragma unroll
+          for (int m = 0; m < 8; ++m)
+            w[m] = pack_bf16(fmaf(__uint_as_float(r1[2 * m]), g, __uint_as_float(r0[2 * m])),
+                             fmaf(__uint_as_float(r1[2 * m + 1]), g, __uint_as_float(r0[2 * m + 1])));
+          *reinterpret_cast<uint4*>(o + x) = make_uint4(w[0], w[1], w[2], w[3]);
+          *reinterpret_cast<uint4*>(o + x + 8) = make_uint4(w[4], w[5], w[6], w[7]);
+        }
+      }
+      fence_before_sync();
+      mbar_arrive(B_OF);
+    }
+  }
+  __syncwarp();
+  fence_before_sync();
+  __syncthreads();
+  if (warp == 8) {
+    fence_after_sync();
+    tmem_dealloc(tmem, 512);
+  }
+}
+
+}  // namespace
+
+int read_tc_status_lightning(unsigned int* out, int reset) {
+  unsigned int v = 0;
+  cudaError_t e = cudaMemcpyFromSymbol(&v, g_tc_status_lightning, sizeof(v));
+  if (e != cudaSuccess) return (int)e;
+  if (out) *out = v;
+  if (reset && v != 0) {
+    v = 0;
+    e = cudaMemcpyToSymbol(g_tc_status_lightning, &v, sizeof(v));
+  }
+  return (int)e;
+}
+
+// BASED_ERR_IMPL: sizes or strides this kernel does not take.
+int launch_lightning_tc(const void* q, const void* k, const void* v, const float* decay, float* state, void* out, int B, int L,
+                        int H, int d, int dv, Strides2 sq, Strides2 sk, Strides2 sv, Strides2 so, const int32_t* offsets,
+                        int offset, cudaStream_t stream) {
+  if (d % 16 || d > 128 || dv % 16 || B > 65535) return BASED_ERR_IMPL;
+  if (!aligned16(q) || !aligned16(k) || !aligned16(v) || !aligned16(out) || !aligned16(state)) return BASED_ERR_IMPL;
+  for (const Strides2& s : {sq, sk, sv, so})
+    if (s.h % 8 || (B > 1 && s.b % 8)) return BASED_ERR_IMPL;
+  Params p{static_cast<const bf16*>(q), static_cast<const bf16*>(k), static_cast<const bf16*>(v), decay, state,
+           static_cast<bf16*>(out), offsets, sq.b, sq.h, sk.b, sk.h, sv.b, sv.h, so.b, so.h, offset, L, H, d, dv, 0, nullptr};
+  // few (batch, head) pairs: their value columns over several CTAs, at least 32 each
+  int slices = (dv + 127) / 128;
+  while ((int64_t)B * H * slices * 2 <= 148 && dv / (slices * 2) >= 32) slices *= 2;
+  p.cols = ((dv + slices - 1) / slices + 15) / 16 * 16;
+  slices = (dv + p.cols - 1) / p.cols;
+  const int aq = (d + 63) / 64, av = (p.cols + 63) / 64;
+  constexpr int kMaxSmem = 227 * 1024;
+  const int smem = (aq + 2 + 4 * av) * (int)kAtom + 132 * 4 + 64 + 1024;
+  if (smem > kMaxSmem || slices > 65535) return BASED_ERR_IMPL;
+  {
+    constexpr int kMaxDevices = 64;
+    static std::mutex mu;
+    static unsigned int* status[kMaxDevices] = {};
+    int dev = 0;
+    cudaError_t e = cudaGetDevice(&dev);
+    if (e != cudaSuccess) return (int)e;
+    if (dev < 0 || dev >= kMaxDevices) return BASED_ERR_TOO_LARGE;
+    std::lock_guard<std::mutex> lock(mu);
+    if (status[dev] == nullptr) {
+      unsigned int* addr = nullptr;
+      e = cudaGetSymbolAddress(reinterpret_cast<void**>(&addr), g_tc_status_lightning);
+      if (e != cudaSuccess) return (int)e;
+      e = cudaFuncSetAttribute(lightning_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, kMaxSmem);
+      if (e != cudaSuccess) return (int)e;
+      status[dev] = addr;
+    }
+    p.status = status[dev];
+  }
+  lightning_tc_kernel<<<dim3(H, B, slices), NT, smem, stream>>>(p);
+  return (int)cudaGetLastError();
+}
+
+}  // namespace based

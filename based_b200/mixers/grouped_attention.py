@@ -44,9 +44,7 @@ class GroupedAttention(StatefulMixer):
             self.out_proj.weight.copy_(t.get(prefix + "o", (W, H * d)))
 
     def allocate_inference_cache(self, batch_size, max_seqlen, dtype=None, **kwargs):
-        dev = self.q_norm.device
-        return {"keys": torch.zeros(batch_size, max_seqlen, self.kv_heads * self.dim, dtype=dtype, device=dev),
-                "factor": torch.zeros(batch_size, self.kv_heads, max_seqlen, dtype=torch.float32, device=dev)}
+        return ops.tied_attention_state(batch_size, self.num_heads, self.kv_heads, self.dim, max_seqlen, dtype, self.q_norm.device)
 
     def heads(self, h, inference_params, out):
         B, L, _ = h.shape
@@ -56,5 +54,5 @@ class GroupedAttention(StatefulMixer):
         q = self.in_proj.slice(x, "q")
         ops.tied_prepare_(q, self.in_proj.slice(x, "k"), self.q_norm, self.k_norm, st["keys"], st["factor"], pos=pos, eps=self.eps,
                           temp_coef=self.temp_coef, temp_every=self.temp_every)
-        ops.tied_attention(q, st["keys"], st["factor"], self.num_heads, self.scale, gate=self.in_proj.slice(x, "g"), pos=pos,
+        ops.tied_attention(q, st["keys"], st["factor"], st["count"], self.num_heads, self.scale, gate=self.in_proj.slice(x, "g"), pos=pos,
                            sink=self.sink, out=out)

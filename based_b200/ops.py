@@ -9,10 +9,10 @@ from typing import Optional, Tuple
 import torch
 
 from . import _capi
-from ._capi import BASED_BF16, BASED_F32, IMPL_AUTO, IMPL_SIMT, IMPL_TCGEN05  # noqa: F401
+from ._capi import BASED_BF16, BASED_F32, IMPL_AUTO, IMPL_DECODE, IMPL_SIMT, IMPL_TCGEN05  # noqa: F401
 
 EXPANDED_DIM = 273
-_IMPLS = {"auto": IMPL_AUTO, "simt": IMPL_SIMT, "tcgen05": IMPL_TCGEN05}
+_IMPLS = {"auto": IMPL_AUTO, "simt": IMPL_SIMT, "tcgen05": IMPL_TCGEN05, "decode": IMPL_DECODE}
 
 
 def _dt(t: torch.dtype) -> int:
@@ -1027,8 +1027,17 @@ def token_gate(z: torch.Tensor, tokens: torch.Tensor, table: torch.Tensor, colum
 def _check_tied(q, cache, factor, B, H, G, d):
     if H % G or q.shape[2] != H * d or cache.shape[0] < B or cache.shape[2] != G * d or cache.dtype != q.dtype or cache.stride(2) != 1:
         raise ValueError("q must be [B, L, H d] and cache [>= B, max_len, G d] in its dtype, H a multiple of G")
-    if factor.dtype != torch.float32 or factor.shape[0] < B or factor.shape[1:] != (G, cache.shape[1]) or factor.stride(2) != 1:
-        raise ValueError("factor must be float32 [>= B, G, max_len]")
+    if factor.dtype != torch.float32 or factor.shape[0] < B or factor.shape[1] != G or factor.shape[2] < cache.shape[1] or factor.stride(2) != 1:
+        raise ValueError("factor must be float32 [>= B, G, >= max_len]")
+
+
+def tied_attention_state(batch: int, heads: int, kv_heads: int, dim: int, max_len: int, dtype, device) -> dict:
+    """What :func:`tied_prepare_` and :func:`tied_attention` keep for ``batch`` sequences: the keys, their factors (rows padded to
+    whole key tiles) and the zeroed counters of a decode step whose keys are split."""
+    rows = max(_capi.TIED_DECODE_ROWS, heads // kv_heads)
+    return {"keys": torch.zeros(batch, max_len, kv_heads * dim, dtype=dtype, device=device),
+            "factor": torch.zeros(batch, kv_heads, (max_len + 127) // 128 * 128, dtype=torch.float32, device=device),
+            "count": torch.zeros(batch * kv_heads * ((rows + 15) // 16), dtype=torch.int32, device=device)}
 
 
 def tied_prepare_(q: torch.Tensor, k: torch.Tensor, q_weight: torch.Tensor, k_weight: torch.Tensor, cache: torch.Tensor,
@@ -1055,12 +1064,14 @@ def tied_prepare_(q: torch.Tensor, k: torch.Tensor, q_weight: torch.Tensor, k_we
     return q
 
 
-def tied_attention(q: torch.Tensor, cache: torch.Tensor, factor: torch.Tensor, heads: int, scale: float, *,
+def tied_attention(q: torch.Tensor, cache: torch.Tensor, factor: torch.Tensor, count: torch.Tensor, heads: int, scale: float, *,
                    gate: Optional[torch.Tensor] = None, pos=0, sink: float = 0.0, out: torch.Tensor, impl: str = "auto") -> torch.Tensor:
     """Causal attention of prepared queries ``q [B, L, H d]`` at positions ``pos ..`` over ``cache [B, max_len, G d]``, whose rows
     are keys (scores times ``factor``) and values; ``sink`` scores of 0 without a value in each softmax sum; ``out [B, L, H d]``
-    times ``sigmoid(gate [B, L, H d])``."""
-    _need_cuda(q, cache, factor, gate, out)
+    times ``sigmoid(gate [B, L, H d])``.  ``count``: int32 zeros, see :func:`tied_attention_state`."""
+    _need_cuda(q, cache, factor, count, gate, out)
+    if count.dtype != torch.int32 or not count.is_contiguous():
+        raise TypeError("count must be a contiguous int32 tensor")
     B, L, W = q.shape
     d = W // heads
     G = cache.shape[2] // d
@@ -1072,10 +1083,14 @@ def tied_attention(q: torch.Tensor, cache: torch.Tensor, factor: torch.Tensor, h
     if out.numel() == 0:
         return out
     with torch.cuda.device(q.device):
+        need = 0
+        if q.dtype == torch.bfloat16 and (impl == "decode" or impl == "auto" and (off is not None or L * (heads // G) <= _capi.TIED_DECODE_ROWS)):
+            need = _capi.lib().based_tied_attention_scratch_bytes(B, L, heads, G, d, cache.shape[1])
+        scratch = torch.empty(need, dtype=torch.uint8, device=q.device) if need else None
         code = _capi.lib().based_tied_attention(
             q.data_ptr(), cache.data_ptr(), factor.data_ptr(), _ptr(gate), out.data_ptr(), B, L, heads, G, d, cache.shape[1],
             _strides_bl(q), _strides_bl(cache), _strides_bl(factor), _strides_bl(gate) if gate is not None else None, _strides_bl(out),
-            off, scalar, float(scale), float(sink), _dt(q.dtype), _IMPLS[impl], None, 0, _stream())
+            off, scalar, float(scale), float(sink), _dt(q.dtype), _IMPLS[impl], _ptr(scratch), need, count.data_ptr(), count.numel(), _stream())
     _capi.check(code, "based_tied_attention")
     return out
 

@@ -605,10 +605,11 @@ def razesun_config(size):
             "residual_mult": 0.5, "logit_scale": 1.0}
 
 
-def random_razesun(size, device="cuda"):
+def random_model(config, device="cuda"):
+    """A model of the registry with random weights."""
     from based_b200.registry import build_model
     torch.manual_seed(0)
-    model = build_model(razesun_config(size), device=device, dtype=torch.bfloat16).eval()
+    model = build_model(config, device=device, dtype=torch.bfloat16).eval()
     with torch.no_grad():
         for name, p in model.named_parameters():
             if p.dim() > 1:
@@ -618,15 +619,15 @@ def random_razesun(size, device="cuda"):
     return model
 
 
-def razesun_generation(B, L, new_tokens, size):
-    """Prompt pass and CUDA-graph decode of a Razesun stack, the same measurement as generation_bench."""
-    model = random_razesun(size)
+def stack_generation(B, L, new_tokens, config, size):
+    """Prompt pass and CUDA-graph decode of a stack of the registry, the same measurement as generation_bench."""
+    model = random_model(config)
     ids = torch.randint(0, model.config.vocab_size, (B, L), device="cuda")
     for _ in range(2):   # at full size: allocator, cuBLAS heuristics
         model.generate(ids, max_new_tokens=new_tokens, cg=True)
     t = {}
     model.generate(ids, max_new_tokens=new_tokens, cg=True, timings=t)
-    res = {"model": f"razesun-{size} (random init)", "params": sum({p.data_ptr(): p.numel() for p in model.parameters()}.values()),
+    res = {"model": f"{config['architecture'].lower()}-{size} (random init)", "params": sum({p.data_ptr(): p.numel() for p in model.parameters()}.values()),
            "B": B, "prompt": L, "new_tokens": new_tokens, "prefill_ms": t["prefill_ms"],
            "prefill_tok_per_s": B * L / (t["prefill_ms"] * 1e-3), "steps_ms_per_step": t["steps_ms"] / (new_tokens - 1),
            "decode_tok_per_s": B * (new_tokens - 1) / (t["steps_ms"] * 1e-3)}
@@ -746,6 +747,119 @@ def razesun_kernels(ops, peaks):
     return out
 
 
+def vubenex_config(size):
+    """A Vubenex stack of the Based model's size: grouped attention where that has SlidingAttention, linear attention with a
+    constant decay in the other layers."""
+    from based_b200.model import BasedConfig
+    cfg = BasedConfig.based_360m() if size == "360m" else BasedConfig.based_1b()
+    d, heads = cfg.n_embd, cfg.n_embd // 128
+    layers = []
+    for i in range(cfg.n_layer):
+        if i in cfg.alt_mixer_2_layers:
+            layer = {"type": "attention", "mixer": {"heads": heads, "kv_heads": max(heads // 4, 1) if heads % 4 == 0 else heads // 2, "dim": 128,
+                                                    "vdim": 128, "scale": 128 ** -0.5, "q_temp": {"coef": 0.1, "every": 1024}}}
+        else:
+            layer = {"type": "lightning", "mixer": {"heads": heads, "dim": 128, "vdim": 128, "decay": [1 - 2.0 ** -(5 + 5 * h / heads) for h in range(heads)]}}
+        layer["mlp"] = {"kind": "dense", "ff": 2 * d}
+        layers.append(layer)
+    return {"architecture": "Vubenex", "vocab": cfg.padded_vocab_size, "width": d, "layers": layers, "norm": {"eps": 1e-6},
+            "embedding": {"scale": d ** 0.5}, "max_positions": 8192, "token_side": {"dim": 64}}
+
+
+def vubenex_kernels(ops, peaks, likes):
+    """Every kernel of the design at layer sizes of a 2048-wide model; ``likes`` are the records of razesun_kernels (same
+    timing), the like kernels among them are named."""
+    dev = "cuda"
+    flush = torch.empty(256 * 1024 * 1024, dtype=torch.uint8, device=dev)
+    g = torch.Generator(device=dev).manual_seed(0)
+    out = {}
+
+    def rnd(*shape, dtype=torch.bfloat16):
+        return torch.randn(*shape, device=dev, generator=g).to(dtype)
+
+    def record(name, what, fn, nbytes, flop=0, iters=10, like=None):
+        t = time_flushed(fn, flush, iters)[0]
+        t_hbm, t_tc = nbytes / (peaks["hbm_gbs"] * 1e9) * 1e3, flop / (peaks["bf16_tflops"] * 1e12) * 1e3
+        out[name] = {"what": what, "ms": t, "roofline_ms": max(t_hbm, t_tc), "frac": max(t_hbm, t_tc) / t,
+                     "bound": "hbm" if t_hbm >= t_tc else "tensor", "like": like}
+        if like:
+            out[name]["distance_ratio"] = likes[like]["frac"] / out[name]["frac"]
+
+    with torch.inference_mode():
+        Hn, G, d, Bd = 16, 4, 128, 256
+        n, m = Hn * d, G * d
+        decay = torch.linspace(0.95, 0.999, Hn, device=dev)
+        for B, L in ((8, 8192), (1, 8192)):
+            x = rnd(B, L, 4 * n)
+            q, k, v, z = x.split(n, -1)
+            S, o = torch.zeros(B, Hn, d, d, device=dev), torch.empty(B, L, n, dtype=torch.bfloat16, device=dev)
+            record(f"lightning_B{B}", f"B={B} L={L} H=16 d=dv=128", lambda: ops.lightning(q, k, v, decay, S, out=o), B * L * n * 8,
+                   4 * d * d * B * L * Hn, like="delta_prefill")
+        B, L = 8, 8192
+        x = rnd(B * L, 2 * n)
+        o, w = torch.empty(B * L, n, dtype=torch.bfloat16, device=dev), rnd(n)
+        record("norm_gate", "rows=65536 D=2048", lambda: ops.norm_gate(x[:, :n], w, x[:, n:], 1e-6, out=o), B * L * n * 6, like="stream_norm")
+        del x, o, q, k, v, z
+        x, S, o = rnd(Bd, 4 * n), torch.zeros(Bd, Hn, d, d, device=dev), torch.empty(Bd, n, dtype=torch.bfloat16, device=dev)
+        read, count = torch.empty(Bd, n, device=dev), torch.zeros(Bd, dtype=torch.int32, device=dev)
+        pos = torch.full((Bd,), 100, dtype=torch.int32, device=dev)
+        record("lightning_step", "B=256 H=16 d=dv=128", lambda: ops.lightning_step(*x.split(n, -1), decay, w, S, read, count, pos=pos, eps=1e-6, out=o),
+               S.numel() * 8 + Bd * n * 10, like="delta_step")
+        del S, x
+        wq = rnd(d)
+        for B, L in ((4, 8192), (8, 2048)):
+            x = rnd(B, L, 2 * n + m)
+            q, k, z = x.split([n, m, n], -1)
+            st, o = ops.tied_attention_state(B, Hn, G, d, L, torch.bfloat16, dev), torch.empty(B, L, n, dtype=torch.bfloat16, device=dev)
+            ops.tied_prepare_(q, k, wq, wq, st["keys"], st["factor"])
+            record(f"tied_prefill_L{L}", f"B={B} L={L} H=16 kv_heads=4 d=128, gate", lambda: ops.tied_attention(
+                   q, st["keys"], st["factor"], st["count"], Hn, d ** -0.5, gate=z, sink=1.0, out=o),
+                   B * L * (3 * n + m) * 2, 2 * B * Hn * L * L * d, like=f"latent_prefill_L{L}")
+            record(f"tied_prepare_L{L}", f"B={B} L={L} H=16 kv_heads=4 d=128", lambda: ops.tied_prepare_(
+                   q, k, wq, wq, st["keys"], st["factor"], temp_coef=0.1, temp_every=1024), B * L * (n + m) * 4, like="latent_prepare")
+            del x, q, k, z, st, o
+        T = 4096
+        for B in (64, 16):
+            st, x = ops.tied_attention_state(B, Hn, G, d, T, torch.bfloat16, dev), rnd(B, 1, 2 * n)
+            st["keys"].normal_()
+            st["factor"].fill_(1.0)
+            o, pos = torch.empty(B, 1, n, dtype=torch.bfloat16, device=dev), torch.full((B,), T - 1, dtype=torch.int32, device=dev)
+            record(f"tied_decode_B{B}", f"B={B} keys=4096 H=16 kv_heads=4 d=128, gate", lambda: ops.tied_attention(
+                   x[..., :n], st["keys"], st["factor"], st["count"], Hn, d ** -0.5, gate=x[..., n:], pos=pos, sink=1.0, out=o),
+                   st["keys"].numel() * 2 + st["factor"].numel() * 4, 4 * B * T * Hn * d, like=f"latent_decode_B{B}")
+        M, D, ns = 16 * 2048, 2048, 256
+        res, br, w1 = rnd(M, D, dtype=torch.float32), rnd(M, D), rnd(D)
+        record("stream_post_norm", "rows=32768 D=2048", lambda: ops.stream_post_norm(res, br, w1), M * D * 12, like="stream_norm")
+        table, tab, ids = rnd(50280, D), rnd(2048, D), torch.randint(0, 50280, (16, 2048), device=dev)
+        record("stream_embed", "rows=32768 D=2048", lambda: ops.stream_embed(res.view(16, 2048, D), ids, table, 45.0, tab), M * D * 8 + 2048 * D * 2,
+               like="stream_norm")
+        zs, te = rnd(M, ns), rnd(50280, 4 * ns)
+        record("token_gate", "rows=32768 n=256", lambda: ops.token_gate(zs, ids, te, ns), M * ns * 6, like="stream_norm")
+    return out
+
+
+def run_vubenex(args):
+    """The --vubenex option: one JSON line with the design's kernels and generation beside the Razesun model's."""
+    from based_b200 import build_library, ops
+    build_library()
+    peaks = load_peaks()
+    sampler = ClockSampler(0)
+    sampler.start()
+    likes = razesun_kernels(ops, peaks)
+    torch.cuda.empty_cache()
+    line = {"bench": "vubenex", "data": "synthetic", "dtype": "bf16", "peaks": peaks, "kernels": vubenex_kernels(ops, peaks, likes), "like_kernels": likes}
+    torch.cuda.empty_cache()
+    line["generation"] = []
+    for size, B, L, new in (("360m", 16, 2048, 256), ("1b", 8, 4096, 256)):
+        ours = stack_generation(B, L, new, vubenex_config(size), size)
+        other = stack_generation(B, L, new, razesun_config(size), size)
+        line["generation"].append({"vubenex": ours, "razesun": other, "prefill_ratio": ours["prefill_tok_per_s"] / other["prefill_tok_per_s"],
+                                   "decode_ratio": other["steps_ms_per_step"] / ours["steps_ms_per_step"]})
+    line["clocks"] = sampler.stop()
+    line["status"] = ops.check_status()
+    print(json.dumps(line), flush=True)
+
+
 def run_razesun(args):
     """The --razesun option: one JSON line with the design's kernels and generation beside the Based model's."""
     from based_b200 import build_library, ops
@@ -757,7 +871,7 @@ def run_razesun(args):
     torch.cuda.empty_cache()
     line["generation"] = []
     for size, B, L, new in (("360m", 16, 2048, 256), ("1b", 8, 4096, 256)):
-        ours = razesun_generation(B, L, new, size)
+        ours = stack_generation(B, L, new, razesun_config(size), size)
         based = generation_bench(B=B, L=L, new_tokens=new, size=size)
         line["generation"].append({"razesun": ours, "based": based, "prefill_ratio": ours["prefill_tok_per_s"] / based["prefill_tok_per_s"],
                                    "decode_ratio": based["steps_ms_per_step"] / ours["steps_ms_per_step"]})
@@ -782,6 +896,8 @@ def main():
                     "median / min / max record (the first one is the headline)")
     ap.add_argument("--razesun", action="store_true",
                     help="instead of the headline: kernels and generation of the Razesun design beside the Based model's (one GPU)")
+    ap.add_argument("--vubenex", action="store_true",
+                    help="instead of the headline: kernels and generation of the Vubenex design beside the Razesun model's (one GPU)")
     args = ap.parse_args()
     args.warmup = max(args.warmup, 3)
 
@@ -794,6 +910,10 @@ def main():
 
     if args.razesun:
         run_razesun(args)
+        return
+
+    if args.vubenex:
+        run_vubenex(args)
         return
 
     import torch.distributed as dist

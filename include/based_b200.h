@@ -569,18 +569,28 @@ int based_tied_prepare(void* q, const void* k, const void* q_weight, const void*
 /*
  * Causal attention of prepared queries over that cache: score = (q . k) * factor * scale, values = k, query head h reads key
  * head h / (H / G), `sink` scores of 0 without a value in every softmax sum; out [B, L, H d], times sigmoid(gate) element by
- * element when gate [B, L, H d] is given.  Query l sees keys 0 .. offset + l.  AUTO picks by dtype, sizes and the number of
- * query rows.  scratch: based_tied_attention_scratch_bytes bytes, 16-byte aligned (NULL when that is 0).
+ * element when gate [B, L, H d] is given.  Query l sees keys 0 .. offset + l.  Rows of factor must be readable up to the next
+ * multiple of 128 keys for the tensor-core kernels.  For bf16 AUTO takes BASED_IMPL_DECODE for device offsets and up to
+ * BASED_TIED_DECODE_ROWS query rows per key head (tokens x heads of the group), BASED_IMPL_TCGEN05 above, and
+ * BASED_IMPL_SIMT where those do not take the sizes.  The decode form may split the keys: scratch is
+ * based_tied_attention_scratch_bytes bytes, 16-byte aligned (NULL when that is 0), count [B * G * ceil(rows / 16)] int32 (a
+ * shorter one: no split) is
+ * zero before the first call and zero again after every call.
  */
+#define BASED_IMPL_DECODE 3
+#define BASED_TIED_DECODE_ROWS 64
+size_t based_tied_attention_scratch_bytes(int B, int L, int H, int G, int d, int max_len);
 int based_tied_attention(const void* q, const void* cache, const void* factor, const void* gate, void* out, int B, int L, int H,
                          int G, int d, int max_len, const int64_t q_strides[2], const int64_t cache_strides[2],
                          const int64_t factor_strides[2], const int64_t gate_strides[2], const int64_t out_strides[2],
                          const int32_t* offsets, int offset, float scale, float sink, int io_dtype, int impl, void* scratch,
-                         size_t scratch_bytes, void* stream);
+                         size_t scratch_bytes, void* count, int count_len, void* stream);
 
 /*
  * S <- decay S + silu(k) silu(v)^T, out = S^T silu(q) over the tokens of a call: q, k [B, L, H d], v [B, L, H dv] before silu
  * (strides batch, token; heads contiguous), decay [H] fp32, state [B, H, d, dv] fp32 updated, out [B, L, H dv].  d <= 512.
+ * AUTO: the chunked tensor-core kernel (BASED_IMPL_TCGEN05) for bf16 calls of 16 tokens or more with d <= 128, d and dv multiples of
+ * 16, strides multiples of 8 and 16-byte alignment, else token by token (BASED_IMPL_SIMT).
  */
 int based_lightning(const void* q, const void* k, const void* v, const void* decay, void* state, void* out, int B, int L, int H,
                     int d, int dv, const int64_t q_strides[2], const int64_t k_strides[2], const int64_t v_strides[2],
