@@ -36,7 +36,7 @@ const char* based_error_string(int code) {
 }
 
 int based_read_status(unsigned int* out, int reset) {
-  unsigned int a = 0, b = 0, c = 0, d = 0, e = 0, f = 0, g = 0, h = 0;
+  unsigned int a = 0, b = 0, c = 0, d = 0, e = 0, f = 0, g = 0, h = 0, i = 0;
   int rc = read_tc_status ? read_tc_status(&a, reset) : 0;
   if (rc == 0 && read_tc_status_swa) rc = read_tc_status_swa(&b, reset);
   if (rc == 0 && read_tp_status) rc = read_tp_status(&c, reset);
@@ -45,7 +45,8 @@ int based_read_status(unsigned int* out, int reset) {
   if (rc == 0 && read_tc_status_rglru) rc = read_tc_status_rglru(&f, reset);
   if (rc == 0 && read_tc_status_tied) rc = read_tc_status_tied(&g, reset);
   if (rc == 0 && read_tc_status_lightning) rc = read_tc_status_lightning(&h, reset);
-  if (out) *out = a | b | c | d | e | f | g | h;
+  if (rc == 0 && read_tc_status_tied_decode) rc = read_tc_status_tied_decode(&i, reset);
+  if (out) *out = a | b | c | d | e | f | g | h | i;
   return rc;
 }
 

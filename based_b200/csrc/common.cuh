@@ -203,6 +203,7 @@ BASED_WEAK int launch_tied_prefill_tc(const void* q, const void* cache, const fl
                                       int64_t fh, int64_t gb, int64_t gl, int64_t ob, int64_t ol, int offset, float scale,
                                       float sink, cudaStream_t stream);
 BASED_WEAK int read_tc_status_tied(unsigned int* out, int reset);
+BASED_WEAK int read_tc_status_tied_decode(unsigned int* out, int reset);
 BASED_WEAK size_t tied_decode_scratch_bytes(int B, int R, int G, int d, int max_len);
 BASED_WEAK int launch_tied_decode(const void* q, const void* cache, const float* factor, const void* gate, void* out,
                                   void* scratch, size_t scratch_bytes, int* count, int count_len, int B, int L, int H, int G,

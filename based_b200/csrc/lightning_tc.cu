@@ -6,7 +6,7 @@
 //   warps 0-3    scores: (Q K^T)_ij times g^(i-j) to P (bf16, in the scores' columns); read-out: O = P V + g^(i+1) Q S0
 //   warps 4-7    state: S0 (TMEM) to the bf16 operand of Q S0, and g^n S0 back to TMEM
 //   warp 8       MMA issue
-//   warps 9-24   loads: raw projections of the next chunk to registers, silu there, then to shared memory when the chunk
+//   warps 12-27  loads: raw projections of the next chunk to registers, silu there, then to shared memory when the chunk
 //                before is done - the registers are the second buffer, shared memory holds one chunk
 // 32-bit in the recurrence: the state is the fp32 accumulator and is scaled in fp32; g^(n-1-j) v_j enters as a bf16 pair
 // hi + lo (16 mantissa bits) against k as the activation stored it.  Scores and decays are fp32 until P, and nothing feeds
@@ -28,9 +28,12 @@ using namespace tc;
 using bf16 = __nv_bfloat16;
 
 constexpr int C = 128;                      // tokens per chunk
-constexpr int kLoaders = 512, NT = 9 * 32 + kLoaders;
+constexpr int kLoaders = 512, NT = 12 * 32 + kLoaders;   // seven warpgroups; three warps beside the MMA warp are idle
+// registers per thread: 72 at launch; the loaders take what the others leave (7 * 72 = 72 + 48 + 32 + 4 * 88)
+constexpr int kStateRegs = 48, kMmaRegs = 32, kLoadRegs = 88;
 constexpr int kItems = C * 16 / kLoaders;   // 16-byte pieces per thread and tensor at 128 columns
 constexpr uint32_t kAtom = 128 * 128;       // bytes of 128 rows x 64 columns
+constexpr int kTables = 32 + 132 + 32;
 
 struct Params {
   const bf16 *q, *k, *v;
@@ -46,12 +49,34 @@ struct Params {
 __device__ __forceinline__ float ex2(float x) { float r; asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(x)); return r; }
 __device__ __forceinline__ float rcp(float x) { float r; asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(x)); return r; }
 
-// silu of two packed values; both sigmoids from one reciprocal
-__device__ __forceinline__ uint32_t silu2(uint32_t w) {
-  const float a = seq::bf16_lo(w), b = seq::bf16_hi(w);
-  const float ea = 1.f + ex2(fminf(a * -1.4426950408889634f, 60.f)), eb = 1.f + ex2(fminf(b * -1.4426950408889634f, 60.f));
-  const float r = rcp(ea * eb);
-  return pack_bf16(a * (r * eb), b * (r * ea));
+// two fp32 values in one 64-bit register, for the packed arithmetic instructions
+__device__ __forceinline__ uint64_t pair(float lo, float hi) { uint64_t r; asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(lo), "f"(hi)); return r; }
+__device__ __forceinline__ void split(uint64_t v, float& lo, float& hi) { asm("mov.b64 {%0, %1}, %2;" : "=f"(lo), "=f"(hi) : "l"(v)); }
+__device__ __forceinline__ uint64_t mul2(uint64_t a, uint64_t b) { uint64_t r; asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b)); return r; }
+__device__ __forceinline__ uint64_t add2(uint64_t a, uint64_t b) { uint64_t r; asm("add.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b)); return r; }
+__device__ __forceinline__ uint32_t pack2(uint64_t v) { float lo, hi; split(v, lo, hi); return pack_bf16(lo, hi); }
+
+// volatile: stays where it is written, a chunk ahead of its use
+__device__ __forceinline__ uint4 load16(const bf16* src) {
+  uint4 v;
+  asm volatile("ld.global.nc.L1::no_allocate.v4.b32 {%0, %1, %2, %3}, [%4];" : "=r"(v.x), "=r"(v.y), "=r"(v.z), "=r"(v.w) : "l"(src));
+  return v;
+}
+
+// silu of four packed values; the four sigmoids share one reciprocal.  Below -20 silu counts as its value there, -4e-8.
+__device__ __forceinline__ void silu4(uint32_t& u, uint32_t& w) {
+  asm("max.bf16x2 %0, %0, %1;" : "+r"(u) : "r"(0xc1a0c1a0u));
+  asm("max.bf16x2 %0, %0, %1;" : "+r"(w) : "r"(0xc1a0c1a0u));
+  const uint64_t x = pair(seq::bf16_lo(u), seq::bf16_hi(u)), y = pair(seq::bf16_lo(w), seq::bf16_hi(w));
+  const uint64_t nl = pair(-1.4426950408889634f, -1.4426950408889634f), one = pair(1.f, 1.f);
+  float a, b, c, d;
+  split(mul2(x, nl), a, b);
+  split(mul2(y, nl), c, d);
+  split(add2(pair(ex2(a), ex2(b)), one), a, b);    // at most 2^29 each
+  split(add2(pair(ex2(c), ex2(d)), one), c, d);
+  const float ab = a * b, cd = c * d, r = rcp(ab * cd), rab = r * cd, rcd = r * ab;
+  u = pack2(mul2(x, mul2(pair(rab, rab), pair(b, a))));
+  w = pack2(mul2(y, mul2(pair(rcd, rcd), pair(d, c))));
 }
 
 __global__ void __launch_bounds__(NT, 1) lightning_tc_kernel(const __grid_constant__ Params p) {
@@ -65,8 +90,10 @@ __global__ void __launch_bounds__(NT, 1) lightning_tc_kernel(const __grid_consta
   const int aq = (p.d + 63) / 64, av = (p.cols + 63) / 64;
   // shared memory: Q, K (always two atoms: its transpose is a 128-row operand), V, hi and lo of the decayed V, S0
   const uint32_t SM_K = aq * kAtom, SM_V = SM_K + 2 * kAtom, SM_W = SM_V + av * kAtom, SM_S = SM_W + 2 * av * kAtom,
-                 SM_POW = SM_S + av * kAtom, SM_BAR = SM_POW + 132 * 4;
-  float* pw = reinterpret_cast<float*>(smem + SM_POW);   // g^0 .. g^128
+                 SM_POW = SM_S + av * kAtom, SM_BAR = SM_POW + kTables * 4;
+  float* pz = reinterpret_cast<float*>(smem + SM_POW);   // 32 zeros, g^0 .. g^128
+  float* pw = pz + 32;
+  float* pr = pw + 132;                                  // g^31 .. g^0
   const uint32_t B_FULL = sb + SM_BAR, B_A = B_FULL + 8, B_P = B_FULL + 16, B_S0 = B_FULL + 24, B_S = B_FULL + 32,
                  B_O = B_FULL + 40, B_OF = B_FULL + 48;
   uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(smem + SM_BAR + 56);
@@ -81,6 +108,7 @@ __global__ void __launch_bounds__(NT, 1) lightning_tc_kernel(const __grid_consta
     float r = 1.f, x = p.decay[h];
     for (int e = tid; e > 0; e >>= 1) { if (e & 1) r *= x; x *= x; }
     pw[tid] = r;
+    if (tid < 32) { pz[tid] = 0.f; pr[31 - tid] = r; }
   }
   for (uint32_t i = tid * 16; i < 2 * kAtom; i += NT * 16) *reinterpret_cast<uint4*>(smem + SM_K + i) = make_uint4(0, 0, 0, 0);
   fence_proxy_async();
@@ -91,74 +119,88 @@ __global__ void __launch_bounds__(NT, 1) lightning_tc_kernel(const __grid_consta
   const uint32_t tmem = *tmem_slot;
   constexpr uint32_t TM_A = 0, TM_S = 128, TM_O = 256, TM_I = 384;
 
-  if (warp >= 9) {
+  if (warp >= 12) {
+    asm volatile("setmaxnreg.inc.sync.aligned.u32 %0;" ::"n"(kLoadRegs));
     // ---------------- loads, silu, operands
-    const int t = tid - 9 * 32;
+    // a thread keeps one 16-byte column and takes every `step`-th row of it; a row's columns are padded to a power of two
+    const int t = tid - 12 * 32;
     const int cq = p.d / 8, cv = cols / 8;
-    const uint32_t iq = ((1u << 20) + cq - 1) / cq, iv = ((1u << 20) + cv - 1) / cv;   // exact quotients for the indices used
-    const bf16* q = p.q + b * p.qb + (int64_t)h * p.d;
-    const bf16* k = p.k + b * p.kb + (int64_t)h * p.d;
-    const bf16* v = p.v + b * p.vb + (int64_t)h * p.dv + col0;
+    const int wq = 32 - __clz(cq - 1), wv = 32 - __clz(cv - 1);           // log2 of the padded widths
+    const int rowq = t >> wq, rowv = t >> wv, colq = t & ((1 << wq) - 1), colv = t & ((1 << wv) - 1);
+    const int stepq = kLoaders >> wq, stepv = kLoaders >> wv;
+    const bool onq = colq < cq && rowq < C, onv = colv < cv && rowv < C;
+    const bf16* q = p.q + b * p.qb + (int64_t)h * p.d + rowq * p.ql + colq * 8;
+    const bf16* k = p.k + b * p.kb + (int64_t)h * p.d + rowq * p.kl + colq * 8;
+    const bf16* v = p.v + b * p.vb + (int64_t)h * p.dv + col0 + rowv * p.vl + colv * 8;
+    // steps are multiples of 8 rows (or there is one row only): the swizzle is the same for all of a thread's rows
+    const uint32_t atq = (colq >> 3) * kAtom + tma::sw128_offset(rowq & (C - 1), colq & 7), atv = (colv >> 3) * kAtom + tma::sw128_offset(rowv & (C - 1), colv & 7);
     uint4 rq[kItems], rk[kItems], rv[kItems];
-    auto fetch = [&](int c) {
-      const int l0 = c * C;
+    auto load = [&](uint4 (&r)[kItems], const bf16* src, int64_t stride, int row, int step, bool on, int n) {
 #pragma unroll
-      for (int i = 0; i < kItems; ++i) {
-        const int e = t + i * kLoaders, row = (int)((e * iq) >> 20), cc = (e - row * cq) * 8, l = l0 + row;
-        const bool ok = row < C && l < p.L;
-        rq[i] = ok ? __ldg(reinterpret_cast<const uint4*>(q + (int64_t)l * p.ql + cc)) : make_uint4(0, 0, 0, 0);
-        rk[i] = ok ? __ldg(reinterpret_cast<const uint4*>(k + (int64_t)l * p.kl + cc)) : make_uint4(0, 0, 0, 0);
-      }
-#pragma unroll
-      for (int i = 0; i < kItems; ++i) {
-        const int e = t + i * kLoaders, row = (int)((e * iv) >> 20), cc = (e - row * cv) * 8, l = l0 + row;
-        rv[i] = row < C && l < p.L ? __ldg(reinterpret_cast<const uint4*>(v + (int64_t)l * p.vl + cc)) : make_uint4(0, 0, 0, 0);
-      }
+      for (int i = 0; i < kItems; ++i)
+        if (i * step < C) r[i] = on && row + i * step < n ? load16(src + i * step * stride) : make_uint4(0, 0, 0, 0);
     };
-    auto act = [&](uint4& x) { x.x = silu2(x.x); x.y = silu2(x.y); x.z = silu2(x.z); x.w = silu2(x.w); };
-    fetch(0);
+    auto act = [&](uint4 (&r)[kItems], int step) {
+#pragma unroll
+      for (int i = 0; i < kItems; ++i)
+        if (i * step < C) { silu4(r[i].x, r[i].y); silu4(r[i].z, r[i].w); }
+    };
+    // shared memory holds one chunk: a tensor's registers are written when the products of the chunk before no longer
+    // read its place, and take the next chunk's values at once
+    const int n0 = min(C, p.L);
+    load(rq, q, p.ql, rowq, stepq, onq, n0);
+    load(rk, k, p.kl, rowq, stepq, onq, n0);
+    load(rv, v, p.vl, rowv, stepv, onv, n0);
     for (int c = 0; c < nc; ++c) {
+      const int n = min(C, p.L - c * C), next = min(C, p.L - (c + 1) * C);   // not positive: the loads give zeros
+      q += C * p.ql;
+      k += C * p.kl;
+      v += C * p.vl;
+      act(rq, stepq);
+      if (c > 0) mbar_wait_bounded(B_S, (c - 1) & 1, abort_flag, p.status, 1u << 0);
+      if (onq) {
 #pragma unroll
-      for (int i = 0; i < kItems; ++i) act(rq[i]);
-#pragma unroll
-      for (int i = 0; i < kItems; ++i) act(rk[i]);
-#pragma unroll
-      for (int i = 0; i < kItems; ++i) act(rv[i]);
-      if (c > 0) mbar_wait_bounded(B_O, (c - 1) & 1, abort_flag, p.status, 1u << 0);
-      const int n = min(C, p.L - c * C);
-#pragma unroll
-      for (int i = 0; i < kItems; ++i) {
-        const int e = t + i * kLoaders, row = (int)((e * iq) >> 20), cc = e - row * cq;
-        if (row < C) {
-          const uint32_t at = (cc >> 3) * kAtom + tma::sw128_offset(row, cc & 7);
-          *reinterpret_cast<uint4*>(smem + at) = rq[i];
-          *reinterpret_cast<uint4*>(smem + SM_K + at) = rk[i];
-        }
+        for (int i = 0; i < kItems; ++i)
+          if (i * stepq < C) *reinterpret_cast<uint4*>(smem + atq + i * stepq * 128) = rq[i];
       }
+      load(rq, q, p.ql, rowq, stepq, onq, next);
+      act(rk, stepq);
+      if (onq) {
 #pragma unroll
-      for (int i = 0; i < kItems; ++i) {
-        const int e = t + i * kLoaders, row = (int)((e * iv) >> 20), cc = e - row * cv;
-        if (row < C) {
-          const uint32_t at = (cc >> 3) * kAtom + tma::sw128_offset(row, cc & 7);
-          *reinterpret_cast<uint4*>(smem + SM_V + at) = rv[i];
-          const float f = row < n ? pw[n - 1 - row] : 0.f;
-          uint32_t hi[4], lo[4];
-          const uint32_t w[4] = {rv[i].x, rv[i].y, rv[i].z, rv[i].w};
+        for (int i = 0; i < kItems; ++i)
+          if (i * stepq < C) *reinterpret_cast<uint4*>(smem + SM_K + atq + i * stepq * 128) = rk[i];
+      }
+      load(rk, k, p.kl, rowq, stepq, onq, next);
+      act(rv, stepv);
+      if (c > 0) mbar_wait_bounded(B_O, (c - 1) & 1, abort_flag, p.status, 1u << 9);
+      if (onv) {
 #pragma unroll
-          for (int m = 0; m < 4; ++m) {
-            const float x = seq::bf16_lo(w[m]) * f, y = seq::bf16_hi(w[m]) * f;
-            hi[m] = pack_bf16(x, y);
-            lo[m] = pack_bf16(x - seq::bf16_lo(hi[m]), y - seq::bf16_hi(hi[m]));
+        for (int i = 0; i < kItems; ++i)
+          if (i * stepv < C) {
+            uint8_t* dst = smem + SM_V + atv + i * stepv * 128;
+            *reinterpret_cast<uint4*>(dst) = rv[i];
+            const float f = pw[max(n - 1 - rowv - i * stepv, 0)];      // rows past the end are zero
+            const uint64_t f2 = pair(f, f);
+            uint32_t hi[4], lo[4];
+            const uint32_t w[4] = {rv[i].x, rv[i].y, rv[i].z, rv[i].w};
+#pragma unroll
+            for (int m = 0; m < 4; ++m) {
+              float x, y;
+              split(mul2(pair(seq::bf16_lo(w[m]), seq::bf16_hi(w[m])), f2), x, y);
+              hi[m] = pack_bf16(x, y);
+              lo[m] = pack_bf16(x - seq::bf16_lo(hi[m]), y - seq::bf16_hi(hi[m]));
+            }
+            *reinterpret_cast<uint4*>(dst + av * kAtom) = make_uint4(hi[0], hi[1], hi[2], hi[3]);
+            *reinterpret_cast<uint4*>(dst + 2 * av * kAtom) = make_uint4(lo[0], lo[1], lo[2], lo[3]);
           }
-          *reinterpret_cast<uint4*>(smem + SM_W + at) = make_uint4(hi[0], hi[1], hi[2], hi[3]);
-          *reinterpret_cast<uint4*>(smem + SM_W + av * kAtom + at) = make_uint4(lo[0], lo[1], lo[2], lo[3]);
-        }
       }
+      load(rv, v, p.vl, rowv, stepv, onv, next);
       fence_proxy_async();
       mbar_arrive(B_FULL);
-      if (c + 1 < nc) fetch(c + 1);
     }
-  } else if (warp == 8) {
+  } else if (warp >= 8) {
+    asm volatile("setmaxnreg.dec.sync.aligned.u32 %0;" ::"n"(kMmaRegs));
+    if (warp == 8) {
     // ---------------- MMA issue (converged warp, one elected lane)
     const uint32_t tm = __shfl_sync(0xffffffffu, tmem, 0);
     const bool leader = elect_one_sync();
@@ -200,7 +242,9 @@ __global__ void __launch_bounds__(NT, 1) lightning_tc_kernel(const __grid_consta
       if (leader) mma_commit(B_O);     // read-out complete, and every operand of this chunk read
       __syncwarp();
     }
+    }
   } else if (warp >= 4) {
+    asm volatile("setmaxnreg.dec.sync.aligned.u32 %0;" ::"n"(kStateRegs));
     // ---------------- state: one row (key dimension) per thread
     const int row = tid - 128;
     const uint32_t ts = tmem + ((uint32_t)((warp & 3) * 32) << 16) + TM_S;
@@ -269,16 +313,17 @@ __global__ void __launch_bounds__(NT, 1) lightning_tc_kernel(const __grid_consta
           tmem_ld_wait();
           if (x < warp) {             // g^(i-j) = g^(i-last column) g^(last column-j): no power of it is negative
             const float f = pw[i - 32 * x - 31];
+            const uint64_t f2 = pair(f, f);
 #pragma unroll
-            for (int j = 0; j < 16; ++j)
-              w[j] = pack_bf16(__uint_as_float(r[2 * j]) * (f * pw[31 - 2 * j]), __uint_as_float(r[2 * j + 1]) * (f * pw[30 - 2 * j]));
+            for (int j = 0; j < 8; ++j) {
+              const float4 y = *reinterpret_cast<const float4*>(pr + 4 * j);
+              w[2 * j] = pack2(mul2(pair(__uint_as_float(r[4 * j]), __uint_as_float(r[4 * j + 1])), mul2(f2, pair(y.x, y.y))));
+              w[2 * j + 1] = pack2(mul2(pair(__uint_as_float(r[4 * j + 2]), __uint_as_float(r[4 * j + 3])), mul2(f2, pair(y.z, y.w))));
+            }
           } else {
 #pragma unroll
-            for (int j = 0; j < 16; ++j) {
-              const int u = lane - 2 * j;
-              const float f0 = u >= 0 ? pw[u] : 0.f, f1 = u >= 1 ? pw[u - 1] : 0.f;
-              w[j] = pack_bf16(u >= 0 ? __uint_as_float(r[2 * j]) * f0 : 0.f, u >= 1 ? __uint_as_float(r[2 * j + 1]) * f1 : 0.f);
-            }
+            for (int j = 0; j < 16; ++j)
+              w[j] = pack_bf16(__uint_as_float(r[2 * j]) * pw[lane - 2 * j], __uint_as_float(r[2 * j + 1]) * pw[lane - 2 * j - 1]);
           }
         } else {
 #pragma unroll
@@ -354,7 +399,7 @@ int launch_lightning_tc(const void* q, const void* k, const void* v, const float
   slices = (dv + p.cols - 1) / p.cols;
   const int aq = (d + 63) / 64, av = (p.cols + 63) / 64;
   constexpr int kMaxSmem = 227 * 1024;
-  const int smem = (aq + 2 + 4 * av) * (int)kAtom + 132 * 4 + 64 + 1024;
+  const int smem = (aq + 2 + 4 * av) * (int)kAtom + kTables * 4 + 64 + 1024;
   if (smem > kMaxSmem || slices > 65535) return BASED_ERR_IMPL;
   {
     constexpr int kMaxDevices = 64;
