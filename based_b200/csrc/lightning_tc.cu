@@ -5,9 +5,11 @@
 // One CTA walks the chunks of one (batch, head) (or of a slice of its value columns) with the state as a TMEM accumulator:
 //   warps 0-3    scores: (Q K^T)_ij times g^(i-j) to P (bf16, in the scores' columns); read-out: O = P V + g^(i+1) Q S0
 //   warps 4-7    state: S0 (TMEM) to the bf16 operand of Q S0, and g^n S0 back to TMEM
-//   warp 8       MMA issue
-//   warps 12-27  loads: raw projections of the next chunk to registers, silu there, then to shared memory when the chunk
-//                before is done - the registers are the second buffer, shared memory holds one chunk
+//   warps 8, 9   MMA issue; TMA loads of v and prefetches into L2
+//   warps 12-27  operands: silu of the next chunk while the tensor cores work on this one.  q and k wait in registers, the
+//                second buffer that shared memory has no room for; v arrives by TMA in one of two buffers and is replaced
+//                by its silu in place.  When a chunk's read-out is complete its v buffer takes the output tile on its way
+//                to a TMA store
 // 32-bit in the recurrence: the state is the fp32 accumulator and is scaled in fp32; g^(n-1-j) v_j enters as a bf16 pair
 // hi + lo (16 mantissa bits) against k as the activation stored it.  Scores and decays are fp32 until P, and nothing feeds
 // the read-out back.
@@ -28,7 +30,7 @@ using namespace tc;
 using bf16 = __nv_bfloat16;
 
 constexpr int C = 128;                      // tokens per chunk
-constexpr int kLoaders = 512, NT = 12 * 32 + kLoaders;   // seven warpgroups; three warps beside the MMA warp are idle
+constexpr int kLoaders = 512, NT = 12 * 32 + kLoaders;   // seven warpgroups; two of them idle
 // registers per thread: 72 at launch; the loaders take what the others leave (7 * 72 = 72 + 48 + 32 + 4 * 88)
 constexpr int kStateRegs = 48, kMmaRegs = 32, kLoadRegs = 88;
 constexpr int kItems = C * 16 / kLoaders;   // 16-byte pieces per thread and tensor at 128 columns
@@ -36,13 +38,14 @@ constexpr uint32_t kAtom = 128 * 128;       // bytes of 128 rows x 64 columns
 constexpr int kTables = 32 + 132 + 32;
 
 struct Params {
-  const bf16 *q, *k, *v;
+  CUtensorMap mq, mk, mv, mo;               // [B][H][L][.]; q and k for prefetches into L2
+  const bf16 *q, *k;
   const float* decay;
   float* state;
   bf16* out;
   const int32_t* offsets;
-  int64_t qb, ql, kb, kl, vb, vl, ob, ol;
-  int offset, L, H, d, dv, cols;            // cols: value columns per CTA
+  int64_t qb, ql, kb, kl, ob, ol;
+  int offset, L, H, d, dv, cols, tma_out;   // cols: value columns per CTA
   unsigned int* status;
 };
 
@@ -88,19 +91,19 @@ __global__ void __launch_bounds__(NT, 1) lightning_tc_kernel(const __grid_consta
   const int cols = min(p.cols, p.dv - col0);
   const int nc = (p.L + C - 1) / C;
   const int aq = (p.d + 63) / 64, av = (p.cols + 63) / 64;
-  // shared memory: Q, K (always two atoms: its transpose is a 128-row operand), V, hi and lo of the decayed V, S0
-  const uint32_t SM_K = aq * kAtom, SM_V = SM_K + 2 * kAtom, SM_W = SM_V + av * kAtom, SM_S = SM_W + 2 * av * kAtom,
+  // shared memory: Q, K (always two atoms: its transpose is a 128-row operand), two of V, hi and lo of the decayed V, S0
+  const uint32_t SM_K = aq * kAtom, SM_V = SM_K + 2 * kAtom, SM_W = SM_V + 2 * av * kAtom, SM_S = SM_W + 2 * av * kAtom,
                  SM_POW = SM_S + av * kAtom, SM_BAR = SM_POW + kTables * 4;
   float* pz = reinterpret_cast<float*>(smem + SM_POW);   // 32 zeros, g^0 .. g^128
   float* pw = pz + 32;
   float* pr = pw + 132;                                  // g^31 .. g^0
   const uint32_t B_FULL = sb + SM_BAR, B_A = B_FULL + 8, B_P = B_FULL + 16, B_S0 = B_FULL + 24, B_S = B_FULL + 32,
-                 B_O = B_FULL + 40, B_OF = B_FULL + 48;
-  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(smem + SM_BAR + 56);
+                 B_O = B_FULL + 40, B_OF = B_FULL + 48, B_VF = B_FULL + 56, B_R = B_FULL + 64;
+  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(smem + SM_BAR + 80);
   volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_slot + 1);
   if (tid == 0) {
     mbar_init(B_FULL, kLoaders); mbar_init(B_A, 1); mbar_init(B_P, 128); mbar_init(B_S0, 128); mbar_init(B_S, 1);
-    mbar_init(B_O, 1); mbar_init(B_OF, 128);
+    mbar_init(B_O, 1); mbar_init(B_OF, 128); mbar_init(B_VF, 1); mbar_init(B_R, 1); mbar_init(B_R + 8, 1);
     *abort_flag = 0;
     fence_mbar_init();
   }
@@ -131,10 +134,9 @@ __global__ void __launch_bounds__(NT, 1) lightning_tc_kernel(const __grid_consta
     const bool onq = colq < cq && rowq < C, onv = colv < cv && rowv < C;
     const bf16* q = p.q + b * p.qb + (int64_t)h * p.d + rowq * p.ql + colq * 8;
     const bf16* k = p.k + b * p.kb + (int64_t)h * p.d + rowq * p.kl + colq * 8;
-    const bf16* v = p.v + b * p.vb + (int64_t)h * p.dv + col0 + rowv * p.vl + colv * 8;
     // steps are multiples of 8 rows (or there is one row only): the swizzle is the same for all of a thread's rows
     const uint32_t atq = (colq >> 3) * kAtom + tma::sw128_offset(rowq & (C - 1), colq & 7), atv = (colv >> 3) * kAtom + tma::sw128_offset(rowv & (C - 1), colv & 7);
-    uint4 rq[kItems], rk[kItems], rv[kItems];
+    uint4 rq[kItems], rk[kItems];
     auto load = [&](uint4 (&r)[kItems], const bf16* src, int64_t stride, int row, int step, bool on, int n) {
 #pragma unroll
       for (int i = 0; i < kItems; ++i)
@@ -145,44 +147,43 @@ __global__ void __launch_bounds__(NT, 1) lightning_tc_kernel(const __grid_consta
       for (int i = 0; i < kItems; ++i)
         if (i * step < C) { silu4(r[i].x, r[i].y); silu4(r[i].z, r[i].w); }
     };
-    // shared memory holds one chunk: a tensor's registers are written when the products of the chunk before no longer
-    // read its place, and take the next chunk's values at once
-    const int n0 = min(C, p.L);
-    load(rq, q, p.ql, rowq, stepq, onq, n0);
-    load(rk, k, p.kl, rowq, stepq, onq, n0);
-    load(rv, v, p.vl, rowv, stepv, onv, n0);
+    load(rq, q, p.ql, rowq, stepq, onq, min(C, p.L));
+    load(rk, k, p.kl, rowq, stepq, onq, min(C, p.L));
     for (int c = 0; c < nc; ++c) {
-      const int n = min(C, p.L - c * C), next = min(C, p.L - (c + 1) * C);   // not positive: the loads give zeros
-      q += C * p.ql;
-      k += C * p.kl;
-      v += C * p.vl;
+      const int n = min(C, p.L - c * C);
+      uint8_t* vb = smem + SM_V + (c & 1) * av * kAtom + atv;
       act(rq, stepq);
-      if (c > 0) mbar_wait_bounded(B_S, (c - 1) & 1, abort_flag, p.status, 1u << 0);
-      if (onq) {
-#pragma unroll
-        for (int i = 0; i < kItems; ++i)
-          if (i * stepq < C) *reinterpret_cast<uint4*>(smem + atq + i * stepq * 128) = rq[i];
-      }
-      load(rq, q, p.ql, rowq, stepq, onq, next);
       act(rk, stepq);
+      mbar_wait_bounded(B_R + 8 * (c & 1), (c >> 1) & 1, abort_flag, p.status, 1u << 10);
+      if (onv) {
+        uint4 rv[kItems];
+#pragma unroll
+        for (int i = 0; i < kItems; ++i)
+          if (i * stepv < C) rv[i] = *reinterpret_cast<const uint4*>(vb + i * stepv * 128);
+        act(rv, stepv);
+#pragma unroll
+        for (int i = 0; i < kItems; ++i)
+          if (i * stepv < C) *reinterpret_cast<uint4*>(vb + i * stepv * 128) = rv[i];
+      }
+      if (c > 0) mbar_wait_bounded(B_S, (c - 1) & 1, abort_flag, p.status, 1u << 0);   // Q, K and W of the chunk before are free
       if (onq) {
 #pragma unroll
         for (int i = 0; i < kItems; ++i)
-          if (i * stepq < C) *reinterpret_cast<uint4*>(smem + SM_K + atq + i * stepq * 128) = rk[i];
+          if (i * stepq < C) {
+            *reinterpret_cast<uint4*>(smem + atq + i * stepq * 128) = rq[i];
+            *reinterpret_cast<uint4*>(smem + SM_K + atq + i * stepq * 128) = rk[i];
+          }
       }
-      load(rk, k, p.kl, rowq, stepq, onq, next);
-      act(rv, stepv);
-      if (c > 0) mbar_wait_bounded(B_O, (c - 1) & 1, abort_flag, p.status, 1u << 9);
       if (onv) {
 #pragma unroll
         for (int i = 0; i < kItems; ++i)
           if (i * stepv < C) {
-            uint8_t* dst = smem + SM_V + atv + i * stepv * 128;
-            *reinterpret_cast<uint4*>(dst) = rv[i];
+            uint8_t* dst = smem + SM_W + atv + i * stepv * 128;
+            const uint4 r = *reinterpret_cast<const uint4*>(vb + i * stepv * 128);
             const float f = pw[max(n - 1 - rowv - i * stepv, 0)];      // rows past the end are zero
             const uint64_t f2 = pair(f, f);
             uint32_t hi[4], lo[4];
-            const uint32_t w[4] = {rv[i].x, rv[i].y, rv[i].z, rv[i].w};
+            const uint32_t w[4] = {r.x, r.y, r.z, r.w};
 #pragma unroll
             for (int m = 0; m < 4; ++m) {
               float x, y;
@@ -190,13 +191,18 @@ __global__ void __launch_bounds__(NT, 1) lightning_tc_kernel(const __grid_consta
               hi[m] = pack_bf16(x, y);
               lo[m] = pack_bf16(x - seq::bf16_lo(hi[m]), y - seq::bf16_hi(hi[m]));
             }
-            *reinterpret_cast<uint4*>(dst + av * kAtom) = make_uint4(hi[0], hi[1], hi[2], hi[3]);
-            *reinterpret_cast<uint4*>(dst + 2 * av * kAtom) = make_uint4(lo[0], lo[1], lo[2], lo[3]);
+            *reinterpret_cast<uint4*>(dst) = make_uint4(hi[0], hi[1], hi[2], hi[3]);
+            *reinterpret_cast<uint4*>(dst + av * kAtom) = make_uint4(lo[0], lo[1], lo[2], lo[3]);
           }
       }
-      load(rv, v, p.vl, rowv, stepv, onv, next);
       fence_proxy_async();
       mbar_arrive(B_FULL);
+      if (c + 1 < nc) {
+        q += C * p.ql;
+        k += C * p.kl;
+        load(rq, q, p.ql, rowq, stepq, onq, min(C, p.L - (c + 1) * C));
+        load(rk, k, p.kl, rowq, stepq, onq, min(C, p.L - (c + 1) * C));
+      }
     }
   } else if (warp >= 8) {
     asm volatile("setmaxnreg.dec.sync.aligned.u32 %0;" ::"n"(kMmaRegs));
@@ -205,7 +211,7 @@ __global__ void __launch_bounds__(NT, 1) lightning_tc_kernel(const __grid_consta
     const uint32_t tm = __shfl_sync(0xffffffffu, tmem, 0);
     const bool leader = elect_one_sync();
     const uint32_t id_a = make_idesc_bf16(128, C, 0, 0), id_i = make_idesc_bf16(128, cols, 0, 1), id_s = make_idesc_bf16(128, cols, 1, 1);
-    const uint64_t dk_t = make_smem_desc_sw128(sb + SM_K, kAtom, 1024), dv_ = make_smem_desc_sw128(sb + SM_V, kAtom, 1024);
+    const uint64_t dk_t = make_smem_desc_sw128(sb + SM_K, kAtom, 1024), dv_[2] = {make_smem_desc_sw128(sb + SM_V, kAtom, 1024), make_smem_desc_sw128(sb + SM_V + av * kAtom, kAtom, 1024)};
     const uint64_t dw0 = make_smem_desc_sw128(sb + SM_W, kAtom, 1024), dw1 = make_smem_desc_sw128(sb + SM_W + av * kAtom, kAtom, 1024);
     const uint64_t ds = make_smem_desc_sw128(sb + SM_S, kAtom, 1024);
     const int ks = p.d / 16;
@@ -238,10 +244,25 @@ __global__ void __launch_bounds__(NT, 1) lightning_tc_kernel(const __grid_consta
       fence_after_sync();
 #pragma unroll
       for (int k = 0; k < C / 16; ++k)
-        if (leader) mma_ts(tm + TM_O, tm + TM_A + 8 * k, dv_ + 128 * k, id_i, k > 0 ? 1u : 0u);
+        if (leader) mma_ts(tm + TM_O, tm + TM_A + 8 * k, (ph ? dv_[1] : dv_[0]) + 128 * k, id_i, k > 0 ? 1u : 0u);
       if (leader) mma_commit(B_O);     // read-out complete, and every operand of this chunk read
       __syncwarp();
     }
+    } else if (warp == 9 && lane == 0) {
+      // ---------------- v by TMA; the chunk after the next into L2
+      for (int c = 0; c < nc; ++c) {
+        if (c >= 2) mbar_wait_bounded<false>(B_VF, c & 1, abort_flag, p.status, 1u << 8);   // chunk c - 2 has given its output away
+        const uint32_t full = B_R + 8 * (c & 1);
+        tma::mbar_expect_tx(full, av * kAtom);
+        for (int a = 0; a < av; ++a) tma::load_4d(sb + SM_V + ((c & 1) * av + a) * kAtom, &p.mv, full, col0 + 64 * a, c * C, h, b);
+        if (c + 1 < nc) {
+          for (int a = 0; a < av; ++a) tma::prefetch_4d(&p.mv, col0 + 64 * a, (c + 1) * C, h, b);
+          for (int a = 0; a < aq; ++a) {
+            tma::prefetch_4d(&p.mq, 64 * a, (c + 1) * C, h, b);
+            tma::prefetch_4d(&p.mk, 64 * a, (c + 1) * C, h, b);
+          }
+        }
+      }
     }
   } else if (warp >= 4) {
     asm volatile("setmaxnreg.dec.sync.aligned.u32 %0;" ::"n"(kStateRegs));
@@ -340,24 +361,40 @@ __global__ void __launch_bounds__(NT, 1) lightning_tc_kernel(const __grid_consta
       const float g = pw[i + 1];
       const bool live = c * C + i < p.L;
       bf16* o = out + (int64_t)(c * C + i) * p.ol;
+      uint8_t* tile = smem + SM_V + (c & 1) * av * kAtom;
       for (int x = 0; x < cols; x += 16) {
-        uint32_t r0[16], r1[16];
+        uint32_t r0[16], r1[16], w[8];
         tmem_ld16(tl + TM_O + x, r0);
         tmem_ld16(tl + TM_I + x, r1);
         tmem_ld_wait();
-        if (live) {
-          uint32_t w[8];
 #pragma unroll
-          for (int m = 0; m < 8; ++m)
-            w[m] = pack_bf16(fmaf(__uint_as_float(r1[2 * m]), g, __uint_as_float(r0[2 * m])),
-                             fmaf(__uint_as_float(r1[2 * m + 1]), g, __uint_as_float(r0[2 * m + 1])));
-          *reinterpret_cast<uint4*>(o + x) = make_uint4(w[0], w[1], w[2], w[3]);
-          *reinterpret_cast<uint4*>(o + x + 8) = make_uint4(w[4], w[5], w[6], w[7]);
+        for (int m = 0; m < 8; ++m)
+          w[m] = pack_bf16(fmaf(__uint_as_float(r1[2 * m]), g, __uint_as_float(r0[2 * m])),
+                           fmaf(__uint_as_float(r1[2 * m + 1]), g, __uint_as_float(r0[2 * m + 1])));
+        const uint4 lo = make_uint4(w[0], w[1], w[2], w[3]), hi = make_uint4(w[4], w[5], w[6], w[7]);
+        if (p.tma_out) {
+          uint8_t* atom = tile + (x >> 6) * kAtom;
+          *reinterpret_cast<uint4*>(atom + tma::sw128_offset(i, (x & 63) >> 3)) = lo;
+          *reinterpret_cast<uint4*>(atom + tma::sw128_offset(i, ((x & 63) >> 3) + 1)) = hi;
+        } else if (live) {
+          *reinterpret_cast<uint4*>(o + x) = lo;
+          *reinterpret_cast<uint4*>(o + x + 8) = hi;
         }
       }
       fence_before_sync();
       mbar_arrive(B_OF);
+      if (p.tma_out) fence_proxy_async();
+      asm volatile("bar.sync 1, 128;" ::: "memory");   // these four warps
+      if (tid == 0) {
+        if (p.tma_out) {               // rows past the sequence and columns past the head are clipped
+          for (int a = 0; a < av; ++a) tma::store_4d(&p.mo, sb + SM_V + ((c & 1) * av + a) * kAtom, col0 + 64 * a, c * C, h, b);
+          bulk_commit();
+          bulk_wait_read_all();
+        }
+        mbar_arrive(B_VF);
+      }
     }
+    if (tid == 0) bulk_wait_all();
   }
   __syncwarp();
   fence_before_sync();
@@ -390,8 +427,8 @@ int launch_lightning_tc(const void* q, const void* k, const void* v, const float
   if (!aligned16(q) || !aligned16(k) || !aligned16(v) || !aligned16(out) || !aligned16(state)) return BASED_ERR_IMPL;
   for (const Strides2& s : {sq, sk, sv, so})
     if (s.h % 8 || (B > 1 && s.b % 8)) return BASED_ERR_IMPL;
-  Params p{static_cast<const bf16*>(q), static_cast<const bf16*>(k), static_cast<const bf16*>(v), decay, state,
-           static_cast<bf16*>(out), offsets, sq.b, sq.h, sk.b, sk.h, sv.b, sv.h, so.b, so.h, offset, L, H, d, dv, 0, nullptr};
+  Params p{{}, {}, {}, {}, static_cast<const bf16*>(q), static_cast<const bf16*>(k), decay, state, static_cast<bf16*>(out), offsets,
+           sq.b, sq.h, sk.b, sk.h, so.b, so.h, offset, L, H, d, dv, 0, 0, nullptr};
   // few (batch, head) pairs: their value columns over several CTAs, at least 32 each
   int slices = (dv + 127) / 128;
   while ((int64_t)B * H * slices * 2 <= 148 && dv / (slices * 2) >= 32) slices *= 2;
@@ -399,7 +436,7 @@ int launch_lightning_tc(const void* q, const void* k, const void* v, const float
   slices = (dv + p.cols - 1) / p.cols;
   const int aq = (d + 63) / 64, av = (p.cols + 63) / 64;
   constexpr int kMaxSmem = 227 * 1024;
-  const int smem = (aq + 2 + 4 * av) * (int)kAtom + kTables * 4 + 64 + 1024;
+  const int smem = (aq + 2 + 5 * av) * (int)kAtom + kTables * 4 + 88 + 1024;
   if (smem > kMaxSmem || slices > 65535) return BASED_ERR_IMPL;
   {
     constexpr int kMaxDevices = 64;
@@ -420,6 +457,19 @@ int launch_lightning_tc(const void* q, const void* k, const void* v, const float
     }
     p.status = status[dev];
   }
+  static tma::MapCache maps;
+  auto fix = [](int64_t st, int extent) { return extent == 1 ? (int64_t)8 : st; };
+  auto get_map = [&](CUtensorMap* m, const void* base, int w, const Strides2& st) -> int {
+    const int64_t sl = fix(st.h, L), sbt = fix(st.b, B);
+    if (sl <= 0 || sbt <= 0) return 1;
+    const tma::MapKey key = tma::make_key(base, w, L, H, B, 0, sl, w, sbt, 0, 64, C, 0, 4);
+    if (maps.find(key, m)) return 0;
+    if (tma::encode_bf16_4d_sw128(m, base, w, L, H, B, sl, w, sbt, 64, C)) return 1;
+    maps.put(key, *m);
+    return 0;
+  };
+  if (get_map(&p.mq, q, d, sq) || get_map(&p.mk, k, d, sk) || get_map(&p.mv, v, dv, sv) || get_map(&p.mo, out, dv, so)) return BASED_ERR_IMPL;
+  p.tma_out = slices == 1 || p.cols % 64 == 0;   // a slice's tile must not reach into the next one
   lightning_tc_kernel<<<dim3(H, B, slices), NT, smem, stream>>>(p);
   return (int)cudaGetLastError();
 }

@@ -144,6 +144,12 @@ __device__ __forceinline__ void load_5d(uint32_t dst_saddr, const CUtensorMap* m
       "l"(map), "r"(mbar_saddr), "r"(c0), "r"(c1), "r"(c2), "r"(c3), "r"(c4)
       : "memory");
 }
+// The tile a load with these coordinates would bring, into L2 only.
+__device__ __forceinline__ void prefetch_4d(const CUtensorMap* map, int c0, int c1, int c2, int c3) {
+  asm volatile("cp.async.bulk.prefetch.tensor.4d.L2.global.tile [%0, {%1, %2, %3, %4}];\n" ::"l"(map), "r"(c0), "r"(c1), "r"(c2),
+               "r"(c3)
+               : "memory");
+}
 // Tile store shared -> global (rows past the tensor's extent are clipped); never started at a
 // negative coordinate.
 __device__ __forceinline__ void store_4d(const CUtensorMap* map, uint32_t src_saddr, int c0, int c1, int c2, int c3) {
