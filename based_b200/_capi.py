@@ -76,6 +76,7 @@ SIGNATURES = {
     "based_norm_gate": (c_int, [c_void_p, c_int64, c_void_p, c_void_p, c_int64, c_void_p, c_int64, c_int64, c_int, c_float, c_int,
                                 c_void_p]),
     "based_token_gate": (c_int, [c_void_p, c_int64, c_void_p, c_void_p] + [c_int64] * 3 + [c_void_p, c_int64, c_int, c_int, c_void_p]),
+    "based_token_side": (c_int, [c_void_p, c_int64] + [c_void_p] * 4 + [c_int64] * 3 + [c_void_p] * 4 + [c_int] * 3 + [c_float, c_int, c_void_p]),
     "based_tied_prepare": (c_int, [c_void_p] * 6 + [c_int] * 6 + [_I64P] * 4 + _POS + [c_float] * 3 + [c_int, c_void_p]),
     "based_tied_attention": (c_int, [c_void_p] * 5 + [c_int] * 6 + [_I64P] * 5 + _POS
                              + [c_float, c_float, c_int, c_int, c_void_p, ctypes.c_size_t, c_void_p, c_int, c_void_p]),

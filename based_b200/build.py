@@ -14,7 +14,7 @@ LIBNAME = "libbased_b200.so"
 HYBRID = ("capi.cu", "norm_act.cu", "decode_linear.cu", "short_conv.cu", "gated_delta.cu", "gated_delta_chunk.cu", "rglru.cu",
           "rglru_tc.cu", "latent_attention.cu", "latent_decode.cu", "latent_prefill_tc.cu")
 POSTNORM = ("capi.cu", "norm_act.cu", "decode_linear.cu", "latent_attention.cu", "tied_attention.cu", "tied_decode.cu",
-            "tied_prefill_tc.cu", "lightning.cu", "lightning_tc.cu")
+            "tied_prefill_tc.cu", "lightning.cu", "lightning_tc.cu", "token_side.cu")
 PARTS = {"hybrid": ("libbased_b200_hybrid.so", HYBRID), "postnorm": ("libbased_b200_postnorm.so", POSTNORM)}
 _chosen = None   # library of the part this process asked for, when that is not the whole one
 

@@ -615,6 +615,19 @@ int based_token_gate(const void* z, int64_t z_row_stride, const void* tokens, co
                            io_dtype, static_cast<cudaStream_t>(stream));
 }
 
+int based_token_side(const void* x, int64_t x_row_stride, const void* tokens, const void* gate_weight, const void* proj_weight,
+                     const void* table, int64_t V, int64_t table_row_stride, int64_t column, const void* norm_weight, void* residual,
+                     const void* out_weight, void* out, int M, int W, int n, float eps, int io_dtype, void* stream) {
+  if (!x || !tokens || !gate_weight || !proj_weight || !table || !norm_weight || !residual || !out) return BASED_ERR_NULL;
+  if (!dtype_ok(io_dtype)) return BASED_ERR_DTYPE;
+  if (M < 0 || W <= 0 || n <= 0 || V <= 0 || column < 0 || column + n > table_row_stride) return BASED_ERR_SHAPE;
+  if (M == 0) return BASED_OK;
+  if (io_dtype != BASED_BF16 || !launch_token_side) return BASED_ERR_IMPL;
+  return launch_token_side(x, x_row_stride, static_cast<const int64_t*>(tokens), gate_weight, proj_weight, table, V, table_row_stride,
+                           column, norm_weight, static_cast<float*>(residual), out_weight, out, M, W, n, eps,
+                           static_cast<cudaStream_t>(stream));
+}
+
 int based_tied_prepare(void* q, const void* k, const void* q_weight, const void* k_weight, void* cache, void* factor, int B,
                        int L, int H, int G, int d, int max_len, const int64_t q_strides[2], const int64_t k_strides[2],
                        const int64_t cache_strides[2], const int64_t factor_strides[2], const int32_t* offsets, int offset,

@@ -194,6 +194,9 @@ int launch_norm_gate(const void* x, int64_t sx, const void* w, const void* gate,
                      int D, float eps, int io_dtype, cudaStream_t stream);
 int launch_token_gate(const void* z, int64_t sz, const int64_t* tokens, const void* table, int64_t V, int64_t st,
                       int64_t column, void* out, int64_t M, int n, int io_dtype, cudaStream_t stream);
+BASED_WEAK int launch_token_side(const void* x, int64_t sx, const int64_t* tokens, const void* wg, const void* wp, const void* table,
+                                 int64_t V, int64_t st, int64_t column, const void* norm, float* residual, const void* out_norm,
+                                 void* out, int M, int W, int n, float eps, cudaStream_t stream);
 BASED_WEAK int launch_tied_prepare(void* q, const void* k, const void* wq, const void* wk, void* cache, float* factor, int B,
                                    int L, int H, int G, int d, int max_len, int64_t qb, int64_t ql, int64_t kb, int64_t kl,
                                    int64_t cb, int64_t cl, int64_t fb, int64_t fh, const int32_t* offsets, int offset,

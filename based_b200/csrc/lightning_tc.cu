@@ -31,8 +31,8 @@ using bf16 = __nv_bfloat16;
 
 constexpr int C = 128;                      // tokens per chunk
 constexpr int kLoaders = 512, NT = 12 * 32 + kLoaders;   // seven warpgroups; two of them idle
-// registers per thread: 72 at launch; the loaders take what the others leave (7 * 72 = 72 + 48 + 32 + 4 * 88)
-constexpr int kStateRegs = 48, kMmaRegs = 32, kLoadRegs = 88;
+// registers per thread: 72 at launch; the loaders take what the others leave (7 * 72 = 72 + 40 + 40 + 4 * 88)
+constexpr int kStateRegs = 40, kMmaRegs = 40, kLoadRegs = 88;
 constexpr int kItems = C * 16 / kLoaders;   // 16-byte pieces per thread and tensor at 128 columns
 constexpr uint32_t kAtom = 128 * 128;       // bytes of 128 rows x 64 columns
 constexpr int kTables = 32 + 132 + 32;
@@ -233,19 +233,19 @@ __global__ void __launch_bounds__(NT, 1) lightning_tc_kernel(const __grid_consta
         const uint64_t da = make_smem_desc_sw128(sb + (k >> 2) * kAtom + (k & 3) * 32, 16, 1024);
         if (leader) mma_ss(tm + TM_I, da, ds + 128 * k, id_i, k > 0 ? 1u : 0u);
       }
-#pragma unroll
-      for (int k = 0; k < C / 16; ++k) {
-        if (leader) mma_ss(tm + TM_S, dk_t + 128 * k, dw0 + 128 * k, id_s, 1u);
-        if (leader) mma_ss(tm + TM_S, dk_t + 128 * k, dw1 + 128 * k, id_s, 1u);
-      }
-      if (leader) mma_commit(B_S);
-      __syncwarp();
+      // the read-out before the state: its buffers have the longer way back
       mbar_wait_bounded(B_P, ph, abort_flag, p.status, 1u << 4);
       fence_after_sync();
 #pragma unroll
       for (int k = 0; k < C / 16; ++k)
         if (leader) mma_ts(tm + TM_O, tm + TM_A + 8 * k, (ph ? dv_[1] : dv_[0]) + 128 * k, id_i, k > 0 ? 1u : 0u);
-      if (leader) mma_commit(B_O);     // read-out complete, and every operand of this chunk read
+      if (leader) mma_commit(B_O);
+#pragma unroll
+      for (int k = 0; k < C / 16; ++k) {
+        if (leader) mma_ss(tm + TM_S, dk_t + 128 * k, dw0 + 128 * k, id_s, 1u);
+        if (leader) mma_ss(tm + TM_S, dk_t + 128 * k, dw1 + 128 * k, id_s, 1u);
+      }
+      if (leader) mma_commit(B_S);     // every operand of this chunk read
       __syncwarp();
     }
     } else if (warp == 9 && lane == 0) {

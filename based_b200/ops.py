@@ -1024,6 +1024,42 @@ def token_gate(z: torch.Tensor, tokens: torch.Tensor, table: torch.Tensor, colum
     return out
 
 
+TOKEN_SIDE_MAX_WEIGHT = 200_000   # elements of one matrix up to which one cluster per 16 rows beats the separate launches
+
+
+def token_side_step(residual: torch.Tensor, x: torch.Tensor, tokens: torch.Tensor, gate_weight: torch.Tensor, proj_weight: torch.Tensor,
+                    table: torch.Tensor, column: int, norm_weight: torch.Tensor, *, out_weight: Optional[torch.Tensor] = None,
+                    eps: float = 1e-6) -> Optional[torch.Tensor]:
+    """A layer's token input for a few rows in one launch: ``x [..., W]`` through ``gate_weight [n, W]``, :func:`token_gate`,
+    ``proj_weight [W, n]`` and :func:`stream_post_norm`.  None, nothing launched, for rows, sizes or dtypes it does not take."""
+    _need_cuda(residual, x, tokens, gate_weight, proj_weight, table, norm_weight, out_weight)
+    n, W = gate_weight.shape
+    M = x.numel() // W if W else 0
+    if x.dtype != torch.bfloat16 or not 0 < M <= DECODE_LINEAR_MAX_ROWS or n * W > TOKEN_SIDE_MAX_WEIGHT:
+        return None
+    _same_dtype(x, x=x, gate_weight=gate_weight, proj_weight=proj_weight, table=table, norm_weight=norm_weight, out_weight=out_weight)
+    x2 = flat_rows(x)
+    if residual.dtype != torch.float32 or not residual.is_contiguous() or residual.shape != x.shape:
+        raise TypeError("residual must be a contiguous float32 tensor of x's shape")
+    if proj_weight.shape != (W, n) or not (gate_weight.is_contiguous() and proj_weight.is_contiguous()):
+        raise ValueError("gate_weight must be [n, W] and proj_weight [W, n], contiguous")
+    if tokens.dtype != torch.int64 or tokens.numel() != M or not 0 <= column <= table.shape[1] - n:
+        raise ValueError("tokens must be int64, one per row, and the slice inside the table")
+    if norm_weight.shape != (W,) or (out_weight is not None and out_weight.shape != (W,)):
+        raise ValueError("norm weights must have the stream's width")
+    out = torch.empty(x.shape, dtype=x.dtype, device=x.device)
+    tokens = tokens.contiguous()
+    with torch.cuda.device(x.device):
+        code = _capi.lib().based_token_side(
+            x2.data_ptr(), x2.stride(0), tokens.data_ptr(), gate_weight.data_ptr(), proj_weight.data_ptr(), table.data_ptr(), table.shape[0],
+            table.stride(0), int(column), norm_weight.data_ptr(), residual.data_ptr(), _ptr(out_weight), out.data_ptr(), M, W, n, float(eps),
+            _dt(x.dtype), _stream())
+    if code == _capi.ERR_IMPL:
+        return None
+    _capi.check(code, "based_token_side")
+    return out
+
+
 def _check_tied(q, cache, factor, B, H, G, d):
     if H % G or q.shape[2] != H * d or cache.shape[0] < B or cache.shape[2] != G * d or cache.dtype != q.dtype or cache.stride(2) != 1:
         raise ValueError("q must be [B, L, H d] and cache [>= B, max_len, G d] in its dtype, H a multiple of G")

@@ -66,8 +66,13 @@ class TokenSide(nn.Module):
             self.proj.weight.copy_(t.get(prefix + "proj", (W, d)))
             self.norm.copy_(t.get(prefix + "norm", (W,)))
 
-    def forward(self, x, tokens, table):
-        return ops.linear(ops.token_gate(ops.linear(x, self.gate.weight), tokens, table, self.column), self.proj.weight)
+    def forward(self, stream, x, tokens, table, out_norm, eps):
+        """Adds to the stream in place; returns it as :func:`ops.stream_post_norm` does."""
+        y = ops.token_side_step(stream, x, tokens, self.gate.weight, self.proj.weight, table, self.column, self.norm, out_weight=out_norm, eps=eps)
+        if y is None:
+            y = ops.linear(ops.token_gate(ops.linear(x, self.gate.weight), tokens, table, self.column), self.proj.weight)
+            y = ops.stream_post_norm(stream, y, self.norm, out_weight=out_norm, eps=eps)
+        return y
 
 
 class PostNormBlock(nn.Module):
@@ -106,7 +111,7 @@ class PostNormBlock(nn.Module):
         x = ops.stream_post_norm(stream, self.mixer(x, inference_params), self.norm1, eps=self.eps)
         if self.mlp is not None:
             x = ops.stream_post_norm(stream, self.mlp(x), self.norm2, eps=self.eps)
-        return ops.stream_post_norm(stream, self.side(x, tokens, side_table), self.side.norm, out_weight=out_norm, eps=self.eps)
+        return self.side(stream, x, tokens, side_table, out_norm, self.eps)
 
 
 class VubenexLMHeadModel(GenerationMixin, nn.Module):

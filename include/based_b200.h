@@ -555,6 +555,16 @@ int based_token_gate(const void* z, int64_t z_row_stride, const void* tokens, co
                      int64_t table_row_stride, int64_t column, void* out, int64_t M, int n, int io_dtype, void* stream);
 
 /*
+ * The whole token input of a layer for the few rows of a decode step (bf16): residual += norm(W_proj (gelu_tanh(W_gate x) *
+ * table[token, column ..])) * norm_weight and out as in based_stream_post_norm; gate_weight [n, W], proj_weight [W, n]
+ * contiguous.  Built for M <= 64 (more rows re-read the weights per 16).  BASED_ERR_IMPL: fp32, W or n no multiple of 8,
+ * n above 256, W above 8192, unaligned.
+ */
+int based_token_side(const void* x, int64_t x_row_stride, const void* tokens, const void* gate_weight, const void* proj_weight,
+                     const void* table, int64_t V, int64_t table_row_stride, int64_t column, const void* norm_weight, void* residual,
+                     const void* out_weight, void* out, int M, int W, int n, float eps, int io_dtype, void* stream);
+
+/*
  * Between the projections and the attention of a layer whose values are its keys before their norm: q [B, L, H d] becomes
  * q / rms(q) * q_weight * k_weight * (1 + temp_coef ln(floor((p + 1) / temp_every) + 1)) in place; k [B, L, G d] is copied to
  * the cache rows of its positions and 1 / rms(k) (eps inside the root) to factor [B, G, max_len] fp32.  Strides are

@@ -216,3 +216,28 @@ def test_token_gate(n, dtype):
         assert float((got.double().cpu() - want).abs().max() / want.abs().max()) < (2e-6 if dtype == torch.float32 else 1e-2)
     with pytest.raises(ValueError, match="inside"):
         ops.token_gate(z.to(dtype).cuda(), ids.cuda(), table.to(dtype).cuda(), 3 * n + 1)
+
+
+@pytest.mark.parametrize("M,W,n", [(1, 64, 8), (5, 320, 24), (16, 512, 64), (17, 512, 256), (33, 96, 16), (64, 2048, 88), (3, 4096, 40), (2, 8192, 8)])
+def test_token_input_in_one_launch(M, W, n):
+    from based_b200 import ops
+    g = torch.Generator().manual_seed(M)
+    rnd = lambda *s, scale=1.0: (torch.randn(*s, generator=g) * scale).bfloat16()
+    x, wg, wp, table = rnd(M, W), rnd(n, W, scale=W ** -0.5), rnd(W, n, scale=n ** -0.5), rnd(30, 3 * n)
+    norm, out_norm, stream = rnd(W), rnd(W), torch.randn(M, W, generator=g)
+    ids = torch.randint(0, 30, (M,), generator=g)
+    e = table.double()[ids][:, n:2 * n]
+    want = stream.double() + V.rms((V.gelu_tanh(x.double() @ wg.double().T) * e) @ wp.double().T, EPS, norm.double())
+    for last in (None, out_norm):
+        s = stream.cuda()
+        y = ops.token_side_step(s, x.cuda(), ids.cuda(), wg.cuda(), wp.cuda(), table.cuda(), n, norm.cuda(), out_weight=None if last is None else last.cuda(), eps=EPS)
+        assert float((s.double().cpu() - want).abs().max()) < 5e-2
+        ref = s.double().cpu() if last is None else V.rms(s.double().cpu(), EPS, last.double())
+        assert float((y.double().cpu() - ref).abs().max() / ref.abs().max()) < 1e-2
+        again = stream.cuda()                       # the separate steps
+        z = ops.token_gate(torch.nn.functional.linear(x.cuda(), wg.cuda()), ids.cuda(), table.cuda(), n)
+        ops.stream_post_norm(again, torch.nn.functional.linear(z, wp.cuda()), norm.cuda(), eps=EPS)
+        assert float((again - s).abs().max()) < 8e-2
+    assert ops.token_side_step(stream.cuda(), x.float().cuda(), ids.cuda(), wg.float().cuda(), wp.float().cuda(), table.float().cuda(), n, norm.float().cuda()) is None
+    big = torch.zeros(128, 2048).bfloat16().cuda()     # too much weight for one cluster
+    assert ops.token_side_step(torch.zeros(1, 2048, device="cuda"), big[:1], ids[:1].cuda(), big, big.view(2048, 128), table.cuda().repeat(1, 128), 0, big[0]) is None
