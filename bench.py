@@ -783,7 +783,7 @@ def vubenex_kernels(ops, peaks, likes):
         out[name] = {"what": what, "ms": t, "roofline_ms": max(t_hbm, t_tc), "frac": max(t_hbm, t_tc) / t,
                      "bound": "hbm" if t_hbm >= t_tc else "tensor", "like": like}
         if like:
-            out[name]["distance_ratio"] = likes[like]["frac"] / out[name]["frac"]
+            out[name]["distance_ratio"] = (likes.get(like) or out[like])["frac"] / out[name]["frac"]
 
     with torch.inference_mode():
         Hn, G, d, Bd = 16, 4, 128, 256
@@ -793,8 +793,12 @@ def vubenex_kernels(ops, peaks, likes):
             x = rnd(B, L, 4 * n)
             q, k, v, z = x.split(n, -1)
             S, o = torch.zeros(B, Hn, d, d, device=dev), torch.empty(B, L, n, dtype=torch.bfloat16, device=dev)
+            if B == 1:   # the like kernel at this size: one sequence does not fill the machine
+                a, A, wn, h4 = rnd(B, L, Hn, dtype=torch.float32), rnd(Hn, dtype=torch.float32), rnd(d), [t.unflatten(-1, (Hn, d)) for t in (q, k, v, z)]
+                record("delta_prefill_B1", "B=1 L=8192 H=16 d=128 dv=128 (Razesun)", lambda: ops.delta_prefill(*h4, a, a, A, A, wn, S, out=o),
+                       B * L * Hn * (5 * d * 2 + 8), 6 * d * d * B * L * Hn)
             record(f"lightning_B{B}", f"B={B} L={L} H=16 d=dv=128", lambda: ops.lightning(q, k, v, decay, S, out=o), B * L * n * 8,
-                   4 * d * d * B * L * Hn, like="delta_prefill")
+                   4 * d * d * B * L * Hn, like="delta_prefill" if B > 1 else "delta_prefill_B1")
         B, L = 8, 8192
         x = rnd(B * L, 2 * n)
         o, w = torch.empty(B * L, n, dtype=torch.bfloat16, device=dev), rnd(n)
@@ -833,8 +837,15 @@ def vubenex_kernels(ops, peaks, likes):
         table, tab, ids = rnd(50280, D), rnd(2048, D), torch.randint(0, 50280, (16, 2048), device=dev)
         record("stream_embed", "rows=32768 D=2048", lambda: ops.stream_embed(res.view(16, 2048, D), ids, table, 45.0, tab), M * D * 8 + 2048 * D * 2,
                like="stream_norm")
-        zs, te = rnd(M, ns), rnd(50280, 4 * ns)
-        record("token_gate", "rows=32768 n=256", lambda: ops.token_gate(zs, ids, te, ns), M * ns * 6, like="stream_norm")
+        zs, te, ya = rnd(M, ns), rnd(50280, 4 * ns), rnd(M, 2 * ns)
+        record("gated_act", "rows=32768 F=256 (Based, Razesun)", lambda: ops.gated_act(ya), M * ns * 6)
+        record("token_gate", "rows=32768 n=256", lambda: ops.token_gate(zs, ids, te, ns), M * ns * 6, like="gated_act")
+        W, ns, rows = 1024, 64, 16
+        x1, s1, wg, wp, w1 = rnd(rows, W), rnd(rows, W, dtype=torch.float32), rnd(ns, W), rnd(W, ns), rnd(W)
+        wl, te = rnd(2 * ns, W), rnd(50280, ns)
+        record("decode_linear_gated", "rows=16 K=1024 N=128 (Based, Razesun): the same weight bytes", lambda: ops.decode_linear(x1, wl, epilogue="gated"), 4 * ns * W)
+        record("token_side_step", "rows=16 W=1024 n=64: two products, gate, norm, stream", lambda: ops.token_side_step(
+               s1, x1, ids[0, :rows], wg, wp, te, 0, w1), 4 * ns * W + rows * W * 14, like="decode_linear_gated")
     return out
 
 
