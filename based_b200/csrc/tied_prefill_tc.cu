@@ -9,7 +9,9 @@
 // A tile of 128 keys is loaded once (64-column atoms, 128-byte swizzle) and is the K-major operand of S and the MN-major
 // operand of O; its 128 factors come with it by an untiled bulk copy.  The accumulator is rescaled only when a row's
 // maximum grew by more than 2^8 since the last rescale; the reader of S(j) may touch O because S(j) was issued behind
-// P K (j-1) and its commit covers both.
+// P K (j-1) and its commit covers both.  A tile's Q is free when its last S has been computed: the gate tile is loaded into
+// its place by TMA under the last softmax, replaced by the output, and stored from there by TMA (a thread owns a row, and
+// rows are far apart in memory).
 #include <initializer_list>
 #include <mutex>
 
@@ -26,18 +28,18 @@ namespace {
 using namespace tc;
 
 constexpr int TQ = 128, TK = 128;
-constexpr int NT = 320;
+constexpr int NT = 384;                // two softmax warpgroups; producer, MMA and two idle warps
+// registers per thread: 168 at launch, 3 * 168 = 2 * 232 + 40 after the split
+constexpr int kSoftmaxRegs = 232, kOtherRegs = 40;
 constexpr uint32_t kAtom = 128 * 128;  // bytes
 constexpr int kMaxStages = 6;
 constexpr float kRescale = 8.0f;       // log2 units
 
 struct Params {
-  CUtensorMap mq, mk;
+  CUtensorMap mq, mk, mg, mo;    // q, gate and out [B][H][L][d], cache [B][G][T][d]
   const float* factor;
-  const __nv_bfloat16* gate;
-  __nv_bfloat16* out;
-  int64_t fb, fh, gb, gl, ob, ol;
-  int offset, L, group, d, atoms, stages;
+  int64_t fb, fh;
+  int offset, L, group, d, atoms, stages, gated;
   float scale_log2e, sink;
   unsigned int* status;
 };
@@ -53,6 +55,12 @@ __device__ __forceinline__ void mul2(uint32_t& a, uint32_t& b, float fa, float f
       : "+r"(a), "+r"(b) : "f"(fa), "f"(fb));
 }
 
+__device__ __forceinline__ uint64_t pair(float lo, float hi) { uint64_t r; asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(lo), "f"(hi)); return r; }
+__device__ __forceinline__ void split(uint64_t v, float& lo, float& hi) { asm("mov.b64 {%0, %1}, %2;" : "=f"(lo), "=f"(hi) : "l"(v)); }
+__device__ __forceinline__ uint64_t add2(uint64_t a, uint64_t b) { uint64_t r; asm("add.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b)); return r; }
+__device__ __forceinline__ uint64_t fma2(uint64_t a, uint64_t b, uint64_t c) { uint64_t r; asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c)); return r; }
+__device__ __forceinline__ float max3(float a, float b, float c) { float r; asm("max.f32 %0, %1, %2, %3;" : "=f"(r) : "f"(a), "f"(b), "f"(c)); return r; }
+
 __global__ void __launch_bounds__(NT, 1) tied_prefill_tc_kernel(const __grid_constant__ Params p) {
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = smem_raw + ((1024u - (smem_u32(smem_raw) & 1023u)) & 1023u);
@@ -63,10 +71,10 @@ __global__ void __launch_bounds__(NT, 1) tied_prefill_tc_kernel(const __grid_con
   const int na = p.atoms;
   const uint32_t kTile = (uint32_t)na * kAtom;
   const uint32_t SM_K = 2u * kTile, SM_F = SM_K + (uint32_t)p.stages * kTile, SM_BAR = SM_F + (uint32_t)p.stages * TK * 4;
-  // barriers: q, full[stages], empty[stages], s_full[2], p_full[2], o_full[2]
+  // barriers: q, full[stages], empty[stages], s_full[2], p_full[2], o_full[2], gate[2]
   const uint32_t B_Q = sb + SM_BAR, B_F = B_Q + 8, B_E = B_F + 8 * kMaxStages, B_S = B_E + 8 * kMaxStages, B_P = B_S + 16,
-                 B_O = B_P + 16;
-  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(smem + SM_BAR + 8 * (1 + 2 * kMaxStages + 6));
+                 B_O = B_P + 16, B_G = B_O + 16;
+  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(smem + SM_BAR + 8 * (1 + 2 * kMaxStages + 8));
   volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_slot + 1);
 
   // keys tile x's last row sees, in tiles (a tile with no valid row at all is skipped)
@@ -81,7 +89,7 @@ __global__ void __launch_bounds__(NT, 1) tied_prefill_tc_kernel(const __grid_con
   if (tid == 0) {
     mbar_init(B_Q, 1);
     for (int i = 0; i < p.stages; ++i) { mbar_init(B_F + 8 * i, 1); mbar_init(B_E + 8 * i, 1); }
-    for (int x = 0; x < 2; ++x) { mbar_init(B_S + 8 * x, 1); mbar_init(B_P + 8 * x, TQ); mbar_init(B_O + 8 * x, 1); }
+    for (int x = 0; x < 2; ++x) { mbar_init(B_S + 8 * x, 1); mbar_init(B_P + 8 * x, TQ); mbar_init(B_O + 8 * x, 1); mbar_init(B_G + 8 * x, 1); }
     *abort_flag = 0;
     fence_mbar_init();
     fence_proxy_async();
@@ -93,7 +101,9 @@ __global__ void __launch_bounds__(NT, 1) tied_prefill_tc_kernel(const __grid_con
   const uint32_t tmem = *tmem_slot;
   const uint32_t TM_S[2] = {0u, 128u}, TM_O[2] = {256u, 384u};
 
-  if (warp == 8) {
+  if (warp >= 8) {
+    asm volatile("setmaxnreg.dec.sync.aligned.u32 %0;" ::"n"(kOtherRegs));
+    if (warp == 8) {
     // ---------------- producer
     if (lane == 0) {
       const int nx = ntile[1] > 0 ? 2 : 1;
@@ -111,7 +121,7 @@ __global__ void __launch_bounds__(NT, 1) tied_prefill_tc_kernel(const __grid_con
         if (++st == p.stages) { st = 0; ph ^= 1; }
       }
     }
-  } else if (warp == 9) {
+    } else if (warp == 9) {
     // ---------------- MMA issue (converged warp, one elected lane)
     const uint32_t tmem_u = __shfl_sync(0xffffffffu, tmem, 0);
     const bool leader = elect_one_sync();
@@ -157,7 +167,9 @@ __global__ void __launch_bounds__(NT, 1) tied_prefill_tc_kernel(const __grid_con
       if (++next == p.stages) { next = 0; ph ^= 1; }
       __syncwarp();
     }
+    }
   } else {
+    asm volatile("setmaxnreg.inc.sync.aligned.u32 %0;" ::"n"(kSoftmaxRegs));
     // ---------------- softmax: one query row per thread
     const int x = warp >> 2, row = tid & 127;
     const int n = x == 0 ? ntile[0] : ntile[1];
@@ -172,6 +184,11 @@ __global__ void __launch_bounds__(NT, 1) tied_prefill_tc_kernel(const __grid_con
       mbar_wait_bounded(bs, j & 1, abort_flag, p.status, 1u << 13);   // S(j) read tile j, so its factors have landed, too
       fence_after_sync();
       mbar_wait_bounded(B_F + 8 * st, (j / p.stages) & 1, abort_flag, p.status, 1u << 12);
+      if (p.gated && j == n - 1 && row == 0) {
+        tma::mbar_expect_tx(B_G + 8 * x, kTile);
+        for (int a = 0; a < na; ++a) tma::load_4d(sb + x * kTile + a * kAtom, &p.mg, B_G + 8 * x, 64 * a, q0 + x * TQ, h, b);
+      }
+      __syncwarp();
       uint32_t r[4][32];
 #pragma unroll
       for (int c = 0; c < 4; ++c) tmem_ld32(ts + 32 * c, r[c]);
@@ -198,7 +215,7 @@ __global__ void __launch_bounds__(NT, 1) tied_prefill_tc_kernel(const __grid_con
 #pragma unroll
       for (int c = 0; c < 4; ++c)
 #pragma unroll
-        for (int i = 0; i < 32; ++i) m4[i & 3] = fmaxf(m4[i & 3], __uint_as_float(r[c][i]));
+        for (int i = 0; i < 32; i += 2) m4[(i >> 1) & 3] = max3(m4[(i >> 1) & 3], __uint_as_float(r[c][i]), __uint_as_float(r[c][i + 1]));
       const float mt = fmaxf(fmaxf(m4[0], m4[1]), fmaxf(m4[2], m4[3])) * p.scale_log2e;
       const bool grow = mt > m + kRescale;
       if (j == 0) {                             // the sink is one more score of 0
@@ -219,20 +236,25 @@ __global__ void __launch_bounds__(NT, 1) tied_prefill_tc_kernel(const __grid_con
         }
         tmem_st_wait();
       }
-      float s4[4] = {0.f, 0.f, 0.f, 0.f};
+      uint64_t s2[4] = {0ull, 0ull, 0ull, 0ull};
+      const uint64_t sc2 = pair(p.scale_log2e, p.scale_log2e), nm2 = pair(-m, -m);
 #pragma unroll
       for (int c = 0; c < 4; ++c) {
         uint32_t pk[16];
 #pragma unroll
         for (int i = 0; i < 16; ++i) {
-          const float e0 = ex2(fmaf(__uint_as_float(r[c][2 * i]), p.scale_log2e, -m));
-          const float e1 = ex2(fmaf(__uint_as_float(r[c][2 * i + 1]), p.scale_log2e, -m));
-          s4[i & 3] += e0 + e1;
+          float e0, e1;
+          split(fma2(pair(__uint_as_float(r[c][2 * i]), __uint_as_float(r[c][2 * i + 1])), sc2, nm2), e0, e1);
+          e0 = ex2(e0);
+          e1 = ex2(e1);
+          s2[i & 3] = add2(s2[i & 3], pair(e0, e1));
           pk[i] = pack_bf16(e0, e1);
         }
         tmem_st16(ts + 16 * c, pk);
       }
-      sum += (s4[0] + s4[1]) + (s4[2] + s4[3]);
+      float sl, sh;
+      split(add2(add2(s2[0], s2[1]), add2(s2[2], s2[3])), sl, sh);
+      sum += sl + sh;
       tmem_st_wait();
       fence_before_sync();
       mbar_arrive(bp);
@@ -240,29 +262,34 @@ __global__ void __launch_bounds__(NT, 1) tied_prefill_tc_kernel(const __grid_con
     if (n > 0) {
       mbar_wait_bounded(B_O + 8 * x, 0, abort_flag, p.status, 1u << 14);
       fence_after_sync();
+      if (p.gated) mbar_wait_bounded(B_G + 8 * x, 0, abort_flag, p.status, 1u << 15);
       const float f = 1.0f / sum;
-      const bool live = qi < p.L;
-      const int64_t col = (int64_t)h * p.d;
-      const __nv_bfloat16* gate = p.gate ? p.gate + b * p.gb + (int64_t)qi * p.gl + col : nullptr;
-      __nv_bfloat16* o = p.out + b * p.ob + (int64_t)qi * p.ol + col;
+      uint8_t* tile = smem + x * kTile;
       for (int c = 0; c < p.d; c += 16) {
         uint32_t t[16];
         tmem_ld16(to + c, t);
         tmem_ld_wait();
-        if (live) {
 #pragma unroll
-          for (int i = 0; i < 16; i += 8) {
-            float y[8], z[8];
+        for (int i = 0; i < 16; i += 8) {
+          __nv_bfloat16* at = reinterpret_cast<__nv_bfloat16*>(tile + (c >> 6) * kAtom + tma::sw128_offset(row, ((c & 63) + i) >> 3));
+          float y[8], z[8];
 #pragma unroll
-            for (int e = 0; e < 8; ++e) y[e] = __uint_as_float(t[i + e]) * f;
-            if (gate) {
-              seq::Pack<__nv_bfloat16, 8>::load(gate + c + i, z);
+          for (int e = 0; e < 8; ++e) y[e] = __uint_as_float(t[i + e]) * f;
+          if (p.gated) {
+            seq::Pack<__nv_bfloat16, 8>::load(at, z);
 #pragma unroll
-              for (int e = 0; e < 8; ++e) y[e] *= seq::sigmoid_t<__nv_bfloat16>(z[e]);
-            }
-            seq::Pack<__nv_bfloat16, 8>::store(o + c + i, y);
+            for (int e = 0; e < 8; ++e) y[e] *= seq::sigmoid_t<__nv_bfloat16>(z[e]);
           }
+          seq::Pack<__nv_bfloat16, 8>::store(at, y);
         }
+      }
+      fence_proxy_async();
+      if (x == 0) asm volatile("bar.sync 1, 128;" ::: "memory");   // this tile's four warps
+      else asm volatile("bar.sync 2, 128;" ::: "memory");
+      if (row == 0) {                           // rows past the call's tokens are clipped
+        for (int a = 0; a < na; ++a) tma::store_4d(&p.mo, sb + x * kTile + a * kAtom, 64 * a, q0 + x * TQ, h, b);
+        bulk_commit();
+        bulk_wait_all();
       }
     }
   }
@@ -301,7 +328,7 @@ int launch_tied_prefill_tc(const void* q, const void* cache, const float* factor
   auto fix = [&](int64_t s, int extent) { return extent == 1 ? (int64_t)8 : s; };
   for (int64_t s : {fix(qb, B), fix(ql, L), fix(cb, B), fix(cl, T), fix(ob, B), fix(ol, L)})
     if (s % 8 != 0 || s <= 0) return BASED_ERR_IMPL;
-  if (gate && ((B > 1 && gb % 8) || (L > 1 && gl % 8))) return BASED_ERR_IMPL;
+  if (gate && (fix(gb, B) % 8 || fix(gb, B) <= 0 || fix(gl, L) % 8 || fix(gl, L) <= 0)) return BASED_ERR_IMPL;
   if ((G > 1 && fh % 4) || (B > 1 && fb % 4) || fh < (int64_t)(T + TK - 1) / TK * TK) return BASED_ERR_IMPL;
   Params p;
   p.atoms = (d + 63) / 64;
@@ -318,10 +345,10 @@ int launch_tied_prefill_tc(const void* q, const void* cache, const float* factor
     return 0;
   };
   if (get_map(&p.mq, q, L, H, ql, qb) || get_map(&p.mk, cache, T, G, cl, cb)) return BASED_ERR_IMPL;
+  p.gated = gate != nullptr;
+  if (get_map(&p.mo, out, L, H, ol, ob) || (p.gated && get_map(&p.mg, gate, L, H, gl, gb))) return BASED_ERR_IMPL;
   p.factor = factor;
-  p.gate = static_cast<const __nv_bfloat16*>(gate);
-  p.out = static_cast<__nv_bfloat16*>(out);
-  p.fb = fb; p.fh = fh; p.gb = gb; p.gl = gl; p.ob = ob; p.ol = ol;
+  p.fb = fb; p.fh = fh;
   p.offset = offset; p.L = L; p.group = H / G; p.d = d;
   p.scale_log2e = scale * 1.4426950408889634f;
   p.sink = sink;
