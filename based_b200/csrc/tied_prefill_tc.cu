@@ -5,7 +5,7 @@
 //   warps 0-3 / 4-7   softmax of tile 0 / 1, one query row per thread: S (TMEM) -> P (bf16, in S's columns)
 //   warp 8            TMA producer
 //   warp 9            MMA issue: S_x(j+1) = Q_x K(j+1)^T right behind O_x += P_x(j) K(j), so that one tile's softmax runs
-//                     under the other tile's products
+//                     under the other tile's products; P is handed over in two halves
 // A tile of 128 keys is loaded once (64-column atoms, 128-byte swizzle) and is the K-major operand of S and the MN-major
 // operand of O; its 128 factors come with it by an untiled bulk copy.  The accumulator is rescaled only when a row's
 // maximum grew by more than 2^8 since the last rescale; the reader of S(j) may touch O because S(j) was issued behind
@@ -71,10 +71,10 @@ __global__ void __launch_bounds__(NT, 1) tied_prefill_tc_kernel(const __grid_con
   const int na = p.atoms;
   const uint32_t kTile = (uint32_t)na * kAtom;
   const uint32_t SM_K = 2u * kTile, SM_F = SM_K + (uint32_t)p.stages * kTile, SM_BAR = SM_F + (uint32_t)p.stages * TK * 4;
-  // barriers: q, full[stages], empty[stages], s_full[2], p_full[2], o_full[2], gate[2]
+  // barriers: q, full[stages], empty[stages], s_full[2], p_full[2], o_full[2], gate[2], first half of P[2]
   const uint32_t B_Q = sb + SM_BAR, B_F = B_Q + 8, B_E = B_F + 8 * kMaxStages, B_S = B_E + 8 * kMaxStages, B_P = B_S + 16,
-                 B_O = B_P + 16, B_G = B_O + 16;
-  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(smem + SM_BAR + 8 * (1 + 2 * kMaxStages + 8));
+                 B_O = B_P + 16, B_G = B_O + 16, B_H = B_G + 16;
+  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(smem + SM_BAR + 8 * (1 + 2 * kMaxStages + 10));
   volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_slot + 1);
 
   // keys tile x's last row sees, in tiles (a tile with no valid row at all is skipped)
@@ -89,7 +89,7 @@ __global__ void __launch_bounds__(NT, 1) tied_prefill_tc_kernel(const __grid_con
   if (tid == 0) {
     mbar_init(B_Q, 1);
     for (int i = 0; i < p.stages; ++i) { mbar_init(B_F + 8 * i, 1); mbar_init(B_E + 8 * i, 1); }
-    for (int x = 0; x < 2; ++x) { mbar_init(B_S + 8 * x, 1); mbar_init(B_P + 8 * x, TQ); mbar_init(B_O + 8 * x, 1); mbar_init(B_G + 8 * x, 1); }
+    for (int x = 0; x < 2; ++x) { mbar_init(B_S + 8 * x, 1); mbar_init(B_P + 8 * x, TQ); mbar_init(B_O + 8 * x, 1); mbar_init(B_G + 8 * x, 1); mbar_init(B_H + 8 * x, TQ); }
     *abort_flag = 0;
     fence_mbar_init();
     fence_proxy_async();
@@ -138,11 +138,13 @@ __global__ void __launch_bounds__(NT, 1) tied_prefill_tc_kernel(const __grid_con
       }
       if (leader) mma_commit(B_S + 8 * x);
     };
-    auto issue_o = [&](int x, int j, int st) {
+    auto issue_o = [&](int x, int j, int st, int k0) {
       const uint64_t dv = make_smem_desc_sw128(sb + SM_K + st * kTile, kAtom, 1024);
 #pragma unroll
-      for (int k = 0; k < TK / 16; ++k)   // 16 keys are 2048 bytes
+      for (int kk = 0; kk < TK / 32; ++kk) {   // 16 keys are 2048 bytes
+        const int k = k0 + kk;
         if (leader) mma_ts(tmem_u + TM_O[x], tmem_u + TM_S[x] + 8 * k, dv + 128 * k, idesc_o, (j > 0 || k > 0) ? 1u : 0u);
+      }
     };
     mbar_wait_bounded(B_Q, 0, abort_flag, p.status, 1u << 9);
     int st = 0, next = 0, ph = 0;   // stages of tiles j and j + 1, phase of the latter
@@ -155,9 +157,12 @@ __global__ void __launch_bounds__(NT, 1) tied_prefill_tc_kernel(const __grid_con
 #pragma unroll
       for (int x = 0; x < 2; ++x) {
         if (j >= 0 && j < ntile[x]) {
+          mbar_wait_bounded(B_H + 8 * x, j & 1, abort_flag, p.status, 1u << 16);
+          fence_after_sync();
+          issue_o(x, j, st, 0);
           mbar_wait_bounded(B_P + 8 * x, j & 1, abort_flag, p.status, 1u << 11);
           fence_after_sync();
-          issue_o(x, j, st);
+          issue_o(x, j, st, 4);
           if (j == ntile[x] - 1 && leader) mma_commit(B_O + 8 * x);
         }
         if (more && j + 1 < ntile[x]) issue_s(x, next);
@@ -251,6 +256,11 @@ __global__ void __launch_bounds__(NT, 1) tied_prefill_tc_kernel(const __grid_con
           pk[i] = pack_bf16(e0, e1);
         }
         tmem_st16(ts + 16 * c, pk);
+        if (c == 1) {                           // the products of keys 0-63 may start
+          tmem_st_wait();
+          fence_before_sync();
+          mbar_arrive(B_H + 8 * x);
+        }
       }
       float sl, sh;
       split(add2(add2(s2[0], s2[1]), add2(s2[2], s2[3])), sl, sh);

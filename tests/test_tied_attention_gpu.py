@@ -230,10 +230,10 @@ def test_cache_rows_and_factors():
 def test_a_used_cache_is_used_again():
     """A longer sequence's keys and factors are left in the cache of a shorter one."""
     from based_b200 import ops
-    st = ops.tied_attention_state(1, 4, 1, 64, 300, torch.bfloat16, "cuda")
-    first = case(4, 1, 64, 300, seed=11)
+    st = ops.tied_attention_state(1, 5, 1, 80, 300, torch.bfloat16, "cuda")
+    first = case(5, 1, 80, 300, seed=11)
     check(first, product(*first, [300], state=st), TOL)
-    second = case(4, 1, 64, 61, seed=12)
+    second = case(5, 1, 80, 61, seed=12)
     for cuts in ([61], [50, 1], [1]):
         st["keys"][:, 61:] = 50.0                          # whatever is left behind the sequence's end
         st["factor"][..., 61:] = 1e30
