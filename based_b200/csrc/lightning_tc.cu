@@ -30,7 +30,7 @@ using namespace tc;
 using bf16 = __nv_bfloat16;
 
 constexpr int C = 128;                      // tokens per chunk
-constexpr int kLoaders = 512, NT = 12 * 32 + kLoaders;   // seven warpgroups; two of them idle
+constexpr int kLoaders = 512, NT = 12 * 32 + kLoaders;   // seven warpgroups; warps 10 and 11 are idle
 // registers per thread: 72 at launch; the loaders take what the others leave (7 * 72 = 72 + 40 + 40 + 4 * 88)
 constexpr int kStateRegs = 40, kMmaRegs = 40, kLoadRegs = 88;
 constexpr int kItems = C * 16 / kLoaders;   // 16-byte pieces per thread and tensor at 128 columns
